@@ -20,7 +20,7 @@ from typing import Dict, Optional
 
 import torch
 
-from ..parts.base import CacheParts, FixedState, PagedKV, PagedLatent  # noqa: F401  (CacheParts: part of this module's interface)
+from ..parts.base import BorrowedCache, CacheParts, FixedState, PagedKV, PagedLatent  # noqa: F401  (CacheParts: part of this module's interface)
 
 
 @dataclass
@@ -49,6 +49,10 @@ class CacheKind:
 
     def keep_first(self, spec) -> int:
         """With a window: the first positions that stay readable all the same."""
+        return 0
+
+    def chunk(self, spec) -> int:
+        """The length of the runs that queries read within (0: none).  Pages before the next query's run are given back."""
         return 0
 
     def page_bytes(self, spec, page_size: int, element_bytes: int) -> int:
@@ -88,6 +92,9 @@ class PagedKVKind(CacheKind):
 
     def keep_first(self, spec: PagedKV) -> int:
         return spec.keep_first if spec.window > 0 else 0
+
+    def chunk(self, spec: PagedKV) -> int:
+        return spec.chunk
 
     def page_bytes(self, spec: PagedKV, page_size, element_bytes):
         return (spec.num_kv_heads * spec.head_dim + spec.value_heads * spec.value_dim) * page_size * element_bytes
@@ -140,6 +147,15 @@ class FixedStateKind(CacheKind):
 
     def allocate_state(self, spec: FixedState, slots, device):
         return torch.zeros((slots,) + tuple(spec.shape), dtype=getattr(torch, spec.dtype), device=device)
+
+
+def flat_specs(spec) -> list:
+    """The needs that a place's spec is made of, without those that keep nothing: `CacheParts` opened, however deep."""
+    if spec is None or isinstance(spec, BorrowedCache):
+        return []
+    if isinstance(spec, CacheParts):
+        return [m for part in spec.parts for m in flat_specs(part)]
+    return [spec]
 
 
 _KINDS: Dict[type, CacheKind] = {}

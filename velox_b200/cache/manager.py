@@ -36,7 +36,7 @@ import torch
 
 from .. import native
 from ..native import OutOfPages  # noqa: F401  (part of this module's interface)
-from .kinds import CacheKind, CacheParts, LayerCache, cache_kind
+from .kinds import BorrowedCache, CacheKind, CacheParts, LayerCache, cache_kind, flat_specs
 from .pages import CacheAccountingError, PageAllocator, SlotAllocator
 
 
@@ -99,21 +99,21 @@ class CacheManager:
         self.groups: List[CacheGroup] = []
         self._layers: List[LayerCache] = []
         self._state_layers: List[int] = []
-        # A place whose mixer is made of several (`CacheParts`) has one cell per member;
-        # every other place has one cell.  Cells are what groups and state tensors are made of.
+        # A place whose need is made of several (`CacheParts`, at any depth) has one cell per member that keeps
+        # something.  Cells are what groups and state tensors are made of.
         cells: List[object] = []
         cells_of_place: List[List[int]] = []
         for spec in cache_specs:
-            members = list(spec.parts) if isinstance(spec, CacheParts) else [spec]
+            members = flat_specs(spec)
             cells_of_place.append(list(range(len(cells), len(cells) + len(members))))
             cells.extend(members)
         by_spec: Dict[object, int] = {}
         cell_group = [-1] * len(cells)
         specs_of_groups: List[object] = []
         cells_of_groups: List[List[int]] = []
-        kinds = [None if spec is None else cache_kind(spec) for spec in cells]
+        kinds = [cache_kind(spec) for spec in cells]
         for c, spec in enumerate(cells):
-            if spec is not None and kinds[c].paged:
+            if kinds[c].paged:
                 if spec not in by_spec:
                     by_spec[spec] = len(specs_of_groups)
                     specs_of_groups.append(spec)
@@ -134,6 +134,9 @@ class CacheManager:
             kept = int(cache_kind(spec).keep_first(spec))
             if kept:
                 native.check(self._lib.vxh_cache_set_keep_first(self._book, g, kept))
+            chunk = int(cache_kind(spec).chunk(spec))
+            if chunk:
+                native.check(self._lib.vxh_cache_set_chunk(self._book, g, chunk))
         self.slots = SlotAllocator(0, _borrowed=self._lib.vxh_cache_slots(self._book), _owner=self)
         for g, (spec, members) in enumerate(zip(specs_of_groups, cells_of_groups)):
             self.groups.append(CacheGroup(spec, cache_kind(spec), sorted({place_of_cell[c] for c in members}),
@@ -155,9 +158,7 @@ class CacheManager:
         self._states: List = []
         cell_cache: List[LayerCache] = []
         for c, spec in enumerate(cells):
-            if spec is None:
-                cell_cache.append(LayerCache())
-            elif kinds[c].paged:
+            if kinds[c].paged:
                 g = self.groups[cell_group[c]]
                 cell_cache.append(g.kind.layer_cache_of(g.spec, g.storage, cells_of_groups[cell_group[c]].index(c),
                                                         cell_group[c], self.page_size))
@@ -168,11 +169,23 @@ class CacheManager:
                 if place_of_cell[c] not in self._state_layers:
                     self._state_layers.append(place_of_cell[c])
         for i, spec in enumerate(cache_specs):
-            mine = [cell_cache[c] for c in cells_of_place[i]]
-            self._layers.append(LayerCache(parts=mine) if isinstance(spec, CacheParts) else mine[0])
-        for i, j in enumerate(cache_of):
-            if j is not None:
-                self._layers[i] = self._reader(self._layers[j])
+            lender = self._layers[cache_of[i]] if i < len(cache_of) and cache_of[i] is not None else None
+            self._layers.append(self._assemble(spec, iter([cell_cache[c] for c in cells_of_place[i]]), lender))
+
+    @classmethod
+    def _assemble(cls, spec, cells: Iterator[LayerCache], lender: Optional[LayerCache]) -> LayerCache:
+        """A place's cache from its cells, in the order of its spec; what it keeps nothing of itself is read from `lender`,
+        the cache of the earlier place that it names."""
+        if isinstance(spec, CacheParts):
+            lent = lender.parts if lender is not None and lender.parts is not None else [None] * len(spec.parts)
+            if len(lent) != len(spec.parts):
+                raise ValueError("a place reads the cache of one that is made of another number of parts")
+            return LayerCache(parts=[cls._assemble(s, cells, l) for s, l in zip(spec.parts, lent)])
+        if isinstance(spec, BorrowedCache) and lender is None:
+            raise ValueError("a place borrows a cache but names no earlier place that has it")
+        if spec is None or isinstance(spec, BorrowedCache):
+            return cls._reader(lender) if lender is not None else LayerCache()
+        return next(cells)
 
     @classmethod
     def _reader(cls, src: LayerCache) -> LayerCache:

@@ -756,3 +756,152 @@ class FovenexConfig(ModelConfig):
                 positive(at + ".mlp", mlp, "ff")
         if faults:
             raise ConfigError("Fovenex configuration: " + "; ".join(faults))
+
+
+@dataclass(frozen=True)
+class NegilornConfig(ModelConfig):
+    """Negilorn: a decoder whose config.json is nested and lists its layers one by one.
+
+        architecture   "Negilorn"
+        vocab, width, norm.eps
+        logit_scale    multiplier of the logits (absent: 1)
+        layers[i]      type "attention":  mixer (heads, kv_heads, dim, vdim, scale, softcap (optional bound of the scores),
+                                          rot.base, rot.dims, rot.scaling.{factor, low, high, original} (optional),
+                                          mask.size (the length of a chunk; absent: the whole sequence),
+                                          kv_from (optional: the layer whose cached keys and values it reads))
+                       type "wkv":        mixer (heads, dim; optional rank: the middle width of the decay's projection, otherwise
+                                          read off the weight file)
+                       mlp: null | kind "dense" (ff)
+                            | kind "moe" (router.experts, router.top, expert.ff, shared.ff (optional))
+
+    Every size and constant is read from there; the layers may differ from one another."""
+
+    architecture: ClassVar[str] = "Negilorn"
+    model_type: ClassVar[str] = "negilorn"
+    LAYER_TYPES: ClassVar[Tuple[str, ...]] = ("attention", "wkv")
+
+    vocab: int = _field(int)
+    width: int = _field(int)
+    norm_eps: float = _field(float)
+    logit_scale: float = _field(float, default=1.0)
+    layers: Tuple[Dict[str, Any], ...] = _field(tuple, default=())
+
+    @classmethod
+    def from_dict(cls, raw: Dict[str, Any]) -> "NegilornConfig":
+        faults: list = []
+
+        def get(d, path, kind, default=dataclasses.MISSING):
+            cur = d
+            for key in path.split("."):
+                if not isinstance(cur, dict) or cur.get(key) is None:
+                    if default is dataclasses.MISSING:
+                        faults.append("missing key %r" % path)
+                    return None if default is dataclasses.MISSING else default
+                cur = cur[key]
+            return _typed(path, cur, kind, faults)
+
+        values = dict(vocab=get(raw, "vocab", int), width=get(raw, "width", int), norm_eps=get(raw, "norm.eps", float),
+                      logit_scale=get(raw, "logit_scale", float, 1.0))
+        layers = raw.get("layers")
+        if not isinstance(layers, list) or not layers:
+            faults.append("key 'layers': expected a list of layers")
+            layers = []
+        if faults:
+            raise ConfigError("config.json for %s: %s" % (cls.__name__, "; ".join(faults)))
+        cfg = cls(layers=tuple(json.loads(json.dumps(layer)) for layer in layers), **values)
+        cfg.validate()
+        return cfg
+
+    def to_dict(self) -> Dict[str, Any]:
+        return {"architecture": self.architecture, "layers": json.loads(json.dumps(list(self.layers))),
+                "logit_scale": self.logit_scale, "norm": {"eps": self.norm_eps}, "vocab": self.vocab, "width": self.width}
+
+    def chunk_of(self, i: int) -> int:
+        """The length of layer i's chunks, 0 for a layer that sees the whole sequence."""
+        mask = (self.layers[i].get("mixer") or {}).get("mask")
+        return int(mask.get("size") or 0) if isinstance(mask, dict) else 0
+
+    def kv_source(self, i: int) -> Optional[int]:
+        """The layer whose cached keys and values layer i reads, or None if it makes its own (or is no attention)."""
+        m = self.layers[i].get("mixer") or {}
+        return m.get("kv_from") if self.layers[i].get("type") == "attention" else None
+
+    def validate(self) -> None:
+        faults = []
+
+        def positive(where, d, *keys):
+            ok = True
+            for k in keys:
+                v = d.get(k) if isinstance(d, dict) else None
+                if not isinstance(v, int) or isinstance(v, bool) or v <= 0:
+                    faults.append("%s.%s must be a positive integer, got %r" % (where, k, v))
+                    ok = False
+            return ok
+
+        def number(where, d, key, least=None, required=True):
+            v = d.get(key) if isinstance(d, dict) else None
+            if v is None and not required:
+                return True
+            if not isinstance(v, (int, float)) or isinstance(v, bool) or (least is not None and not v > least):
+                faults.append("%s.%s must be a number%s, got %r" % (where, key, "" if least is None else " above %g" % least, v))
+                return False
+            return True
+
+        for name in ("vocab", "width"):
+            if getattr(self, name) <= 0:
+                faults.append("%s must be positive, got %d" % (name, getattr(self, name)))
+        if not self.norm_eps > 0:
+            faults.append("norm.eps must be positive, got %r" % self.norm_eps)
+        for i, layer in enumerate(self.layers):
+            at = "layers[%d]" % i
+            if not isinstance(layer, dict) or layer.get("type") not in self.LAYER_TYPES:
+                faults.append("%s.type %r is not one of %s" % (at, layer.get("type") if isinstance(layer, dict) else layer,
+                                                               list(self.LAYER_TYPES)))
+                continue
+            m, where = layer.get("mixer"), at + ".mixer"
+            if layer["type"] == "attention":
+                if positive(where, m, "heads", "kv_heads", "dim", "vdim"):
+                    if m["heads"] % m["kv_heads"]:
+                        faults.append("%s: heads (%d) is not a multiple of kv_heads (%d)" % (where, m["heads"], m["kv_heads"]))
+                    number(where, m, "scale")
+                    number(where, m, "softcap", 0, required=False)
+                    rot = m.get("rot")
+                    if rot is not None and number(where + ".rot", rot, "base", 0) and (rot.get("dims") is None or positive(where + ".rot", rot, "dims")):
+                        dims = rot.get("dims") or m["dim"]
+                        if dims % 2 or dims > m["dim"]:
+                            faults.append("%s.rot.dims (%d) must be even and within the head's %d channels" % (where, dims, m["dim"]))
+                        if rot.get("scaling"):
+                            for key in ("factor", "low", "high", "original"):
+                                number(where + ".rot.scaling", rot["scaling"], key, 0)
+                    mask = m.get("mask")
+                    if mask is not None and not isinstance(mask, dict):
+                        faults.append("%s.mask must hold a size, got %r" % (where, mask))
+                    elif mask:
+                        positive(where + ".mask", mask, "size")
+                    j = m.get("kv_from")
+                    if j is not None:
+                        src = self.layers[j] if isinstance(j, int) and not isinstance(j, bool) and 0 <= j < i else None
+                        sm = src.get("mixer") if isinstance(src, dict) and src.get("type") == "attention" else None
+                        if not isinstance(sm, dict) or sm.get("kv_from") is not None:
+                            faults.append("%s.kv_from %r must name an earlier attention layer with keys and values of its own" % (where, j))
+                        elif any(sm.get(k) != m[k] for k in ("kv_heads", "dim", "vdim")):
+                            faults.append("%s.kv_from %d: kv_heads, dim and vdim must equal that layer's" % (where, j))
+            elif positive(where, m, "heads", "dim") and m.get("rank") is not None:
+                positive(where, m, "rank")
+            mlp = layer.get("mlp")
+            if mlp is None:
+                continue
+            kind = mlp.get("kind") if isinstance(mlp, dict) else None
+            if kind == "dense":
+                positive(at + ".mlp", mlp, "ff")
+            elif kind == "moe":
+                positive(at + ".mlp.expert", mlp.get("expert"), "ff")
+                router = mlp.get("router")
+                if positive(at + ".mlp.router", router, "experts", "top") and router["top"] > router["experts"]:
+                    faults.append("%s.mlp.router: top (%d) exceeds experts (%d)" % (at, router["top"], router["experts"]))
+                if mlp.get("shared") is not None:
+                    positive(at + ".mlp.shared", mlp["shared"], "ff")
+            else:
+                faults.append("%s.mlp.kind %r is not 'dense' or 'moe'" % (at, kind if isinstance(mlp, dict) else mlp))
+        if faults:
+            raise ConfigError("Negilorn configuration: " + "; ".join(faults))

@@ -3,6 +3,7 @@
 //
 //   score(i, j) = q_i . k_j * scale - slope_h * (i - j),   slope_h = 2^(-bias_exp * (h + 1) / H)
 //   query i sees key j  iff  j <= i and (window == 0 or i - j < window or j < keep_first)
+//                       and, with a chunk, j and i lie in the same run of `chunk` positions counted from 0
 //   keys of size DK (64, 128), values of size DV (32, 64, 128), which need not be equal; also equal sizes of
 //   32, 48, 80, 96 and 112 (a row of a size that is no power of two lies in shared memory padded to the next one)
 //   optionally a sink per query head: the softmax's denominator also holds exp(sinks[h]) (no key, no value,
@@ -80,6 +81,13 @@ __device__ __forceinline__ float ab_score(float dot, float scale_log2, float cap
     return cap_arg > 0.f ? cap_log2 * tanhf(dot * cap_arg) : dot * scale_log2;
 }
 
+// The first position that the query at `pos` sees (kept first positions aside).
+__device__ __forceinline__ int ab_first_key(int pos, int window, int chunk) {
+    int lo = window > 0 ? max(0, pos + 1 - window) : 0;
+    if (chunk > 0) lo = max(lo, pos - pos % chunk);
+    return lo;
+}
+
 struct AbSegments {
     const int* cu_seqlens;    // portions: rows of segment s are [cu_seqlens[s], cu_seqlens[s + 1])
     const int* kv_offsets;    //           at positions kv_offsets[s] ..
@@ -94,7 +102,7 @@ biased_attention_kernel(const bf16* __restrict__ q, int q_row_stride, const bf16
                         const bf16* __restrict__ v_pool, const int* __restrict__ block_table, int max_blocks,
                         AbSegments seg, bf16* __restrict__ out, int out_row_stride, float scale_log2, float bias_exp,
                         int window, int keep_first, int H, int Hk, int S, int share_log2,
-                        const float* __restrict__ sinks, int gate_col, float cap_log2, float cap_arg, AbLayout lay) {
+                        const float* __restrict__ sinks, int gate_col, float cap_log2, float cap_arg, AbLayout lay, int chunk) {
     extern __shared__ __align__(128) unsigned char ab_smem[];
     constexpr int KCH = DK / 8, VCH = DV / 8;
     constexpr int KCHP = ab_chunks(KCH), VCHP = ab_chunks(VCH);   // a row's place in shared memory
@@ -128,7 +136,7 @@ biased_attention_kernel(const bf16* __restrict__ q, int q_row_stride, const bf16
     const int hv = lay.v_share > 1 ? hk / lay.v_share : hk;
     const int toks_live = min(toks_per_tile, n_new - t0);
     const int kv_hi = off + t0 + toks_live;                              // one past the tile's last visible key
-    const int kv_lo = window > 0 ? max(0, off + t0 + 1 - window) : 0;    // first key of the first row's window
+    const int kv_lo = ab_first_key(off + t0, window, chunk);             // first key that the first row sees
     const int tile_lo = kv_lo / AB_BN, tile_hi = (kv_hi + AB_BN - 1) / AB_BN;
     const int kept = window > 0 ? keep_first : 0;
     const int n_kept_tiles = min((kept + AB_BN - 1) / AB_BN, tile_lo);   // tiles with kept positions, before the window's
@@ -194,12 +202,12 @@ biased_attention_kernel(const bf16* __restrict__ q, int q_row_stride, const bf16
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
     const int r0 = warp * 16 + (lane >> 2);
     const int pos0 = off + t0 + (r0 >> share_log2), pos1 = off + t0 + ((r0 + 8) >> share_log2);
-    const int lo0 = window > 0 ? pos0 + 1 - window : 0, lo1 = window > 0 ? pos1 + 1 - window : 0;
+    const int lo0 = ab_first_key(pos0, window, chunk), lo1 = ab_first_key(pos1, window, chunk);
     const int hd0 = head0 + (r0 & (share - 1)), hd1 = head0 + ((r0 + 8) & (share - 1));
     const float sl0 = bias_exp > 0.f ? exp2f(-bias_exp * (float)(hd0 + 1) / (float)H) * AB_LOG2E : 0.f;
     const float sl1 = bias_exp > 0.f ? exp2f(-bias_exp * (float)(hd1 + 1) / (float)H) * AB_LOG2E : 0.f;
     const int warp_hi = off + t0 + ((warp * 16 + 15) >> share_log2) + 1;
-    const int warp_lo = window > 0 ? off + t0 + ((warp * 16) >> share_log2) + 1 - window : 0;
+    const int warp_lo = ab_first_key(off + t0 + ((warp * 16) >> share_log2), window, chunk);
 
     for (int i = 0; i < n_tiles; ++i) {
         const int stage = i & 1;
@@ -373,7 +381,7 @@ biased_decode_kernel(const bf16* __restrict__ q, int q_row_stride, const bf16* _
                      const int* __restrict__ seq_of_token, const int* __restrict__ positions, bf16* __restrict__ out,
                      int out_row_stride, float scale_log2, float bias_exp, int window, int keep_first, int H, int Hk,
                      int S, int share_log2, float* __restrict__ scratch, const float* __restrict__ sinks, int gate_col,
-                     float cap_log2, float cap_arg, int v_share, int out_f32) {
+                     float cap_log2, float cap_arg, int v_share, int out_f32, int chunk) {
     extern __shared__ __align__(128) unsigned char ad_smem[];
     constexpr int KCH = DK / 8, VCH = DV / 8;
     constexpr int KCHP = ab_pow2(KCH), VCHP = ab_pow2(VCH);
@@ -393,7 +401,7 @@ biased_decode_kernel(const bf16* __restrict__ q, int q_row_stride, const bf16* _
     const int pos = positions[t];
     const int* bt = block_table + (size_t)seq_of_token[t] * max_blocks;
     const int kv_len = pos + 1;
-    const int start = (window > 0 && kv_len > window) ? kv_len - window : 0;
+    const int start = ab_first_key(pos, window, chunk);
     const int nkept = window > 0 ? min(keep_first, start) : 0;
     const int nkeys = nkept + kv_len - start;
     // with gridDim.z > 1 the groups of 16 keys are cut into as many runs, one a block; the runs' parts go to the
@@ -601,7 +609,7 @@ static int launch_biased_decode(const bf16* q, int q_row_stride, const bf16* k_p
                                 const int* block_table, int max_blocks, const int* seq_of_token, const int* positions,
                                 bf16* out, int out_row_stride, float scale, float bias_exp, int window, int keep_first,
                                 int tokens, int H, int Hk, int S, float* scratch, int runs, const float* sinks, int gate_col,
-                                float softcap, int v_share, int out_f32, cudaStream_t stream) {
+                                float softcap, int v_share, int out_f32, int chunk, cudaStream_t stream) {
     constexpr int KROW = ab_pow2(DK / 8) * 16, VROW = ab_pow2(DV / 8) * 16;
     const size_t walk = (size_t)AD_WARPS * 2 * (16 * KROW + 16 * VROW), parts = (size_t)AD_WARPS * 16 * (DV + 2) * 4;
     const size_t smem = 16 * KROW + (walk > parts ? walk : parts);
@@ -616,7 +624,7 @@ static int launch_biased_decode(const bf16* q, int q_row_stride, const bf16* k_p
     VX_LAUNCH_K(VX_K_ATTENTION, (biased_decode_kernel<DK, DV>), grid, AD_WARPS * 32, smem, stream, q, q_row_stride, k_pool,
                 v_pool, block_table, max_blocks, seq_of_token, positions, out, out_row_stride, scale * AB_LOG2E, bias_exp,
                 window, keep_first, H, Hk, S, share_log2, scratch, sinks, gate_col, softcap * AB_LOG2E,
-                softcap > 0.f ? scale / softcap : 0.f, v_share, out_f32);
+                softcap > 0.f ? scale / softcap : 0.f, v_share, out_f32, chunk);
     if (runs > 1)
         VX_LAUNCH_K(VX_K_JOIN, biased_decode_join_kernel, dim3(tokens, H), DV >= 128 ? 128 : 64, 0, stream, (const float*)scratch,
                     out, out_row_stride, H, DV, runs, sinks, q, q_row_stride, gate_col, out_f32);
@@ -628,7 +636,8 @@ template <int DK, int DV>
 static int launch_biased(const bf16* q, int q_row_stride, const bf16* k_pool, const bf16* v_pool, const int* block_table,
                          int max_blocks, AbSegments seg, bf16* out, int out_row_stride, float scale, float bias_exp,
                          int window, int keep_first, int segments, int max_new, int H, int Hk, int S, const float* sinks,
-                         int gate_col, float softcap, const AbLayout* layout, int v_share, int out_f32, cudaStream_t stream) {
+                         int gate_col, float softcap, const AbLayout* layout, int v_share, int out_f32, int chunk,
+                         cudaStream_t stream) {
     constexpr int KROW = ab_chunks(DK / 8) * 16, VROW = ab_chunks(DV / 8) * 16;
     const size_t smem = (size_t)AB_BM * KROW + 2 * ((size_t)AB_BN * KROW + (size_t)AB_BN * VROW);
     static bool configured[VX_MAX_DEVICES];
@@ -644,7 +653,7 @@ static int launch_biased(const bf16* q, int q_row_stride, const bf16* k_pool, co
     dim3 grid((max_new + toks_per_tile - 1) / toks_per_tile, share_log2 ? Hk : H, segments);
     VX_LAUNCH_K(VX_K_ATTENTION, (biased_attention_kernel<DK, DV>), grid, AB_WARPS * 32, smem, stream, q, q_row_stride, k_pool,
                 v_pool, block_table, max_blocks, seg, out, out_row_stride, scale * AB_LOG2E, bias_exp, window, keep_first, H,
-                Hk, S, share_log2, sinks, gate_col, softcap * AB_LOG2E, softcap > 0.f ? scale / softcap : 0.f, lay);
+                Hk, S, share_log2, sinks, gate_col, softcap * AB_LOG2E, softcap > 0.f ? scale / softcap : 0.f, lay, chunk);
     VX_LAUNCH_CHECK();
     return VX_OK;
 }
@@ -659,9 +668,10 @@ static int biased_attention_any(const void* q, int q_row_stride, const void* k_p
                                        float scale, float bias_exp, int window, int keep_first, int segments, int max_new,
                                        int H, int Hk, int DK, int DV, int S, float* scratch, int runs, const float* sinks,
                                        int gate_col, float softcap, const int* seq_list, const AbLayout* layout,
-                                       int v_share, int out_f32, cudaStream_t stream) {
+                                       int v_share, int out_f32, int chunk, cudaStream_t stream) {
     if (segments <= 0 || max_new <= 0) return VX_OK;
     if (v_share <= 0) v_share = 1;
+    if (chunk < 0 || (chunk && keep_first)) return VX_ERR_SHAPE;
     if (softcap < 0.f || Hk % v_share || (layout && v_share > 1)) return VX_ERR_SHAPE;
     if (H <= 0 || Hk <= 0 || H % Hk || S <= 0 || S % 16 || window < 0 || keep_first < 0 || bias_exp < 0.f) return VX_ERR_SHAPE;
     if (cu_seqlens ? !kv_offsets : (!seq_of_token || !positions || max_new != 1)) return VX_ERR_SHAPE;
@@ -678,7 +688,7 @@ static int biased_attention_any(const void* q, int q_row_stride, const void* k_p
         return launch_biased_decode<K_, V_>((const bf16*)q, q_row_stride, (const bf16*)k_pool, (const bf16*)v_pool,       \
                                             block_table, max_blocks, seq_of_token, positions, (bf16*)out, out_row_stride, \
                                             scale, bias_exp, window, keep_first, segments, H, Hk, S, scratch, runs, sinks,  \
-                                            gate_col, softcap, v_share, out_f32, stream)
+                                            gate_col, softcap, v_share, out_f32, chunk, stream)
         AD_GO(64, 32); AD_GO(64, 64); AD_GO(64, 128); AD_GO(128, 32); AD_GO(128, 64); AD_GO(128, 128);
         AD_GO(32, 32); AD_GO(48, 48); AD_GO(80, 80); AD_GO(96, 96); AD_GO(112, 112);
 #undef AD_GO
@@ -689,7 +699,7 @@ static int biased_attention_any(const void* q, int q_row_stride, const void* k_p
     if (DK == K_ && DV == V_)                                                                                             \
         return launch_biased<K_, V_>((const bf16*)q, q_row_stride, (const bf16*)k_pool, (const bf16*)v_pool, block_table, \
                                      max_blocks, seg, (bf16*)out, out_row_stride, scale, bias_exp, window, keep_first,    \
-                                     segments, max_new, H, Hk, S, sinks, gate_col, softcap, layout, v_share, out_f32, stream)
+                                     segments, max_new, H, Hk, S, sinks, gate_col, softcap, layout, v_share, out_f32, chunk, stream)
     AB_GO(64, 32); AB_GO(64, 64); AB_GO(64, 128); AB_GO(128, 32); AB_GO(128, 64); AB_GO(128, 128);
     AB_GO(32, 32); AB_GO(48, 48); AB_GO(80, 80); AB_GO(96, 96); AB_GO(112, 112);
     AB_GO(192, 128); AB_GO(192, 64); AB_GO(96, 64); AB_GO(96, 32); AB_GO(256, 128);   // (portions only: no kernel for single tokens)
@@ -707,7 +717,20 @@ extern "C" int vx_biased_attention_shared(const void* q, int q_row_stride, const
                                           int gate_col, float softcap, int v_share, int out_f32, cudaStream_t stream) {
     return biased_attention_any(q, q_row_stride, k_pool, v_pool, block_table, max_blocks, cu_seqlens, kv_offsets, seq_of_token,
                                 positions, out, out_row_stride, scale, bias_exp, window, keep_first, segments, max_new, H, Hk,
-                                DK, DV, S, scratch, runs, sinks, gate_col, softcap, nullptr, nullptr, v_share, out_f32, stream);
+                                DK, DV, S, scratch, runs, sinks, gate_col, softcap, nullptr, nullptr, v_share, out_f32, 0, stream);
+}
+
+// `chunk` > 0: a query sees only keys of its own run of `chunk` positions, the runs counted from position 0 (without kept
+// first positions).
+extern "C" int vx_biased_attention_chunk(const void* q, int q_row_stride, const void* k_pool, const void* v_pool,
+                                         const int* block_table, int max_blocks, const int* cu_seqlens, const int* kv_offsets,
+                                         const int* seq_of_token, const int* positions, void* out, int out_row_stride,
+                                         float scale, float bias_exp, int window, int keep_first, int segments, int max_new,
+                                         int H, int Hk, int DK, int DV, int S, float* scratch, int runs, const float* sinks,
+                                         int gate_col, float softcap, int v_share, int out_f32, int chunk, cudaStream_t stream) {
+    return biased_attention_any(q, q_row_stride, k_pool, v_pool, block_table, max_blocks, cu_seqlens, kv_offsets, seq_of_token,
+                                positions, out, out_row_stride, scale, bias_exp, window, keep_first, segments, max_new, H, Hk,
+                                DK, DV, S, scratch, runs, sinks, gate_col, softcap, nullptr, nullptr, v_share, out_f32, chunk, stream);
 }
 
 extern "C" int vx_biased_attention_cap(const void* q, int q_row_stride, const void* k_pool, const void* v_pool,
@@ -735,7 +758,7 @@ extern "C" int vx_biased_attention_rows_window(const void* q, int q_row_stride, 
     if (k_row < DK || v_row < DV || window < 0) return VX_ERR_SHAPE;
     return biased_attention_any(q, q_row_stride, k, v, block_table, max_blocks, cu_seqlens, kv_offsets, nullptr, nullptr, out,
                                 out_row_stride, scale, 0.f, window, 0, segments, max_new, H, Hk, DK, DV, S, nullptr, 1, nullptr, -1,
-                                softcap, seq_list, &lay, 1, 0, stream);
+                                softcap, seq_list, &lay, 1, 0, 0, stream);
 }
 
 extern "C" int vx_biased_attention_rows(const void* q, int q_row_stride, const void* k, long long k_row, long long k_head,

@@ -6,7 +6,9 @@
 //
 // One block per (token, query head).  The token's absolute position p gives its
 // keys: j in [start, p], start = max(0, p + 1 - window) with a window, else 0; with
-// keep_first > 0 also j in [0, min(keep_first, start)), at their true positions.
+// keep_first > 0 also j in [0, min(keep_first, start)), at their true positions.  With
+// chunk > 0 start is no less than p - p mod chunk: a token sees its own run of `chunk`
+// positions only, the runs counted from the request's position 0.
 // Key j of the token's request lies in page block_table[seq, j / S] at offset
 // j % S; pools are [page, Hk, S, D] and [page, Hk, S, Dv]; query head h reads kv head
 // h / (H / Hk).  score = q.k * scale - slope_h * (p - j) with
@@ -37,7 +39,8 @@ __global__ void paged_attention_generic_kernel(
     const T* __restrict__ v_pool, const int* __restrict__ block_table, int max_blocks,
     const int* __restrict__ seq_of_token, const int* __restrict__ positions, T* __restrict__ out,
     int out_row_stride, float scale, int window, int H, int Hk, int D, int S, int Dv, int keep_first,
-    float bias_exp, const float* __restrict__ sinks, int gate_col, float softcap, int v_stride, int v_share, int out_f32) {
+    float bias_exp, const float* __restrict__ sinks, int gate_col, float softcap, int v_stride, int v_share, int out_f32,
+    int chunk) {
     pdl_wait();
     pdl_trigger();
     __shared__ float q_s[ATT_MAX_D];
@@ -49,7 +52,8 @@ __global__ void paged_attention_generic_kernel(
     const int hk = h / (H / Hk);
     const int seq = seq_of_token[t];
     const int kv_len = positions[t] + 1;
-    const int start = (window > 0 && kv_len > window) ? kv_len - window : 0;
+    int start = (window > 0 && kv_len > window) ? kv_len - window : 0;
+    if (chunk > 0) start = max(start, kv_len - 1 - (kv_len - 1) % chunk);
     const int nkept = min(keep_first, start);   // kept first positions that lie before the window
     const float slope = bias_exp > 0.f ? exp2f(-bias_exp * (float)(h + 1) / (float)H) : 0.f;
     const int* bt = block_table + (size_t)seq * max_blocks;
@@ -140,14 +144,15 @@ __global__ void paged_attention_generic_kernel(
 }
 
 // `v_share` > 1: that many consecutive key heads read one value head (the value pool has Hk / v_share heads);
-// `out_f32`: the output is written as float32 whatever the element type of the inputs.
-extern "C" int vx_paged_attention_generic_shared(const void* q, int q_row_stride, const void* k_pool,
+// `out_f32`: the output is written as float32 whatever the element type of the inputs; `chunk` > 0: see
+// the top (it does not go with kept first positions).
+extern "C" int vx_paged_attention_generic_chunk(const void* q, int q_row_stride, const void* k_pool,
                                                  const void* v_pool, const int* block_table, int max_blocks,
                                                  const int* seq_of_token, const int* positions, void* out,
                                                  int out_row_stride, float scale, int window, int tokens,
                                                  int H, int Hk, int D, int S, int dtype, int Dv, int keep_first,
                                                  float bias_exp, const float* sinks, int gate_col, float softcap,
-                                                 int v_stride, int v_share, int out_f32, cudaStream_t stream) {
+                                                 int v_stride, int v_share, int out_f32, int chunk, cudaStream_t stream) {
     if (tokens <= 0) return VX_OK;
     if (Dv <= 0) Dv = D;
     if (v_stride <= 0) v_stride = Dv;
@@ -156,18 +161,30 @@ extern "C" int vx_paged_attention_generic_shared(const void* q, int q_row_stride
     if (v_stride < Dv || softcap < 0.f) return VX_ERR_SHAPE;
     if (H <= 0 || Hk <= 0 || H % Hk || D <= 0 || D > ATT_MAX_D || Dv > ATT_MAX_D || S <= 0 || max_blocks <= 0)
         return VX_ERR_SHAPE;
-    if (window < 0 || keep_first < 0 || bias_exp < 0.f) return VX_ERR_SHAPE;
+    if (window < 0 || keep_first < 0 || bias_exp < 0.f || chunk < 0 || (chunk && keep_first)) return VX_ERR_SHAPE;
     dim3 grid(tokens, H);
     if (dtype == VX_F32)
         VX_LAUNCH_K(VX_K_ATTENTION, (paged_attention_generic_kernel<float>), grid, ATT_WARPS * 32, 0, stream, (const float*)q, q_row_stride, (const float*)k_pool, (const float*)v_pool, block_table,
-            max_blocks, seq_of_token, positions, (float*)out, out_row_stride, scale, window, H, Hk, D, S, Dv, keep_first, bias_exp, sinks, gate_col, softcap, v_stride, v_share, out_f32);
+            max_blocks, seq_of_token, positions, (float*)out, out_row_stride, scale, window, H, Hk, D, S, Dv, keep_first, bias_exp, sinks, gate_col, softcap, v_stride, v_share, out_f32, chunk);
     else if (dtype == VX_BF16)
         VX_LAUNCH_K(VX_K_ATTENTION, (paged_attention_generic_kernel<bf16>), grid, ATT_WARPS * 32, 0, stream, (const bf16*)q, q_row_stride, (const bf16*)k_pool, (const bf16*)v_pool, block_table,
-            max_blocks, seq_of_token, positions, (bf16*)out, out_row_stride, scale, window, H, Hk, D, S, Dv, keep_first, bias_exp, sinks, gate_col, softcap, v_stride, v_share, out_f32);
+            max_blocks, seq_of_token, positions, (bf16*)out, out_row_stride, scale, window, H, Hk, D, S, Dv, keep_first, bias_exp, sinks, gate_col, softcap, v_stride, v_share, out_f32, chunk);
     else
         return VX_ERR_DTYPE;
     VX_LAUNCH_CHECK();
     return VX_OK;
+}
+
+extern "C" int vx_paged_attention_generic_shared(const void* q, int q_row_stride, const void* k_pool,
+                                                 const void* v_pool, const int* block_table, int max_blocks,
+                                                 const int* seq_of_token, const int* positions, void* out,
+                                                 int out_row_stride, float scale, int window, int tokens,
+                                                 int H, int Hk, int D, int S, int dtype, int Dv, int keep_first,
+                                                 float bias_exp, const float* sinks, int gate_col, float softcap,
+                                                 int v_stride, int v_share, int out_f32, cudaStream_t stream) {
+    return vx_paged_attention_generic_chunk(q, q_row_stride, k_pool, v_pool, block_table, max_blocks, seq_of_token, positions,
+                                            out, out_row_stride, scale, window, tokens, H, Hk, D, S, dtype, Dv, keep_first,
+                                            bias_exp, sinks, gate_col, softcap, v_stride, v_share, out_f32, 0, stream);
 }
 
 extern "C" int vx_paged_attention_generic_cap(const void* q, int q_row_stride, const void* k_pool,

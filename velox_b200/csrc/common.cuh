@@ -187,6 +187,8 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
 #define VX_ACT_GELU_TANH 2
 #define VX_ACT_RELU 3
 #define VX_ACT_IDENTITY 4   // (a plain change of element type through the activation kernel)
+#define VX_ACT_RELU2 5      // the square of relu
+#define VX_ACT_LAST 5
 
 __device__ __forceinline__ float activation(float z, int act) {
     switch (act) {
@@ -197,6 +199,7 @@ __device__ __forceinline__ float activation(float z, int act) {
             return 0.5f * z * (1.f + tanhf(c * (z + 0.044715f * z * z * z)));
         }
         case VX_ACT_IDENTITY: return z;
+        case VX_ACT_RELU2: { const float r = fmaxf(z, 0.f); return r * r; }
         default: return fmaxf(z, 0.f);
     }
 }

@@ -329,7 +329,7 @@ static int launch_gated_act(const void* gate_up, void* out, bool vec, long long 
 extern "C" int vx_gated_act(const void* gate_up, void* out, int rows, int inner, int act, int block, int dtype,
                             int out_dtype, cudaStream_t stream) {
     if (rows <= 0) return VX_OK;
-    if (inner <= 0 || act < 0 || act > 3 || block < 0 || (block > 0 && inner % block)) return VX_ERR_SHAPE;
+    if (inner <= 0 || act < 0 || act > VX_ACT_LAST || block < 0 || (block > 0 && inner % block)) return VX_ERR_SHAPE;
     const long long total = (long long)rows * inner;
     const int threads = 256;
     const bool vec = inner % 8 == 0 && (block == 0 || block == 8) &&

@@ -16,8 +16,13 @@
 // partial tiles are added in shared memory in warp order, so the result is the
 // same on every run and a row's result does not depend on the rows beside it.
 //
-// Epilogues: plain (bf16 or float32 out, optional bias), or gated: row r < 8 of a
-// tile is a gate row, row r + 8 its up row, out = act(gate) * up (float32 math).
+// Epilogues: plain (bf16 or float32 out, optional bias, optional activation of the
+// float32 sum), or gated: row r < 8 of a tile is a gate row, row r + 8 its up row,
+// out = act(gate) * up (float32 math).
+//
+// Several inputs (SEG): rows [i seg_rows, (i + 1) seg_rows) of W, and for the last
+// input all rows that are left, are multiplied with input i, x + i seg_stride: the
+// projections of a sublayer that gives each of them an input of its own, in one launch.
 //
 // Sizes: M <= 8; K a multiple of 32; N any (a multiple of 16 with the gated
 // epilogue); 16-byte aligned rows.
@@ -40,17 +45,25 @@ __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], unsigned a0, unsig
                  : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-template <bool GATED, typename TOut, int SK_WARPS, int SK_UNROLL, int MIN_BLOCKS>
+template <bool GATED, bool SEG, typename TOut, int SK_WARPS, int SK_UNROLL, int MIN_BLOCKS>
 __global__ void __launch_bounds__(SK_WARPS * 32, MIN_BLOCKS)
 gemm_skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ W, const float* __restrict__ bias,
-                   TOut* __restrict__ out, int M, int N, int K, int ldx, int ldw, int ldo, int act, int R) {
+                   TOut* __restrict__ out, int M, int N, int K, int ldx, int ldw, int ldo, int act, int R, int seg_rows,
+                   long long seg_stride, int segments) {
     __shared__ float red[SK_WARPS][16][9];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, t = lane & 3;
     // A block owns R <= 16 rows of W (gated: R <= 8 output features, each a gate row
     // and the up row 8 below it in its 16-row tile); rows of the tile beyond R are
     // not loaded.  R is chosen so that the blocks fill whole waves of the GPU.
-    const int row0 = blockIdx.x * R;
+    int row0 = blockIdx.x * R;
+    if (SEG) {
+        const int per = (seg_rows + R - 1) / R;                         // blocks of an input
+        const int seg = min((int)blockIdx.x / per, segments - 1);
+        row0 = seg * seg_rows + ((int)blockIdx.x - seg * per) * R;
+        if (seg < segments - 1) N = min(N, (seg + 1) * seg_rows);      // (a block's rows end with its input's)
+        x += seg * seg_stride;
+    }
     int ra, rb;
     bool va, vb;
     if (!GATED) {
@@ -129,6 +142,7 @@ gemm_skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ W, const
 #pragma unroll
                 for (int w = 0; w < SK_WARPS; ++w) v += red[w][r][m];
                 if (bias) v += bias[nrow];
+                if (act >= 0) v = activation(v, act);
                 out[(size_t)m * ldo + nrow] = from_f32<TOut>(v);
             }
         }
@@ -172,9 +186,10 @@ static int pick_variant(int N, int K) {
     return 7;
 }
 
-template <bool GATED, typename TOut>
+template <bool GATED, bool SEG, typename TOut>
 static int launch_skinny(const bf16* x, const bf16* W, const float* bias, TOut* out, int M, int N, int K, int ldx,
-                         int ldw, int ldo, int act, int variant, cudaStream_t stream) {
+                         int ldw, int ldo, int act, int variant, cudaStream_t stream, int seg_rows = 0,
+                         long long seg_stride = 0, int segments = 1) {
     const bool balance = variant < 100;  // variant + 100: whole tiles per block, for comparison
     if (variant >= 100) variant -= 100;
     if (variant == 0) variant = pick_variant(N, K);
@@ -190,10 +205,14 @@ static int launch_skinny(const bf16* x, const bf16* W, const float* bias, TOut* 
         R = (int)((units + waves * slots - 1) / (waves * slots));
         R = R < 1 ? 1 : (R > tile ? tile : R);
     }
-    const int blocks = (units + R - 1) / R;
+    int blocks = (units + R - 1) / R;
+    if (SEG) {
+        const int before = (segments - 1) * ((seg_rows + R - 1) / R);
+        blocks = before + (N - (segments - 1) * seg_rows + R - 1) / R;
+    }
 #define SK_GO(WARPS, UNROLL, MINB)                                                                                  \
-    VX_LAUNCH_K(VX_K_GEMM, (gemm_skinny_kernel<GATED, TOut, WARPS, UNROLL, MINB>), blocks, WARPS * 32, 0, stream, x, W, \
-                bias, out, M, N, K, ldx, ldw, ldo, act, R)
+    VX_LAUNCH_K(VX_K_GEMM, (gemm_skinny_kernel<GATED, SEG, TOut, WARPS, UNROLL, MINB>), blocks, WARPS * 32, 0, stream, x, W, \
+                bias, out, M, N, K, ldx, ldw, ldo, act, R, seg_rows, seg_stride, segments)
     switch (variant) {
         case 1: SK_GO(8, 4, 4); break;
         case 2: SK_GO(16, 4, 2); break;
@@ -209,23 +228,47 @@ static int launch_skinny(const bf16* x, const bf16* W, const float* bias, TOut* 
     return VX_OK;
 }
 
-// gated: 0 plain; 1: W rows come in tiles of 16 = 8 gate rows then their 8 up
+// gated: 0 plain (no activation, or with `act` >= 0 through vx_gemm_skinny_act that one); 1: W rows come in tiles of 16 = 8 gate rows then their 8 up
 // rows, and out is [M, N/2] = act(gate) * up.  out_dtype: VX_BF16 or VX_F32.
 // variant: 0 lets the sizes choose (pick_variant); 1..5 name one, for tuning.
-extern "C" int vx_gemm_skinny(const void* x, const void* W, const float* bias, void* out, int M, int N, int K,
-                              int ldx, int ldw, int ldo, int gated, int act, int out_dtype, int variant,
-                              cudaStream_t stream) {
+extern "C" int vx_gemm_skinny_act(const void* x, const void* W, const float* bias, void* out, int M, int N, int K,
+                                  int ldx, int ldw, int ldo, int gated, int act, int out_dtype, int variant,
+                                  cudaStream_t stream) {
     if (M <= 0 || N <= 0) return VX_OK;
     if (M > 8 || K <= 0 || (K & 31)) return VX_ERR_SHAPE;
     if (ldx < K || ldw < K || (ldx & 7) || (ldw & 7)) return VX_ERR_ALIGN;
     if ((((uintptr_t)x) | ((uintptr_t)W)) & 15) return VX_ERR_ALIGN;
-    if (gated && ((N & 15) || bias || act < 0 || act > 3)) return VX_ERR_SHAPE;
+    if (act > VX_ACT_LAST || (gated && ((N & 15) || bias || act < 0))) return VX_ERR_SHAPE;
     if (ldo < (gated ? N / 2 : N)) return VX_ERR_SHAPE;
     const bf16* xp = (const bf16*)x;
     const bf16* wp = (const bf16*)W;
-#define SK_CALL(G, T) launch_skinny<G, T>(xp, wp, bias, (T*)out, M, N, K, ldx, ldw, ldo, act, variant, stream)
+#define SK_CALL(G, T) launch_skinny<G, false, T>(xp, wp, bias, (T*)out, M, N, K, ldx, ldw, ldo, act, variant, stream)
     if (out_dtype == VX_BF16) return gated ? SK_CALL(true, bf16) : SK_CALL(false, bf16);
     if (out_dtype == VX_F32) return gated ? SK_CALL(true, float) : SK_CALL(false, float);
 #undef SK_CALL
+    return VX_ERR_DTYPE;
+}
+
+extern "C" int vx_gemm_skinny(const void* x, const void* W, const float* bias, void* out, int M, int N, int K,
+                              int ldx, int ldw, int ldo, int gated, int act, int out_dtype, int variant,
+                              cudaStream_t stream) {
+    return vx_gemm_skinny_act(x, W, bias, out, M, N, K, ldx, ldw, ldo, gated, gated ? act : -1, out_dtype, variant, stream);
+}
+
+// out[m, n] = sum_k x_i[m, k] W[n, k] with x_i = x + i seg_stride the input of row n: i = n / seg_rows, at most
+// segments - 1.  seg_stride a multiple of 8.
+extern "C" int vx_gemm_skinny_inputs(const void* x, const void* W, void* out, int M, int N, int K, int ldx, int ldw, int ldo,
+                                     int seg_rows, long long seg_stride, int segments, int out_dtype, cudaStream_t stream) {
+    if (M <= 0 || N <= 0) return VX_OK;
+    if (M > 8 || K <= 0 || (K & 31) || seg_rows <= 0 || segments <= 0 || (long long)(segments - 1) * seg_rows >= N) return VX_ERR_SHAPE;
+    if (ldx < K || ldw < K || (ldx & 7) || (ldw & 7) || (seg_stride & 7)) return VX_ERR_ALIGN;
+    if ((((uintptr_t)x) | ((uintptr_t)W)) & 15) return VX_ERR_ALIGN;
+    if (ldo < N) return VX_ERR_SHAPE;
+    if (out_dtype == VX_BF16)
+        return launch_skinny<false, true, bf16>((const bf16*)x, (const bf16*)W, nullptr, (bf16*)out, M, N, K, ldx, ldw, ldo, -1, 0,
+                                                stream, seg_rows, seg_stride, segments);
+    if (out_dtype == VX_F32)
+        return launch_skinny<false, true, float>((const bf16*)x, (const bf16*)W, nullptr, (float*)out, M, N, K, ldx, ldw, ldo, -1, 0,
+                                                 stream, seg_rows, seg_stride, segments);
     return VX_ERR_DTYPE;
 }

@@ -22,7 +22,7 @@
 //            tcgen05.ld, 32 columns at a time, adds the bias, rounds to bfloat16 and
 //            stores; or, gated, takes act(gate) * up of column tiles laid out as 8
 //            gate columns followed by their 8 up columns, in float32, and stores
-//            half as many columns; then they arrive on the accumulator's "empty"
+//            half as many columns, or takes act(.) of every column; then they arrive on the accumulator's "empty"
 //            mbarrier.
 // Rows past M and columns past N are zero-filled by TMA on the way in and masked on
 // the way out; K may end inside a k block (zero-filled too).
@@ -38,11 +38,16 @@
 // weights are W[group * N + column ..], W being all groups' matrices one after the other; see `csrc/moe.cu`.
 #include "tcgen05_gemm.cuh"
 
-template <int BN, int STAGES, bool GATED>
+#define TC_PLAIN 0
+#define TC_GATED 1   // act(gate) * up of paired columns
+#define TC_ACT 2     // act(.) of each column
+
+template <int BN, int STAGES, int EPI>
 __global__ void __launch_bounds__(TC_THREADS)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                     const float* __restrict__ bias, bf16* __restrict__ C, int M, int N, int K, int ldc, int act,
-                    int* __restrict__ error, const int* __restrict__ row_tiles, const int* __restrict__ n_row_tiles) {
+                    int* __restrict__ error, const int* __restrict__ row_tiles, const int* __restrict__ n_row_tiles,
+                    const float* __restrict__ row_scale, const int* __restrict__ src_of_row) {
     extern __shared__ unsigned char tc_smem_raw[];
     __shared__ __align__(8) unsigned long long full_bar[STAGES], empty_bar[STAGES], acc_full[2], acc_empty[2];
     __shared__ unsigned tmem_base_s;
@@ -157,6 +162,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
             const int m0 = row_tiles ? row_tiles[3 * rt + 1] : rt * TC_BM, n0 = (tile / mtiles) * BN;
             // (a grouped tile stores only its own rows: those after them belong to the next group)
             const int row = (row_tiles && quarter * 32 + lane >= row_tiles[3 * rt + 2]) ? M : m0 + quarter * 32 + lane;
+            const float rs = EPI != TC_PLAIN && row_scale && row < M ? row_scale[src_of_row[row]] : 1.f;
             bool ok = tc_mbar_wait(tc_smem_u32(&acc_full[buf]), (unsigned)((ti >> 1) & 1));
             if (!ok && lane == 0) { failed = 1; atomicExch(error, TC_ERR_EPILOGUE); }
             ok = __all_sync(0xffffffffu, ok);
@@ -169,7 +175,11 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                 unsigned r[32];
                 tc_ld32(tmem_acc + (unsigned)c0, r);
                 if (row >= M) continue;
-                if (!GATED) {
+                if (EPI != TC_PLAIN && row_scale) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * rs);
+                }
+                if (EPI != TC_GATED) {
                     bf16* dst = C + (size_t)row * ldc + n0 + c0;
 #pragma unroll
                     for (int j = 0; j < 32; j += 8) {
@@ -179,6 +189,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                         for (int i = 0; i < 8; ++i) {
                             v[i] = __uint_as_float(r[j + i]);
                             if (bias) v[i] += bias[n0 + c0 + j + i];
+                            if (EPI == TC_ACT) v[i] = activation(v[i], act);
                         }
                         uint4 pk;
                         __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&pk);
@@ -220,26 +231,27 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 }
 
 // ---- host side ----
-template <int BN, int STAGES, bool GATED>
+template <int BN, int STAGES, int EPI>
 static int tc_launch(const CUtensorMap& ma, const CUtensorMap& mw, const float* bias, bf16* C, int M, int N, int K,
                      int ldc, int act, int* error, cudaStream_t stream, const int* row_tiles = nullptr,
-                     const int* n_row_tiles = nullptr, int max_row_tiles = 0) {
+                     const int* n_row_tiles = nullptr, int max_row_tiles = 0, const float* row_scale = nullptr,
+                     const int* src_of_row = nullptr) {
     const size_t smem = (size_t)STAGES * (TC_BM * TC_BK * 2 + BN * TC_BK * 2) + 1024;
     static bool configured[VX_MAX_DEVICES];
-    if (int rc = vx_configure_smem(gemm_tcgen05_kernel<BN, STAGES, GATED>, smem, configured)) return rc;
+    if (int rc = vx_configure_smem(gemm_tcgen05_kernel<BN, STAGES, EPI>, smem, configured)) return rc;
     // persistent: one block per SM (its shared memory fills one), fewer if there are fewer tiles
     static int sm_counts[VX_MAX_DEVICES];
     const int sms = vx_sm_count(sm_counts);
     const int tiles = (row_tiles ? max_row_tiles : (M + TC_BM - 1) / TC_BM) * ((N + BN - 1) / BN);
     dim3 grid(tiles < sms ? tiles : sms);
-    VX_LAUNCH_K(VX_K_GEMM, (gemm_tcgen05_kernel<BN, STAGES, GATED>), grid, TC_THREADS, smem, stream, ma, mw, bias, C, M,
-                N, K, ldc, act, error, row_tiles, n_row_tiles);
+    VX_LAUNCH_K(VX_K_GEMM, (gemm_tcgen05_kernel<BN, STAGES, EPI>), grid, TC_THREADS, smem, stream, ma, mw, bias, C, M,
+                N, K, ldc, act, error, row_tiles, n_row_tiles, row_scale, src_of_row);
     VX_LAUNCH_CHECK();
     return VX_OK;
 }
 
 // gated: 0 plain, C is [M, N]; 1: W's rows come in tiles of 8 gate rows followed by
-// their 8 up rows and C is [M, N/2] = act(gate) * up.  `error` is a device int that
+// their 8 up rows and C is [M, N/2] = act(gate) * up; 2: C is [M, N] = act(.).  `error` is a device int that
 // a block sets (TC_ERR_*) if one of its bounded waits runs out; the caller zeroes it
 // and reads it when it wants to know.  `wide` picks 128 x 256 tiles (else 128 x 128).
 extern "C" int vx_gemm_tcgen05(const void* A, const void* W, const float* bias, void* C, int M, int N, int K, int lda,
@@ -248,34 +260,44 @@ extern "C" int vx_gemm_tcgen05(const void* A, const void* W, const float* bias, 
     if (K <= 0 || (K & 7) || (N & 15) || !error) return VX_ERR_SHAPE;
     if ((lda & 7) || (ldw & 7) || (ldc & 7) || lda < K || ldw < K) return VX_ERR_ALIGN;
     if ((((uintptr_t)A) | ((uintptr_t)W) | ((uintptr_t)C)) & 15) return VX_ERR_ALIGN;
-    if (gated && (bias || act < 0 || act > 3)) return VX_ERR_SHAPE;
-    if (ldc < (gated ? N / 2 : N)) return VX_ERR_SHAPE;
+    if (gated < 0 || gated > TC_ACT || (gated && (act < 0 || act > VX_ACT_LAST)) || (gated == TC_GATED && bias)) return VX_ERR_SHAPE;
+    if (ldc < (gated == TC_GATED ? N / 2 : N)) return VX_ERR_SHAPE;
     CUtensorMap ma, mw;
     const int bn = wide ? 256 : 128;
     if (!tc_make_map(&ma, A, M, K, lda, TC_BM) || !tc_make_map(&mw, W, N, K, ldw, bn)) return VX_ERR_DRIVER;
     bf16* c = (bf16*)C;
-    if (wide)
-        return gated ? tc_launch<256, 4, true>(ma, mw, bias, c, M, N, K, ldc, act, error, stream)
-                     : tc_launch<256, 4, false>(ma, mw, bias, c, M, N, K, ldc, act, error, stream);
-    return gated ? tc_launch<128, 6, true>(ma, mw, bias, c, M, N, K, ldc, act, error, stream)
-                 : tc_launch<128, 6, false>(ma, mw, bias, c, M, N, K, ldc, act, error, stream);
+#define TC_GO(BN_, ST_, E_) tc_launch<BN_, ST_, E_>(ma, mw, bias, c, M, N, K, ldc, act, error, stream)
+    if (wide) return gated == TC_GATED ? TC_GO(256, 4, TC_GATED) : (gated == TC_ACT ? TC_GO(256, 4, TC_ACT) : TC_GO(256, 4, TC_PLAIN));
+    return gated == TC_GATED ? TC_GO(128, 6, TC_GATED) : (gated == TC_ACT ? TC_GO(128, 6, TC_ACT) : TC_GO(128, 6, TC_PLAIN));
+#undef TC_GO
 }
 
 // The grouped product of a routed feed-forward: A [rows, K] in group order, W [groups, N, K], row tiles of up to
 // 128 rows (group, first row, rows) whose number is on the device (at most max_row_tiles).  C [rows, N], or
-// [rows, N/2] = act(gate) * up when gated.
-extern "C" int vx_moe_gemm_tcgen05(const void* A, const void* W, void* C, int rows, int groups, int N, int K, int lda,
+// [rows, N/2] = act(gate) * up when gated (1), act(.) of each element with gated = 2.  With row_scale (then gated is not 0)
+// row p's sums are first multiplied by row_scale[src_of_row[p]].
+extern "C" int vx_moe_gemm_tcgen05_scaled(const void* A, const void* W, void* C, int rows, int groups, int N, int K, int lda,
                                    int ldc, int gated, int act, const int* row_tiles, const int* n_row_tiles,
-                                   int max_row_tiles, int* error, cudaStream_t stream) {
+                                   int max_row_tiles, int* error, const float* row_scale, const int* src_of_row,
+                                   cudaStream_t stream) {
+    if (row_scale && (!src_of_row || !gated)) return VX_ERR_SHAPE;
     if (rows <= 0 || N <= 0 || max_row_tiles <= 0) return VX_OK;
     if (K <= 0 || (K & 7) || (N & 15) || groups <= 0 || !error || !row_tiles || !n_row_tiles) return VX_ERR_SHAPE;
     if ((lda & 7) || (ldc & 7) || lda < K) return VX_ERR_ALIGN;
     if ((((uintptr_t)A) | ((uintptr_t)W) | ((uintptr_t)C)) & 15) return VX_ERR_ALIGN;
-    if (gated && (act < 0 || act > 3)) return VX_ERR_SHAPE;
-    if (ldc < (gated ? N / 2 : N) || (long long)groups * N > 0x7fffffffLL) return VX_ERR_SHAPE;
+    if (gated < 0 || gated > TC_ACT || (gated && (act < 0 || act > VX_ACT_LAST))) return VX_ERR_SHAPE;
+    if (ldc < (gated == TC_GATED ? N / 2 : N) || (long long)groups * N > 0x7fffffffLL) return VX_ERR_SHAPE;
     CUtensorMap ma, mw;
     if (!tc_make_map(&ma, A, rows, K, lda, TC_BM) || !tc_make_map(&mw, W, groups * N, K, K, 256)) return VX_ERR_DRIVER;
     bf16* c = (bf16*)C;
-    return gated ? tc_launch<256, 4, true>(ma, mw, nullptr, c, rows, N, K, ldc, act, error, stream, row_tiles, n_row_tiles, max_row_tiles)
-                 : tc_launch<256, 4, false>(ma, mw, nullptr, c, rows, N, K, ldc, act, error, stream, row_tiles, n_row_tiles, max_row_tiles);
+#define TC_GO(E_) tc_launch<256, 4, E_>(ma, mw, nullptr, c, rows, N, K, ldc, act, error, stream, row_tiles, n_row_tiles, max_row_tiles, row_scale, src_of_row)
+    return gated == TC_GATED ? TC_GO(TC_GATED) : (gated == TC_ACT ? TC_GO(TC_ACT) : TC_GO(TC_PLAIN));
+#undef TC_GO
+}
+
+extern "C" int vx_moe_gemm_tcgen05(const void* A, const void* W, void* C, int rows, int groups, int N, int K, int lda,
+                                   int ldc, int gated, int act, const int* row_tiles, const int* n_row_tiles,
+                                   int max_row_tiles, int* error, cudaStream_t stream) {
+    return vx_moe_gemm_tcgen05_scaled(A, W, C, rows, groups, N, K, lda, ldc, gated, act, row_tiles, n_row_tiles, max_row_tiles, error,
+                                      nullptr, nullptr, stream);
 }

@@ -279,7 +279,7 @@ extern "C" int vx_gemm_tcgen05_pair(const void* A, const void* W, const float* b
     if (K <= 0 || (K & 7) || (N & 15) || !error) return VX_ERR_SHAPE;
     if ((lda & 7) || (ldw & 7) || (ldc & 7) || lda < K || ldw < K) return VX_ERR_ALIGN;
     if ((((uintptr_t)A) | ((uintptr_t)W) | ((uintptr_t)C)) & 15) return VX_ERR_ALIGN;
-    if (gated && (bias || act < 0 || act > 3)) return VX_ERR_SHAPE;
+    if (gated && (bias || act < 0 || act > VX_ACT_LAST)) return VX_ERR_SHAPE;
     if (ldc < (gated ? N / 2 : N)) return VX_ERR_SHAPE;
     CUtensorMap ma, mw;
     if (!tc_make_map(&ma, A, M, K, lda, TC_BM) || !tc_make_map(&mw, W, N, K, ldw, TP_HALF)) return VX_ERR_DRIVER;

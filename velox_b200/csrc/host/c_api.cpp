@@ -49,6 +49,13 @@ int vxh_cache_set_keep_first(void* c, int g, int n) {
     b->group(g).keep_first = n;
     return OK;
 }
+// a group whose queries see their own run of n positions only gives back the pages before the run
+int vxh_cache_set_chunk(void* c, int g, int n) {
+    CacheBook* b = (CacheBook*)c;
+    if (g < 0 || g >= b->num_groups() || n < 0) return fail(ERR_VALUE, "chunk: no such group, or a negative size");
+    b->group(g).chunk = n;
+    return OK;
+}
 void* vxh_cache_pool(void* c, int g) { return &((CacheBook*)c)->group(g).pool; }
 void* vxh_cache_slots(void* c) { return &((CacheBook*)c)->slots(); }
 int vxh_cache_add(void* c, int64_t rid) { return ((CacheBook*)c)->add(rid); }

@@ -7,7 +7,8 @@
 // reference does (src/paged/scheduler.rs:255).  They are given back when the
 // request ends, and in a group with a window as soon as every position of a page
 // lies before the window of the next query (pages that hold one of the group's kept
-// first positions stay); the freed page is the next one handed out.  Beside the tables the book keeps, per group, a dense mirror
+// first positions stay), in a group with chunks as soon as it lies before the next query's
+// chunk; the freed page is the next one handed out.  Beside the tables the book keeps, per group, a dense mirror
 // [slot, block] (-1 where no page is held), from which the step builders copy
 // whole rows.
 //
@@ -32,6 +33,7 @@ struct RequestCache {
 
 struct CacheGroup {
     int window;
+    int chunk = 0;       // a query sees its own run of so many positions only (0: no such limit)
     int keep_first = 0;  // with a window: the first positions that every later query still reads
     PagePool pool;
     std::vector<int32_t> mirror;  // [max_requests, max_blocks]
@@ -126,9 +128,11 @@ public:
             if ((int64_t)table.size() * page_size_ < rc->length)
                 return fail(ERR_ACCOUNTING, "request " + std::to_string(rid) + " wrote " + std::to_string(rc->length) +
                                                 " positions into " + std::to_string(table.size()) + " pages");
-            if (groups_[g].window > 0) {
+            if (groups_[g].window > 0 || groups_[g].chunk > 0) {
                 // the first page that the query at position `length` can still see
-                const int64_t first_key = std::max<int64_t>(0, rc->length + 1 - groups_[g].window);
+                int64_t first_key = groups_[g].window > 0 ? std::max<int64_t>(0, rc->length + 1 - groups_[g].window) : 0;
+                if (groups_[g].chunk > 0)
+                    first_key = std::max<int64_t>(first_key, rc->length - rc->length % groups_[g].chunk);
                 const int64_t keep_from = std::min<int64_t>(first_key / page_size_, (int64_t)table.size());
                 const int64_t kept_pages = ((int64_t)groups_[g].keep_first + page_size_ - 1) / page_size_;
                 for (int64_t i = kept_pages; i < keep_from; ++i) {

@@ -5,6 +5,7 @@
 //             Or (mode 1) scores s = softmax(logits) over ALL outputs, choice by s + correction among the
 //             outputs of the best `keep_groups` of `groups` equal groups of neighbours (a group's score:
 //             its largest choice score), weights s * route_scale, not renormalised.  The router's last
+//             Or (mode 2) scores s = sigmoid(logits), one by one, the rest as in mode 1.  The router's last
 //             outputs may be identity experts (no matrices: the token itself), and one more row of the
 //             router's matrix may hold the gate of a shared expert, sigmoid(w . h) per token
 //   plan      one block: where each expert's rows start in expert order, the list of row tiles
@@ -12,8 +13,10 @@
 //             assignment (token, k) its row in expert order
 //   grouped product   C[p, :] = A[src(p), :] W_e^T for the rows p of each tile, W = [experts, N, K];
 //             optionally with act(gate) * up on the accumulators (W's rows in tiles of 8 gate rows
-//             followed by their 8 up rows)
-//   combine   out[t] = sum_k weight[t, k] * y[row of (t, k)] (+ gate[t] * shared[t]) in float32, k ascending;
+//             followed by their 8 up rows) or act(.) of each; with `row_scale` a row's accumulators are first
+//             multiplied by its assignment's number (as if the row of A had been: the product is linear)
+//   combine   out[t] = sum_k weight[t, k] * y[row of (t, k)] (+ gate[t] * shared[t]) in float32, k ascending
+//             (no `weight`: every weight is 1, the grouped products have applied them);
 //             an assignment to an identity expert adds weight * h[t] instead
 //
 // The grid of a grouped product is sized for the worst case (assignments / tile rows + experts
@@ -60,14 +63,23 @@ __device__ __forceinline__ void route_select(float* z, float* sc, float* gs, uns
                                              const float* __restrict__ correction, int groups, int keep_groups,
                                              float route_scale, float* __restrict__ shared_gate) {
     if (shared_gate && lane == 0) shared_gate[t] = 1.f / (1.f + expf(-z[E]));
-    if (mode == 1) {
-        float mx = -INFINITY;
-        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
-        mx = warp_max(mx);
-        float sum = 0.f;
-        for (int e = lane; e < E; e += 32) { const float p = expf(z[e] - mx); sc[e] = p; sum += p; }
-        sum = warp_sum(sum);
+    if (mode >= 1) {
+        float sum = 1.f;
+        if (mode == 1) {
+            float mx = -INFINITY;
+            for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+            mx = warp_max(mx);
+            sum = 0.f;
+            for (int e = lane; e < E; e += 32) { const float p = expf(z[e] - mx); sc[e] = p; sum += p; }
+            sum = warp_sum(sum);
+        } else {
+            for (int e = lane; e < E; e += 32) sc[e] = 1.f / (1.f + expf(-z[e]));
+        }
+        // (the sigmoid rises with the logit: without a correction the choice is by the logits themselves, which keep apart
+        // what the sigmoid rounds to 1)
+        const bool by_logit = mode == 2 && !correction;
         for (int e = lane; e < E; e += 32) {
+            if (by_logit) continue;
             const float v = sc[e] / sum;
             sc[e] = v;
             z[e] = v + (correction ? correction[e] : 0.f);   // the choice score; the weight stays v
@@ -117,7 +129,7 @@ __device__ __forceinline__ void route_select(float* z, float* sc, float* gs, uns
             if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
         }
         if (lane == 0) {
-            zc[i] = mode == 1 ? sc[arg] : best;
+            zc[i] = mode >= 1 ? sc[arg] : best;
             z[arg] = -INFINITY;
             pick[i] = arg;
         }
@@ -128,7 +140,7 @@ __device__ __forceinline__ void route_select(float* z, float* sc, float* gs, uns
         const int e = pick[lane];
         chosen[(size_t)t * top + lane] = e;
         float w;
-        if (mode == 1) {
+        if (mode >= 1) {
             w = zc[lane] * route_scale;
         } else {
             const float m = zc[0];
@@ -363,7 +375,8 @@ moe_plan_kernel(const int* __restrict__ chosen, const int* __restrict__ pos, int
 }
 
 // E: the router's outputs (experts, then `identity` identity experts).  mode 0: top-k of the logits, softmax over
-// the chosen; mode 1: softmax over all, choice by score + correction within the best groups, weights score * route_scale.
+// the chosen; mode 1: softmax over all, choice by score + correction within the best groups, weights score * route_scale;
+// mode 2: the same with scores sigmoid(logit).
 // With `shared_gate` the router's matrix has one more row and shared_gate[t] = sigmoid(that row . h[t]).
 extern "C" int vx_moe_route(const void* h, int ldh, const float* w_router, const float* bias, int tokens, int K, int E,
                             int top, int tile_rows, int* chosen, float* weight, int* counts, int* pos, int* offsets,
@@ -372,7 +385,7 @@ extern "C" int vx_moe_route(const void* h, int ldh, const float* w_router, const
                             float* shared_gate, cudaStream_t stream) {
     if (tokens <= 0) return VX_OK;
     if (K <= 0 || E <= 0 || top <= 0 || top > E || tile_rows <= 0) return VX_ERR_SHAPE;
-    if (mode < 0 || mode > 1 || identity < 0 || identity >= E) return VX_ERR_SHAPE;
+    if (mode < 0 || mode > 2 || identity < 0 || identity >= E) return VX_ERR_SHAPE;
     if (groups < 1) groups = 1;
     if (E % groups || keep_groups < 1 || keep_groups > groups || top > keep_groups * (E / groups)) return VX_ERR_SHAPE;
     if (E > MOE_MAX_EXPERTS || top > MOE_MAX_TOP) return VX_ERR_LIMIT;
@@ -416,6 +429,15 @@ extern "C" int vx_moe_route(const void* h, int ldh, const float* w_router, const
 }
 
 // ---- grouped product on the CUDA cores: any sizes, float32 sums over k ascending ----
+// epilogues: the sums, act(gate) * up of paired columns, act(.) of each
+#define MOE_PLAIN 0
+#define MOE_GATED 1
+#define MOE_ACT 2
+// the number that the row's assignment multiplies it with (1 without `row_scale`)
+__device__ __forceinline__ float moe_row_scale(const float* __restrict__ row_scale, const int* __restrict__ src_of_row, int p, bool live) {
+    return row_scale && live ? row_scale[src_of_row[p]] : 1.f;
+}
+
 #define MG_BM 64
 #define MG_BN 64
 #define MG_BK 16
@@ -424,7 +446,7 @@ template <typename TA, typename TC>
 __global__ void __launch_bounds__(256)
 moe_gemm_simt_kernel(const TA* __restrict__ A, int lda, const int* __restrict__ src_of_row, int src_div,
                      const TA* __restrict__ W, const int* __restrict__ tiles, const int* __restrict__ n_tiles,
-                     TC* __restrict__ C, int ldc, int N, int K, int gated, int act) {
+                     TC* __restrict__ C, int ldc, int N, int K, int gated, int act, const float* __restrict__ row_scale) {
     pdl_wait();
     pdl_trigger();
     if ((int)blockIdx.y >= n_tiles[0]) return;
@@ -474,17 +496,18 @@ moe_gemm_simt_kernel(const TA* __restrict__ A, int lda, const int* __restrict__ 
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         const int r = ty + 16 * i;
+        const float rs = moe_row_scale(row_scale, src_of_row, row0 + r, r < rows);
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx + 16 * j;
-            float v = acc[i][j];
-            if (gated) {
+            float v = acc[i][j] * rs;
+            if (gated == MOE_GATED) {
                 // columns come as 8 gates, then their 8 ups: the up of this thread's gate is 8 lanes on
                 const float up = __shfl_xor_sync(0xffffffffu, v, 8);
                 if (tx < 8 && r < rows && n < N)
                     C[(size_t)(row0 + r) * ldc + (n >> 4) * 8 + tx] = from_f32<TC>(activation(v, act) * up);
             } else if (r < rows && n < N) {
-                C[(size_t)(row0 + r) * ldc + n] = from_f32<TC>(v);
+                C[(size_t)(row0 + r) * ldc + n] = from_f32<TC>(gated == MOE_ACT ? activation(v, act) : v);
             }
         }
     }
@@ -506,7 +529,7 @@ template <typename TC>
 __global__ void __launch_bounds__(128)
 moe_gemm_mma_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__ src_of_row, int src_div,
                     const bf16* __restrict__ W, const int* __restrict__ tiles, const int* __restrict__ n_tiles,
-                    TC* __restrict__ C, int ldc, int N, int K, int gated, int act) {
+                    TC* __restrict__ C, int ldc, int N, int K, int gated, int act, const float* __restrict__ row_scale) {
     extern __shared__ __align__(16) unsigned char mt_smem[];
     typedef bf16 (*Tile)[MT_BM][MT_LD];
     Tile As = reinterpret_cast<Tile>(mt_smem);
@@ -590,7 +613,8 @@ moe_gemm_mma_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__
             const int r = wm + 16 * i + (lane >> 2) + 8 * half;
             if (r >= rows) continue;
             TC* crow = C + (size_t)(row0 + r) * ldc;
-            if (gated) {
+            const float rs = moe_row_scale(row_scale, src_of_row, row0 + r, true);
+            if (gated == MOE_GATED) {
 #pragma unroll
                 for (int j = 0; j < 4; j += 2) {   // n-tile j: 8 gates, n-tile j + 1: their ups
                     const int n = n0 + wn + 8 * j + 2 * (lane & 3);
@@ -598,7 +622,7 @@ moe_gemm_mma_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__
                     for (int c = 0; c < 2; ++c)
                         if (n + c < N)
                             crow[((n + c) >> 4) * 8 + ((n + c) & 7)] =
-                                from_f32<TC>(activation(acc[i][j][2 * half + c], act) * acc[i][j + 1][2 * half + c]);
+                                from_f32<TC>(activation(acc[i][j][2 * half + c] * rs, act) * (acc[i][j + 1][2 * half + c] * rs));
                 }
             } else {
 #pragma unroll
@@ -606,7 +630,10 @@ moe_gemm_mma_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__
                     const int n = n0 + wn + 8 * j + 2 * (lane & 3);
 #pragma unroll
                     for (int c = 0; c < 2; ++c)
-                        if (n + c < N) crow[n + c] = from_f32<TC>(acc[i][j][2 * half + c]);
+                        if (n + c < N) {
+                            const float v = acc[i][j][2 * half + c] * rs;
+                            crow[n + c] = from_f32<TC>(gated == MOE_ACT ? activation(v, act) : v);
+                        }
                 }
             }
         }
@@ -624,7 +651,7 @@ template <typename TC>
 __global__ void __launch_bounds__(128)
 moe_gemm_mma16_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__ src_of_row, int src_div,
                       const bf16* __restrict__ W, const int* __restrict__ tiles, const int* __restrict__ n_tiles,
-                      TC* __restrict__ C, int ldc, int N, int K, int gated, int act) {
+                      TC* __restrict__ C, int ldc, int N, int K, int gated, int act, const float* __restrict__ row_scale) {
     extern __shared__ __align__(16) unsigned char ms_smem[];
     typedef bf16 (*TileA)[MS_BM][MT_LD];
     typedef bf16 (*TileW)[MT_BN][MT_LD];
@@ -693,15 +720,17 @@ moe_gemm_mma16_kernel(const bf16* __restrict__ A, int lda, const int* __restrict
         if (r >= rows) continue;
         TC* crow = C + (size_t)(row0 + r) * ldc;
         const int n = n0 + wn + 2 * (lane & 3);
+        const float rs = moe_row_scale(row_scale, src_of_row, row0 + r, true);
 #pragma unroll
         for (int c = 0; c < 2; ++c) {
-            if (gated) {   // the warp's 16 columns: 8 gates, then their 8 ups
+            const float v0 = acc[0][2 * half + c] * rs, v1 = acc[1][2 * half + c] * rs;
+            if (gated == MOE_GATED) {   // the warp's 16 columns: 8 gates, then their 8 ups
                 if (n + c < N)
                     crow[((n + c) >> 4) * 8 + ((n + c) & 7)] =
-                        from_f32<TC>(activation(acc[0][2 * half + c], act) * acc[1][2 * half + c]);
+                        from_f32<TC>(activation(v0, act) * v1);
             } else {
-                if (n + c < N) crow[n + c] = from_f32<TC>(acc[0][2 * half + c]);
-                if (n + 8 + c < N) crow[n + 8 + c] = from_f32<TC>(acc[1][2 * half + c]);
+                if (n + c < N) crow[n + c] = from_f32<TC>(gated == MOE_ACT ? activation(v0, act) : v0);
+                if (n + 8 + c < N) crow[n + 8 + c] = from_f32<TC>(gated == MOE_ACT ? activation(v1, act) : v1);
             }
         }
     }
@@ -709,12 +738,15 @@ moe_gemm_mma16_kernel(const bf16* __restrict__ A, int lda, const int* __restrict
 
 // in_dtype: A and W; out_dtype: C.  `tensor_cores`: the bfloat16 kernel (K a multiple of 8,
 // 16-byte aligned rows); else the multiply-add kernel.  max_tiles bounds the tiles of any step.
-// tile_rows: 64, or 16 (tensor cores only) for steps of few tokens.
-extern "C" int vx_moe_gemm(const void* A, int lda, const int* src_of_row, int src_div, const void* W, const int* tiles,
+// tile_rows: 64, or 16 (tensor cores only) for steps of few tokens.  gated: 0 plain, 1 act(gate) * up, 2 act(.).
+// row_scale float32 [assignments] (with src_of_row): row p of C is formed from row_scale[src_of_row[p]] times its sums.
+extern "C" int vx_moe_gemm_scaled(const void* A, int lda, const int* src_of_row, int src_div, const void* W, const int* tiles,
                            const int* n_tiles, int max_tiles, void* C, int ldc, int N, int K, int gated, int act,
-                           int in_dtype, int out_dtype, int tensor_cores, int tile_rows, cudaStream_t stream) {
+                           int in_dtype, int out_dtype, int tensor_cores, int tile_rows, const float* row_scale,
+                           cudaStream_t stream) {
+    if (gated < 0 || gated > MOE_ACT || (gated && (act < 0 || act > VX_ACT_LAST)) || (row_scale && !src_of_row)) return VX_ERR_SHAPE;
     if (max_tiles <= 0 || N <= 0) return VX_OK;
-    if (K <= 0 || lda < K || src_div <= 0 || (gated && N % 16)) return VX_ERR_SHAPE;
+    if (K <= 0 || lda < K || src_div <= 0 || (gated == MOE_GATED && N % 16)) return VX_ERR_SHAPE;
     if (max_tiles > 65535) return VX_ERR_LIMIT;
     if (tile_rows != MT_BM && !(tile_rows == MS_BM && tensor_cores)) return VX_ERR_SHAPE;
     dim3 grid((N + MG_BN - 1) / MG_BN, max_tiles);
@@ -726,10 +758,10 @@ extern "C" int vx_moe_gemm(const void* A, int lda, const int* src_of_row, int sr
                                           : vx_configure_smem(moe_gemm_mma16_kernel<float>, MS_SMEM, conf_f)) return rc;
         if (out_dtype == VX_BF16)
             VX_LAUNCH_K(VX_K_GEMM, (moe_gemm_mma16_kernel<bf16>), grid, 128, MS_SMEM, stream, (const bf16*)A, lda, src_of_row,
-                        src_div, (const bf16*)W, tiles, n_tiles, (bf16*)C, ldc, N, K, gated, act);
+                        src_div, (const bf16*)W, tiles, n_tiles, (bf16*)C, ldc, N, K, gated, act, row_scale);
         else if (out_dtype == VX_F32)
             VX_LAUNCH_K(VX_K_GEMM, (moe_gemm_mma16_kernel<float>), grid, 128, MS_SMEM, stream, (const bf16*)A, lda, src_of_row,
-                        src_div, (const bf16*)W, tiles, n_tiles, (float*)C, ldc, N, K, gated, act);
+                        src_div, (const bf16*)W, tiles, n_tiles, (float*)C, ldc, N, K, gated, act, row_scale);
         else
             return VX_ERR_DTYPE;
     } else if (tensor_cores) {
@@ -740,25 +772,32 @@ extern "C" int vx_moe_gemm(const void* A, int lda, const int* src_of_row, int sr
                                           : vx_configure_smem(moe_gemm_mma_kernel<float>, MT_SMEM, configured_f)) return rc;
         if (out_dtype == VX_BF16)
             VX_LAUNCH_K(VX_K_GEMM, (moe_gemm_mma_kernel<bf16>), grid, 128, MT_SMEM, stream, (const bf16*)A, lda, src_of_row, src_div,
-                        (const bf16*)W, tiles, n_tiles, (bf16*)C, ldc, N, K, gated, act);
+                        (const bf16*)W, tiles, n_tiles, (bf16*)C, ldc, N, K, gated, act, row_scale);
         else if (out_dtype == VX_F32)
             VX_LAUNCH_K(VX_K_GEMM, (moe_gemm_mma_kernel<float>), grid, 128, MT_SMEM, stream, (const bf16*)A, lda, src_of_row, src_div,
-                        (const bf16*)W, tiles, n_tiles, (float*)C, ldc, N, K, gated, act);
+                        (const bf16*)W, tiles, n_tiles, (float*)C, ldc, N, K, gated, act, row_scale);
         else
             return VX_ERR_DTYPE;
     } else if (in_dtype == VX_F32 && out_dtype == VX_F32)
         VX_LAUNCH_K(VX_K_GEMM, (moe_gemm_simt_kernel<float, float>), grid, 256, 0, stream, (const float*)A, lda, src_of_row,
-                    src_div, (const float*)W, tiles, n_tiles, (float*)C, ldc, N, K, gated, act);
+                    src_div, (const float*)W, tiles, n_tiles, (float*)C, ldc, N, K, gated, act, row_scale);
     else if (in_dtype == VX_BF16 && out_dtype == VX_BF16)
         VX_LAUNCH_K(VX_K_GEMM, (moe_gemm_simt_kernel<bf16, bf16>), grid, 256, 0, stream, (const bf16*)A, lda, src_of_row,
-                    src_div, (const bf16*)W, tiles, n_tiles, (bf16*)C, ldc, N, K, gated, act);
+                    src_div, (const bf16*)W, tiles, n_tiles, (bf16*)C, ldc, N, K, gated, act, row_scale);
     else if (in_dtype == VX_BF16 && out_dtype == VX_F32)
         VX_LAUNCH_K(VX_K_GEMM, (moe_gemm_simt_kernel<bf16, float>), grid, 256, 0, stream, (const bf16*)A, lda, src_of_row,
-                    src_div, (const bf16*)W, tiles, n_tiles, (float*)C, ldc, N, K, gated, act);
+                    src_div, (const bf16*)W, tiles, n_tiles, (float*)C, ldc, N, K, gated, act, row_scale);
     else
         return VX_ERR_DTYPE;
     VX_LAUNCH_CHECK();
     return VX_OK;
+}
+
+extern "C" int vx_moe_gemm(const void* A, int lda, const int* src_of_row, int src_div, const void* W, const int* tiles,
+                           const int* n_tiles, int max_tiles, void* C, int ldc, int N, int K, int gated, int act,
+                           int in_dtype, int out_dtype, int tensor_cores, int tile_rows, cudaStream_t stream) {
+    return vx_moe_gemm_scaled(A, lda, src_of_row, src_div, W, tiles, n_tiles, max_tiles, C, ldc, N, K, gated, act, in_dtype,
+                              out_dtype, tensor_cores, tile_rows, nullptr, stream);
 }
 
 // out[p, :] = x[src_of_row[p] / div, :] for the rows p of expert order (16 bytes a thread and step): the
@@ -798,7 +837,7 @@ __global__ void moe_combine_kernel(const TY* __restrict__ y, const int* __restri
         // (a negative row: the assignment went to an identity expert, whose output is the token's own row)
         const bool same = chosen && chosen[(size_t)t * top + threadIdx.x] >= n_real;
         row_s[threadIdx.x] = same ? -1 : row_of[(size_t)t * top + threadIdx.x];
-        w_s[threadIdx.x] = weight[(size_t)t * top + threadIdx.x];
+        w_s[threadIdx.x] = weight ? weight[(size_t)t * top + threadIdx.x] : 1.f;
     }
     __syncthreads();
     const float g = shared_gate ? shared_gate[t] : 1.f;

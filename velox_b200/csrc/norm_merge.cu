@@ -344,7 +344,7 @@ __global__ void act_vec_kernel(const TI* __restrict__ x, int ldx, TO* __restrict
 extern "C" int vx_act(const void* x, int ldx, void* out, int rows, int width, int act, int in_dtype, int out_dtype,
                       cudaStream_t stream) {
     if (rows <= 0 || width <= 0) return VX_OK;
-    if (ldx < width || act < 0 || act > VX_ACT_IDENTITY) return VX_ERR_SHAPE;
+    if (ldx < width || act < 0 || act > VX_ACT_LAST) return VX_ERR_SHAPE;
     const long long total = (long long)rows * width;
     if (width % 8 == 0 && ldx % 8 == 0 && !((((uintptr_t)x) | ((uintptr_t)out)) & 15)) {
         const long long chunks = total / 8;

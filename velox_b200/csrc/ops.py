@@ -20,7 +20,7 @@ from . import build as _build
 _LIB = None
 
 VX_F32, VX_BF16 = 0, 1
-ACTIVATIONS = {"silu": 0, "gelu": 1, "gelu_pytorch_tanh": 2, "relu": 3}
+ACTIVATIONS = {"silu": 0, "gelu": 1, "gelu_pytorch_tanh": 2, "relu": 3, "relu2": 5}   # (relu2: the square of relu)
 _ACT_IDENTITY = 4   # (the activation kernel as a plain change of element type)
 _ERRORS = {
     -1: "a size the kernel does not take",
@@ -124,6 +124,18 @@ def _declare(lib) -> None:
         "vx_biased_attention_shared": [P, I, P, P, P, I, P, P, P, P, P, I, F, F, I, I, I, I, I, I, I, I, I, P, I, P, I, F, I, I, P],
         "vx_biased_attention_rows_window": [P, I, P, c_longlong, c_longlong, P, c_longlong, c_longlong, P, I, P, P, P, P, I, F, I, I,
                                             I, I, I, I, I, F, I, P],
+        "vx_shift_norm": [P, P, P, P, F, P, P, I, P, P, P, I, I, P, P, P, P, I, I, I, P],
+        "vx_shift_mix": [P, P, I, P, P, P, I, P, P, I, I, I, P],
+        "vx_low_rank_decay": [P, I, I, P, P, P, I, I, P],
+        "vx_linear_attention_walk_bonus": [P, I, I, I, I, P, P, I, F, P, I, I, P, F, F, P, P, P, P, I, I, I, I, I, P, I, I, P],
+        "vx_stretch_log_decay_form": [P, I, F, P, P, I, I, I, P],
+        "vx_head_norm_gate_heads": [P, P, I, P, I, P, I, I, I, F, I, I, I, P],
+        "vx_paged_attention_generic_chunk": [P, I, P, P, P, I, P, P, P, I, F, I, I, I, I, I, I, I, I, I, F, P, I, F, I, I, I, I, P],
+        "vx_biased_attention_chunk": [P, I, P, P, P, I, P, P, P, P, P, I, F, F, I, I, I, I, I, I, I, I, I, P, I, P, I, F, I, I, I, P],
+        "vx_gemm_skinny_act": [P, P, P, P, I, I, I, I, I, I, I, I, I, I, P],
+        "vx_gemm_skinny_inputs": [P, P, P, I, I, I, I, I, I, I, c_longlong, I, I, P],
+        "vx_moe_gemm_scaled": [P, I, P, I, P, P, P, I, P, I, I, I, I, I, I, I, I, I, P, P],
+        "vx_moe_gemm_tcgen05_scaled": [P, P, P, I, I, I, I, I, I, I, I, P, P, I, P, P, P, P],
         "vx_latent_gather_window": [P, P, I, P, P, P, P, I, P, I, I, I, I, I, I, I, P],
     }
     lib.vx_set_pdl_mask.argtypes = [I]
@@ -284,7 +296,7 @@ def qk_norm_rope_kv(qkv: torch.Tensor, q_weight, k_weight, eps: float, inv_freq,
     and values into the pools [pages, Hk, S, D] and [pages, Hv, S, Dv] when a slot mapping is given
     (`v_head_dim` 0: values of the keys' size; `num_v_heads` 0: as many value heads as key heads).  The rotation pairs
     channel i with i + rot_dim/2, or, when `interleaved`, channel 2i with 2i + 1; cosines and sines are multiplied by
-    `magnitude`."""
+    `magnitude`.  Without a slot mapping a row may hold queries only (`num_kv_heads` 0)."""
     v_head_dim = int(v_head_dim) or head_dim
     num_v_heads = int(num_v_heads) or num_kv_heads
     _dev(qkv, q_weight, k_weight, inv_freq, positions, slot_mapping, k_pool, v_pool)
@@ -322,7 +334,7 @@ def paged_attention_generic(q: torch.Tensor, q_row_stride: int, k_pool, v_pool, 
                             num_kv_heads: int, head_dim: int, tokens: int, v_head_dim: int = 0, keep_first: int = 0,
                             bias_exponent: float = 0.0, sinks: Optional[torch.Tensor] = None,
                             gate_col: int = -1, softcap: float = 0.0, v_stride: int = 0, v_share: int = 1,
-                            out_float32: bool = False) -> torch.Tensor:
+                            out_float32: bool = False, chunk: int = 0) -> torch.Tensor:
     """The general kernel.  `v_head_dim`: size of a value (0: a key's); `keep_first`: with a window, the
     first positions that stay visible; `bias_exponent` b > 0: head h's scores lose
     2^(-b (h + 1) / heads) * distance; `sinks` (float32 per head): the softmax's denominator also holds
@@ -330,7 +342,8 @@ def paged_attention_generic(q: torch.Tensor, q_row_stride: int, k_pool, v_pool, 
     `softcap` c > 0: a scaled score s becomes c tanh(s / c); `v_stride`: elements from one value row of
     `v_pool` to the next (0: v_head_dim), for a pool whose rows hold the value inside the key's row; `v_share` > 1: that
     many consecutive key heads read one value head (the value pool has num_kv_heads / v_share heads); `out_float32`: the
-    result is float32 whatever the queries' element type."""
+    result is float32 whatever the queries' element type; `chunk` > 0: a query sees keys of its own run of `chunk` positions
+    only, the runs counted from position 0 (not with kept first positions)."""
     _dev(q, k_pool, v_pool, block_table, seq_of_token, positions, sinks)
     _need(v_share >= 1 and num_kv_heads % v_share == 0, "paged_attention: v_share must divide the key heads")
     _check_sinks_gate("paged_attention", sinks, gate_col, num_heads, q_row_stride)
@@ -343,12 +356,12 @@ def paged_attention_generic(q: torch.Tensor, q_row_stride: int, k_pool, v_pool, 
           "paged_attention: head sizes %d / %d (the general kernel takes sizes up to %d)"
           % (head_dim, v_head_dim, ATTENTION_MAX_HEAD_DIM))
     out = torch.empty((tokens, num_heads * v_head_dim), dtype=torch.float32 if out_float32 else q.dtype, device=q.device)
-    _check(library().vx_paged_attention_generic_shared(
+    _check(library().vx_paged_attention_generic_chunk(
         _ptr(q), q_row_stride, _ptr(k_pool), _ptr(v_pool), _ptr(block_table), block_table.shape[1],
         _ptr(seq_of_token), _ptr(positions), _ptr(out), num_heads * v_head_dim, float(scale), int(window), tokens,
         num_heads, num_kv_heads, head_dim, page_size, dtype_code(q.dtype), v_head_dim, int(keep_first),
         float(bias_exponent), _ptr(sinks), int(gate_col), float(softcap), int(v_stride), int(v_share),
-        1 if out_float32 else 0, _stream()), "paged_attention_generic")
+        1 if out_float32 else 0, int(chunk), _stream()), "paged_attention_generic")
     return out
 
 
@@ -376,7 +389,8 @@ def biased_attention_supported(dtype, head_dim: int, v_head_dim: int, page_size:
 
 def _biased_attention(q, q_row_stride, k_pool, v_pool, block_table, cu_seqlens, kv_offsets, seq_of_token, positions,
                       scale, window, keep_first, bias_exponent, num_heads, num_kv_heads, head_dim, v_head_dim, segments,
-                      max_new, tokens, out, max_kv=0, sinks=None, gate_col=-1, softcap=0.0, v_share=1, out_float32=False):
+                      max_new, tokens, out, max_kv=0, sinks=None, gate_col=-1, softcap=0.0, v_share=1, out_float32=False,
+                      chunk=0):
     _dev(q, k_pool, v_pool, block_table, cu_seqlens, kv_offsets, seq_of_token, positions, out, sinks)
     _need(v_share >= 1 and num_kv_heads % v_share == 0 and v_pool.shape[1] * v_share == k_pool.shape[1] == num_kv_heads,
           "biased_attention: value heads times v_share must be the key heads")
@@ -394,43 +408,46 @@ def _biased_attention(q, q_row_stride, k_pool, v_pool, block_table, cu_seqlens, 
     runs, scratch = 1, None
     if cu_seqlens is None and max_kv > 0:
         keys = max_kv if window <= 0 else min(max_kv, window + keep_first)
+        keys = min(keys, chunk) if chunk > 0 else keys
         runs = max(1, min(BIASED_DECODE_MAX_RUNS, -(-keys // 16) // 16))
         if runs > 1:
             scratch = workspace(q.device, tokens * num_heads * runs * (v_head_dim + 2), which="biased_decode")
-    _check(library().vx_biased_attention_shared(
+    _check(library().vx_biased_attention_chunk(
         _ptr(q), q_row_stride, _ptr(k_pool), _ptr(v_pool), _ptr(block_table), block_table.shape[1], _ptr(cu_seqlens),
         _ptr(kv_offsets), _ptr(seq_of_token), _ptr(positions), _ptr(out), num_heads * v_head_dim, float(scale),
         float(bias_exponent), int(window), int(keep_first), int(segments), int(max_new), num_heads, num_kv_heads, head_dim,
         v_head_dim, k_pool.shape[2], _ptr(scratch), runs, _ptr(sinks), int(gate_col), float(softcap), int(v_share),
-        1 if out_float32 else 0, _stream()), "biased_attention")
+        1 if out_float32 else 0, int(chunk), _stream()), "biased_attention")
     return out
 
 
 def biased_prefill_attention(q, q_row_stride, k_pool, v_pool, block_table, cu_seqlens, kv_offsets, scale: float,
                              window: int, keep_first: int, bias_exponent: float, num_heads: int, num_kv_heads: int,
                              head_dim: int, v_head_dim: int, requests: int, max_new: int, tokens: int, out=None,
-                             sinks=None, gate_col: int = -1, softcap: float = 0.0, v_share: int = 1, out_float32: bool = False):
+                             sinks=None, gate_col: int = -1, softcap: float = 0.0, v_share: int = 1, out_float32: bool = False,
+                             chunk: int = 0):
     """Attention of prompt portions (request i: rows cu_seqlens[i] .. at positions kv_offsets[i] ..) with
     score = q.k * scale - 2^(-bias_exponent (h+1) / heads) * distance under a window that keeps the first
     `keep_first` positions; bfloat16, tensor cores, probabilities in two bfloat16 halves.  `sinks`, `gate_col` and
-    `softcap`, `v_share` and `out_float32` as in `paged_attention_generic`."""
+    `softcap`, `v_share`, `out_float32` and `chunk` as in `paged_attention_generic`."""
     return _biased_attention(q, q_row_stride, k_pool, v_pool, block_table, cu_seqlens, kv_offsets, None, None, scale,
                              window, keep_first, bias_exponent, num_heads, num_kv_heads, head_dim, v_head_dim, requests,
                              max_new, tokens, out, sinks=sinks, gate_col=gate_col, softcap=softcap, v_share=v_share,
-                             out_float32=out_float32)
+                             out_float32=out_float32, chunk=chunk)
 
 
 def biased_decode_attention(q, q_row_stride, k_pool, v_pool, block_table, seq_of_token, positions, scale: float,
                             window: int, keep_first: int, bias_exponent: float, num_heads: int, num_kv_heads: int,
                             head_dim: int, v_head_dim: int, tokens: int, out=None, max_kv: int = 0, sinks=None,
-                            gate_col: int = -1, softcap: float = 0.0, v_share: int = 1, out_float32: bool = False):
+                            gate_col: int = -1, softcap: float = 0.0, v_share: int = 1, out_float32: bool = False,
+                            chunk: int = 0):
     """The same for token rows that each stand alone: row t is request seq_of_token[t] at position positions[t].
     `max_kv` (a bound on any row's position + 1; 0: unknown) lets rows with many visible keys be cut into runs that
     several blocks share."""
     return _biased_attention(q, q_row_stride, k_pool, v_pool, block_table, None, None, seq_of_token, positions, scale,
                              window, keep_first, bias_exponent, num_heads, num_kv_heads, head_dim, v_head_dim, tokens, 1,
                              tokens, out, max_kv=max_kv, sinks=sinks, gate_col=gate_col, softcap=softcap, v_share=v_share,
-                             out_float32=out_float32)
+                             out_float32=out_float32, chunk=chunk)
 
 
 def embedding_pair(ids, positions, seq_of_token, cu_seqlens, state_slots, last_token: torch.Tensor,
@@ -620,6 +637,7 @@ class MoePlan:
 
 
 _MOE_COUNTS = {}
+MOE_SCORES = {"softmax_chosen": 0, "softmax_all": 1, "sigmoid": 2}
 
 
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, bias, experts: int, top: int,
@@ -631,13 +649,13 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, bias, experts: int, top: 
     `experts` counts the router's outputs.  `scores="softmax_all"`: scores s = softmax over all outputs, choice by
     s + `correction` (float32 per output) among the outputs of the `keep_groups` best of `groups` equal groups of
     neighbours, weights s * route_scale (not renormalised).  The last `identity` outputs are identity experts (the
-    combination takes the token's own row for them).  With `shared_gate` the router's matrix has one more row, and
+    combination takes the token's own row for them).  `scores="sigmoid"`: the same with scores sigmoid(logit).  With `shared_gate` the router's matrix has one more row, and
     `plan.shared_gate` [tokens] is sigmoid(that row . h)."""
     _dev(h, w_router, bias, correction)
     rows = experts + (1 if shared_gate else 0)
     _need(h.stride(1) == 1 and w_router.dtype == torch.float32 and w_router.is_contiguous()
           and tuple(w_router.shape) == (rows, h.shape[1]), "moe_route: float32 router [outputs (+ 1 for a shared gate), width]")
-    _need(scores in ("softmax_chosen", "softmax_all"), "moe_route: scores %r" % (scores,))
+    _need(scores in MOE_SCORES, "moe_route: scores %r" % (scores,))
     _need(groups >= 1 and experts % groups == 0 and 1 <= keep_groups <= groups and top <= keep_groups * (experts // groups)
           and 0 <= identity < experts, "moe_route: groups, kept groups, top and identity experts do not fit the outputs")
     for b in (bias, correction):
@@ -663,18 +681,23 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, bias, experts: int, top: 
     _check(library().vx_moe_route(_ptr(h), h.stride(0), _ptr(w_router), _ptr(bias), t, h.shape[1], experts, top,
                                   plan.tile_rows, _ptr(plan.chosen), _ptr(plan.weight), _ptr(counts), _ptr(pos), _ptr(offsets),
                                   _ptr(plan.tiles), _ptr(plan.n_tiles), _ptr(plan.src_of_row), _ptr(plan.row_of),
-                                  dtype_code(h.dtype), 1 if scores == "softmax_all" else 0, _ptr(correction), int(groups),
+                                  dtype_code(h.dtype), MOE_SCORES[scores], _ptr(correction), int(groups),
                                   int(keep_groups), float(route_scale), int(identity), _ptr(plan.shared_gate), _stream()),
            "moe_route")
     return plan
 
 
 def moe_gemm(a: torch.Tensor, w: torch.Tensor, plan: MoePlan, gather: bool, out_dtype: torch.dtype,
-             gated_activation: Optional[str] = None) -> torch.Tensor:
+             gated_activation: Optional[str] = None, activation: Optional[str] = None,
+             row_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Grouped product in expert order: row p of the result is a[src(p)] times w[expert of p] transposed, with
     w [experts, N, K]; src(p) is the token of assignment p (`gather`) or p itself.  With `gated_activation`,
-    w's rows come in tiles of 8 gate rows followed by their 8 up rows and the result is act(gate) * up."""
-    _dev(a, w)
+    w's rows come in tiles of 8 gate rows followed by their 8 up rows and the result is act(gate) * up; with `activation` it
+    is act(.) of each sum.  `row_scale` (float32, one per assignment) multiplies an assignment's sums before either."""
+    _dev(a, w, row_scale)
+    code, act = _epilogue("moe_gemm", gated_activation, activation)
+    _need(row_scale is None or (row_scale.dtype == torch.float32 and row_scale.numel() == plan.assignments and row_scale.is_contiguous()),
+          "moe_gemm: one float32 scale per assignment")
     _need(a.stride(1) == 1 and w.is_contiguous() and w.dim() == 3 and w.shape[2] == a.shape[1] and a.dtype == w.dtype,
           "moe_gemm: a [rows, K], w [experts, N, K] of one element type")
     n, k = w.shape[1], w.shape[2]
@@ -683,11 +706,20 @@ def moe_gemm(a: torch.Tensor, w: torch.Tensor, plan: MoePlan, gather: bool, out_
     tc = moe_mma_supported(a, k) and w.data_ptr() % 16 == 0
     _need(plan.tile_rows == MOE_TILE_ROWS or (plan.tile_rows == MOE_SMALL_TILE_ROWS and tc),
           "moe_gemm: row tiles of %d, or of %d on the tensor cores" % (MOE_TILE_ROWS, MOE_SMALL_TILE_ROWS))
-    _check(library().vx_moe_gemm(_ptr(a), a.stride(0), _ptr(plan.src_of_row) if gather else None, plan.top if gather else 1,
-                                 _ptr(w), _ptr(plan.tiles), _ptr(plan.n_tiles), plan.max_tiles, _ptr(out), cols, n, k,
-                                 1 if gated_activation else 0, ACTIVATIONS.get(gated_activation, 0), dtype_code(a.dtype),
-                                 dtype_code(out_dtype), 1 if tc else 0, plan.tile_rows, _stream()), "moe_gemm")
+    _need(gather or row_scale is None, "moe_gemm: scales by assignment go with the product that gathers the tokens' rows")
+    _check(library().vx_moe_gemm_scaled(_ptr(a), a.stride(0), _ptr(plan.src_of_row) if gather else None, plan.top if gather else 1,
+                                        _ptr(w), _ptr(plan.tiles), _ptr(plan.n_tiles), plan.max_tiles, _ptr(out), cols, n, k,
+                                        code, act, dtype_code(a.dtype), dtype_code(out_dtype), 1 if tc else 0, plan.tile_rows,
+                                        _ptr(row_scale), _stream()), "moe_gemm")
     return out
+
+
+def _epilogue(what: str, gated_activation: Optional[str], activation: Optional[str]):
+    """(epilogue code, activation code) of a matrix product: plain, act(gate) * up of paired rows, or act(.)."""
+    _need(gated_activation is None or activation is None, "%s: a gated activation or a plain one" % what)
+    name = gated_activation or activation
+    _need(name is None or name in ACTIVATIONS, "%s: unknown activation %r" % (what, name))
+    return (1 if gated_activation else (2 if activation else 0)), ACTIVATIONS.get(name, 0)
 
 
 def moe_mma_supported(a: torch.Tensor, k: int) -> bool:
@@ -717,28 +749,35 @@ def moe_gather_rows(x: torch.Tensor, plan: MoePlan) -> torch.Tensor:
     return out
 
 
-def moe_gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, plan: MoePlan, gated_activation: Optional[str] = None) -> torch.Tensor:
+def moe_gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, plan: MoePlan, gated_activation: Optional[str] = None,
+                     activation: Optional[str] = None, row_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The grouped product on the tcgen05 tensor cores: `a` [assignments, K] bfloat16 IN EXPERT ORDER, w [experts, N, K];
-    the plan's row tiles must be of `MOE_TCGEN05_TILE_ROWS` rows.  bfloat16 out."""
-    _dev(a, w)
+    the plan's row tiles must be of `MOE_TCGEN05_TILE_ROWS` rows.  bfloat16 out.  `activation` and `row_scale` as in
+    `moe_gemm`."""
+    _dev(a, w, row_scale)
+    code, act = _epilogue("moe_gemm_tcgen05", gated_activation, activation)
+    _need(row_scale is None or (code and row_scale.dtype == torch.float32 and row_scale.numel() == plan.assignments),
+          "moe_gemm_tcgen05: one float32 scale per assignment, with an activation")
     _need(a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.is_contiguous() and w.dim() == 3
           and a.shape == (plan.assignments, w.shape[2]) and plan.tile_rows == MOE_TCGEN05_TILE_ROWS,
           "moe_gemm_tcgen05: bfloat16 a [assignments, K] in expert order, w [experts, N, K], row tiles of 128")
     n, k = w.shape[1], w.shape[2]
     cols = n // 2 if gated_activation else n
     out = torch.empty((plan.assignments, cols), dtype=torch.bfloat16, device=a.device)
-    _check(library().vx_moe_gemm_tcgen05(_ptr(a), _ptr(w), _ptr(out), plan.assignments, w.shape[0], n, k, a.stride(0), cols,
-                                         1 if gated_activation else 0, ACTIVATIONS.get(gated_activation, 0), _ptr(plan.tiles),
-                                         _ptr(plan.n_tiles), plan.max_tiles, _ptr(_error_word(a.device)), _stream()),
+    _check(library().vx_moe_gemm_tcgen05_scaled(_ptr(a), _ptr(w), _ptr(out), plan.assignments, w.shape[0], n, k, a.stride(0), cols,
+                                                code, act, _ptr(plan.tiles), _ptr(plan.n_tiles), plan.max_tiles,
+                                                _ptr(_error_word(a.device)), _ptr(row_scale),
+                                                _ptr(plan.src_of_row) if row_scale is not None else None, _stream()),
            "moe_gemm_tcgen05")
     note_bounded_wait()
     return out
 
 
-def moe_combine(y: torch.Tensor, plan: MoePlan, shared_out, out_dtype: torch.dtype, h=None) -> torch.Tensor:
+def moe_combine(y: torch.Tensor, plan: MoePlan, shared_out, out_dtype: torch.dtype, h=None, weighted: bool = True) -> torch.Tensor:
     """Per token the weighted sum of its experts' rows of `y` (expert order; float32, or the result's element
     type), plus `shared_out` (times the plan's shared gate, if it has one).  A plan with identity experts needs
-    `h`, the tokens' rows that went into the router: an assignment to one of them adds weight * h[t]."""
+    `h`, the tokens' rows that went into the router: an assignment to one of them adds weight * h[t].  `weighted=False`:
+    the plain sum (the weights went into the grouped products)."""
     _dev(y, shared_out, h)
     if plan.identity:
         _need(h is not None and h.dtype == out_dtype and h.stride(1) == 1 and h.shape[1] == y.shape[1],
@@ -749,7 +788,7 @@ def moe_combine(y: torch.Tensor, plan: MoePlan, shared_out, out_dtype: torch.dty
         _need(shared_out.dtype == out_dtype and shared_out.is_contiguous() and tuple(shared_out.shape) == (t, y.shape[1]),
               "moe_combine: the shared expert's output in the result's shape and element type")
     out = torch.empty((t, y.shape[1]), dtype=out_dtype, device=y.device)
-    _check(library().vx_moe_combine(_ptr(y), _ptr(plan.row_of), _ptr(plan.weight), _ptr(shared_out), _ptr(out), t, y.shape[1],
+    _check(library().vx_moe_combine(_ptr(y), _ptr(plan.row_of), _ptr(plan.weight) if weighted else None, _ptr(shared_out), _ptr(out), t, y.shape[1],
                                     plan.top, dtype_code(out_dtype), dtype_code(y.dtype),
                                     _ptr(plan.chosen) if plan.identity else None, plan.experts - plan.identity,
                                     _ptr(h) if plan.identity else None, h.stride(0) if plan.identity else 0,
@@ -956,34 +995,40 @@ def linear_attention_walk(x: torch.Tensor, q_col: int, k_col: int, v_col: int, s
                           seqs: int, heads: int, dim: int, vdim: int, decay: Optional[torch.Tensor] = None,
                           gate: Optional[torch.Tensor] = None, gate_mul: float = 1.0, inv_freq: Optional[torch.Tensor] = None,
                           rot_dim: int = 0, interleaved: bool = False, positions: Optional[torch.Tensor] = None,
-                          q_mul: float = 1.0, k_mul: float = 1.0, stretches: Optional[StretchPlan] = None) -> torch.Tensor:
+                          q_mul: float = 1.0, k_mul: float = 1.0, stretches: Optional[StretchPlan] = None,
+                          bonus: Optional[torch.Tensor] = None, gate_is_log: bool = False) -> torch.Tensor:
     """Per head S = a (.) S + k v^T, o = S^T q over every request's tokens in order, a = decay[h] (float32 per head) or
     sigmoid(gate)^gate_mul per key channel and token (`gate` float32 [tokens, heads * dim], contiguous rows).  q and k
     are turned by position * inv_freq on their first `rot_dim` channels, then multiplied by q_mul / k_mul, all in
     float32.  `state` float32 [slots, heads, dim, vdim] is read and written back.  Returns float32 [tokens, heads * vdim].
+    With `gate_is_log` the gate is the decay's logarithm itself.  With `bonus` u (float32 [heads, dim], with a gate) the
+    output is taken before the update and the token's own key and value enter it weighed by u: o = (S + diag(u) k v^T)^T q.
     With `stretches` (the plan of this step's rows) the stretches are walked side by side: once from zero for what each
     adds to the state, a scan over a request's stretches for the state at the start of each, and once more for the outputs."""
     _dev(x, decay, gate, inv_freq, positions, state, cu_seqlens, state_slots)
-    _need(x.stride(1) == 1 and (decay is None) != (gate is None), "linear_attention_walk: a decay per head or a gate per channel")
+    _need(x.stride(-1) == 1 and (decay is None) != (gate is None), "linear_attention_walk: a decay per head or a gate per channel")
     if decay is not None:
         _need(decay.dtype == torch.float32 and decay.numel() == heads, "linear_attention_walk: float32 decay per head")
     if gate is not None:
-        _need(gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape == (x.shape[0], heads * dim),
+        _need(gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape == (x.shape[-2], heads * dim),
               "linear_attention_walk: float32 gate [tokens, heads * dim]")
     if inv_freq is not None:
         _need(inv_freq.dtype == torch.float32 and inv_freq.numel() * 2 == rot_dim and positions is not None
               and positions.dtype == torch.int32, "linear_attention_walk: inv_freq of rot_dim / 2 numbers, int32 positions")
     _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, dim, vdim),
           "linear_attention_walk: float32 state [slots, heads, dim, vdim]")
-    out = torch.empty((x.shape[0], heads * vdim), dtype=torch.float32, device=x.device)
+    _need(bonus is None or (gate is not None and bonus.dtype == torch.float32 and bonus.is_contiguous() and bonus.numel() == heads * dim),
+          "linear_attention_walk: a float32 bonus [heads, dim], with a gate")
+    tokens = x.shape[0] if x.dim() == 2 else x.shape[1]
+    out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=x.device)
     lib = library()
 
     def walk(st, cu, slots, n, result, fresh):
-        _check(lib.vx_linear_attention_walk_parts(
-            _ptr(x), x.stride(0), int(q_col), int(k_col), int(v_col), _ptr(decay), _ptr(gate), gate.stride(0) if gate is not None else 0,
+        _check(lib.vx_linear_attention_walk_bonus(
+            _ptr(x), x.stride(-2), int(q_col), int(k_col), int(v_col), _ptr(decay), _ptr(gate), gate.stride(0) if gate is not None else 0,
             float(gate_mul), _ptr(inv_freq), int(rot_dim) if inv_freq is not None else 0, 1 if interleaved else 0, _ptr(positions),
             float(q_mul), float(k_mul), _ptr(st), _ptr(cu), _ptr(slots), _ptr(result), int(n), heads, dim, vdim,
-            1 if fresh else 0, dtype_code(x.dtype), _stream()), "linear_attention_walk")
+            1 if fresh else 0, _ptr(bonus), 1 if gate_is_log else 0, dtype_code(x.dtype), _stream()), "linear_attention_walk")
 
     if stretches is None:
         walk(state, cu_seqlens, state_slots, seqs, out, False)
@@ -994,8 +1039,8 @@ def linear_attention_walk(x: torch.Tensor, q_col: int, k_col: int, v_col: int, s
     log_a = None
     if gate is not None:
         log_a = workspace(x.device, stretches.count * heads * dim, which="stretch_decay")
-        _check(lib.vx_stretch_log_decay(_ptr(gate), gate.stride(0), float(gate_mul), _ptr(stretches.cu), _ptr(log_a),
-                                        stretches.count, heads * dim, _stream()), "stretch_log_decay")
+        _check(lib.vx_stretch_log_decay_form(_ptr(gate), gate.stride(0), float(gate_mul), _ptr(stretches.cu), _ptr(log_a),
+                                             stretches.count, heads * dim, 1 if gate_is_log else 0, _stream()), "stretch_log_decay")
     walk(parts, stretches.cu, stretches.ident, stretches.count, None, True)
     _check(lib.vx_stretch_scan(_ptr(parts), _ptr(state), _ptr(log_a), _ptr(decay), _ptr(stretches.cu), _ptr(stretches.first),
                                _ptr(state_slots), seqs, heads, dim, vdim, _stream()), "stretch_scan")
@@ -1004,19 +1049,22 @@ def linear_attention_walk(x: torch.Tensor, q_col: int, k_col: int, v_col: int, s
 
 
 def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.Tensor], heads: int, eps: float,
-                   gate_activation: str = "silu") -> torch.Tensor:
-    """Every head of o (float32 [rows, heads * vdim]) divided by its root mean square, times `weight` [vdim] if given,
-    times silu or sigmoid of `gate` [rows, heads * vdim] (contiguous rows); in the gate's element type."""
+                   gate_activation: str = "silu", out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """Every head of o (float32 [rows, heads * vdim]) divided by its root mean square, times `weight` if given ([vdim], shared
+    by the heads, or [heads * vdim]), times silu or sigmoid of `gate` [rows, heads * vdim] (contiguous rows); in `out_dtype`
+    (the gate's element type unless given)."""
     _dev(o, gate, weight)
     vdim = o.shape[1] // heads
     _need(o.dtype == torch.float32 and o.is_contiguous() and gate.stride(1) == 1 and gate.shape == o.shape
           and o.shape[1] == heads * vdim, "head_norm_gate: float32 outputs and a gate of their shape")
-    _need(weight is None or (weight.dtype == torch.float32 and weight.numel() == vdim), "head_norm_gate: float32 weight [vdim]")
+    _need(weight is None or (weight.dtype == torch.float32 and weight.numel() in (vdim, heads * vdim)),
+          "head_norm_gate: float32 weight [vdim] or [heads * vdim]")
+    per_head = weight is not None and weight.numel() == heads * vdim
     _need(gate_activation in ("silu", "sigmoid"), "head_norm_gate: the gate passes through silu or sigmoid")
-    out = torch.empty(o.shape, dtype=gate.dtype, device=o.device)
-    _check(library().vx_head_norm_gate(_ptr(o), _ptr(gate), gate.stride(0), _ptr(weight), _ptr(out), o.shape[0], heads, vdim,
-                                       float(eps), 1 if gate_activation == "silu" else 0, dtype_code(gate.dtype), _stream()),
-           "head_norm_gate")
+    out = torch.empty(o.shape, dtype=out_dtype or gate.dtype, device=o.device)
+    _check(library().vx_head_norm_gate_heads(_ptr(o), _ptr(gate), gate.stride(0), _ptr(weight), 1 if per_head else 0, _ptr(out),
+                                             o.shape[0], heads, vdim, float(eps), 1 if gate_activation == "silu" else 0,
+                                             dtype_code(gate.dtype), dtype_code(out.dtype), _stream()), "head_norm_gate")
     return out
 
 
@@ -1279,6 +1327,78 @@ def sum_add_rmsnorm(residual: torch.Tensor, branches=(), rows_add: Optional[torc
     return out
 
 
+SHIFT_MAX_MIXES = 8
+
+
+def shift_norm_max_width(width: int) -> int:
+    """The widest row that `shift_norm` takes beside `width`: 512 threads own 8 groups of 4 channels, or of one channel
+    where the width is no multiple of 4."""
+    return 512 * 8 * (4 if width % 4 == 0 else 1)
+
+
+def shift_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, eps: float, shift: torch.Tensor, ctx,
+               state: torch.Tensor, out_dtype: torch.dtype, mixes: Optional[torch.Tensor] = None,
+               mix_state: Optional[torch.Tensor] = None):
+    """x = residual (+ delta) (float32 [tokens, E]); n = rmsnorm(x) * weight; h_t = n_t + (n_(t-1) - n_t) * shift, the row before
+    a request's first one of this step being its slot's row of `state` (float32 [slots, E]), which then takes the request's
+    last n.  Returns (x, h).  With `mixes` (float32 [k, E]) h itself is shifted again, once per row of it:
+    out[i, t] = h_t + (h_(t-1) - h_t) * mixes[i], with `mix_state` [slots, E] holding the requests' last h; the result is then
+    [k, tokens, E].  With a delta x is a new tensor (blocks of the kernel read rows that others update)."""
+    _dev(residual, delta, weight, shift, state, mixes, mix_state)
+    tokens, E = residual.shape
+    _need(residual.dtype == torch.float32 and residual.is_contiguous(), "shift_norm: float32 contiguous residual")
+    _need(delta is None or (delta.dtype == out_dtype and delta.is_contiguous() and delta.shape == residual.shape),
+          "shift_norm: a delta of the residual's shape and the output's element type")
+    for v in (weight, shift):
+        _need(v.dtype == torch.float32 and v.numel() == E and v.is_contiguous(), "shift_norm: float32 vectors of the row's width")
+    for s in (state, mix_state):
+        _need(s is None or (s.dtype == torch.float32 and s.is_contiguous() and s.dim() == 2 and s.shape[1] == E), "shift_norm: float32 state [slots, E]")
+    k = 0
+    if mixes is not None:
+        k = mixes.shape[0]
+        _need(mixes.dtype == torch.float32 and mixes.is_contiguous() and mixes.shape[1] == E and 0 < k <= SHIFT_MAX_MIXES
+              and mix_state is not None, "shift_norm: float32 mixes [k, E] with a state of their own")
+    x = residual if delta is None else torch.empty_like(residual)
+    out = torch.empty((k, tokens, E) if k else (tokens, E), dtype=out_dtype, device=residual.device)
+    save = workspace(residual.device, ctx.n_seqs * 2 * E, which="shift_norm") if ctx.max_new > 1 else None
+    _check(library().vx_shift_norm(_ptr(residual), _ptr(delta), _ptr(x) if delta is not None else None, _ptr(weight), float(eps),
+                                   _ptr(shift), _ptr(mixes), k, _ptr(ctx.seq_of_token), _ptr(ctx.cu_seqlens), _ptr(ctx.state_slots),
+                                   ctx.n_seqs, ctx.max_new, _ptr(state), _ptr(mix_state), _ptr(save), _ptr(out), tokens, E,
+                                   dtype_code(out_dtype), _stream()), "shift_norm")
+    return x, out
+
+
+def shift_mix(h: torch.Tensor, mixes: torch.Tensor, ctx, mix_state: torch.Tensor) -> torch.Tensor:
+    """The second shift of `shift_norm` alone: out[i, t] = h_t + (h_(t-1) - h_t) * mixes[i] ([k, tokens, E] in h's element
+    type); `mix_state` float32 [slots, E] is read for a request's first row and takes its last."""
+    _dev(h, mixes, mix_state)
+    k, (tokens, E) = mixes.shape[0], h.shape
+    _need(h.is_contiguous() and mixes.dtype == torch.float32 and mixes.is_contiguous() and mixes.shape[1] == E
+          and 0 < k <= SHIFT_MAX_MIXES and mix_state.dtype == torch.float32 and mix_state.is_contiguous() and mix_state.shape[1] == E,
+          "shift_mix: rows [tokens, E], float32 mixes [k, E] and state [slots, E]")
+    out = torch.empty((k, tokens, E), dtype=h.dtype, device=h.device)
+    _check(library().vx_shift_mix(_ptr(h), _ptr(mixes), k, _ptr(ctx.seq_of_token), _ptr(ctx.cu_seqlens), _ptr(ctx.state_slots),
+                                  ctx.n_seqs, _ptr(mix_state), _ptr(out), tokens, E, dtype_code(h.dtype), _stream()), "shift_mix")
+    return out
+
+
+LOW_RANK_DECAY_MAX_RANK = 1024
+
+
+def low_rank_decay(x: torch.Tensor, weight_t: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
+    """-exp(tanh(x) weight_t + bias), float32 throughout: the logarithm of a decay per channel.  x [tokens, rank] (contiguous
+    rows), weight_t [rank, channels], bias [channels]."""
+    _dev(x, weight_t, bias)
+    rank, c = weight_t.shape
+    _need(x.dtype == torch.float32 and x.stride(1) == 1 and x.shape[1] == rank and weight_t.dtype == torch.float32
+          and weight_t.is_contiguous() and bias.dtype == torch.float32 and bias.numel() == c and rank <= LOW_RANK_DECAY_MAX_RANK,
+          "low_rank_decay: float32 x [tokens, rank], weight [rank, channels], bias [channels], rank up to %d" % LOW_RANK_DECAY_MAX_RANK)
+    out = torch.empty((x.shape[0], c), dtype=torch.float32, device=x.device)
+    _check(library().vx_low_rank_decay(_ptr(x), x.stride(0), rank, _ptr(weight_t), _ptr(bias), _ptr(out), x.shape[0], c, _stream()),
+           "low_rank_decay")
+    return out
+
+
 def softcap_rows(x: torch.Tensor, cap: float) -> torch.Tensor:
     """cap * tanh(x / cap) on float32 x."""
     _dev(x)
@@ -1370,13 +1490,16 @@ def tcgen05_pair_better(m: int, n: int, device) -> bool:
 
 
 def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, bias=None, gated_activation: Optional[str] = None,
-                 wide: bool = True, pair: bool = False) -> torch.Tensor:
+                 wide: bool = True, pair: bool = False, activation: Optional[str] = None) -> torch.Tensor:
     """a [M,K] times w [N,K] transposed on the tcgen05 tensor cores (bfloat16 in and
     out, float32 accumulation in tensor memory, operands by TMA).  With
     `gated_activation`, w's rows come in tiles of 8 gate rows followed by their 8 up
     rows and the result is act(gate) * up, [M, N/2].  `wide`: 128 x 256 tiles, else
-    128 x 128; `pair`: 256 x 256 tiles, each formed by a pair of blocks."""
+    128 x 128; `pair`: 256 x 256 tiles, each formed by a pair of blocks.  With `activation` the result is act(.) of the
+    float32 sums (single blocks only)."""
     _dev(a, w, bias)
+    code, act = _epilogue("gemm_tcgen05", gated_activation, activation)
+    _need(not (pair and activation), "gemm_tcgen05: a plain activation on tiles of single blocks")
     _need(a.dim() == 2 and w.dim() == 2 and a.shape[1] == w.shape[1], "gemm_tcgen05: a [M,K], w [N,K]")
     _need(tcgen05_supported(a, w), "gemm_tcgen05: bfloat16, K a multiple of 8, N a multiple of 16, 16-byte aligned rows")
     m, k = a.shape
@@ -1394,8 +1517,7 @@ def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, bias=None, gated_activation: 
                                               _ptr(_error_word(a.device)), _stream()), "gemm_tcgen05_pair")
     else:
         _check(library().vx_gemm_tcgen05(_ptr(a), _ptr(w), _ptr(bias), _ptr(out), m, n, k, a.stride(0), w.stride(0), cols,
-                                         1 if gated_activation else 0, ACTIVATIONS.get(gated_activation, 0),
-                                         1 if wide else 0, _ptr(_error_word(a.device)), _stream()), "gemm_tcgen05")
+                                         code, act, 1 if wide else 0, _ptr(_error_word(a.device)), _stream()), "gemm_tcgen05")
     note_bounded_wait()
     return out
 
@@ -1410,11 +1532,12 @@ def skinny_supported(m: int, k: int, a: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def gemm_skinny(a: torch.Tensor, w: torch.Tensor, bias=None, out_dtype: Optional[torch.dtype] = None,
-                gated_activation: Optional[str] = None, variant: int = 0) -> torch.Tensor:
+                gated_activation: Optional[str] = None, variant: int = 0, activation: Optional[str] = None) -> torch.Tensor:
     """a [M<=8, K] times w [N,K] transposed, W streamed once (bfloat16).  With
     `gated_activation`, w's rows come in tiles of 8 gate rows followed by their 8 up
-    rows and the result is act(gate) * up, [M, N/2]."""
+    rows and the result is act(gate) * up, [M, N/2]; with `activation` it is act(.) of the float32 sums."""
     _dev(a, w, bias)
+    code, act = _epilogue("gemm_skinny", gated_activation, activation)
     _need(a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and a.dim() == 2 and w.dim() == 2
           and a.shape[1] == w.shape[1], "gemm_skinny: bfloat16 a [M,K], w [N,K]")
     out_dtype = out_dtype or torch.bfloat16
@@ -1424,10 +1547,48 @@ def gemm_skinny(a: torch.Tensor, w: torch.Tensor, bias=None, out_dtype: Optional
     if gated_activation is not None:
         _need(gated_activation in ACTIVATIONS, "gemm_skinny: unknown activation %r" % gated_activation)
     out = torch.empty((m, cols), dtype=out_dtype, device=a.device)
-    _check(library().vx_gemm_skinny(_ptr(a), _ptr(w), _ptr(bias), _ptr(out), m, n, k, a.stride(0), w.stride(0), cols,
-                                    1 if gated_activation else 0, ACTIVATIONS.get(gated_activation, 0),
-                                    dtype_code(out_dtype), variant, _stream()), "gemm_skinny")
+    _check(library().vx_gemm_skinny_act(_ptr(a), _ptr(w), _ptr(bias), _ptr(out), m, n, k, a.stride(0), w.stride(0), cols,
+                                        1 if code == 1 else 0, act if code else -1, dtype_code(out_dtype), variant, _stream()),
+           "gemm_skinny")
     return out
+
+
+def gemm_inputs(xs: torch.Tensor, w: torch.Tensor, seg_rows: int, out_dtype: torch.dtype) -> torch.Tensor:
+    """Projections with an input each, in one launch: out[m, n] = xs[i, m] . w[n], i = n / seg_rows (at most the last input):
+    xs [inputs, M <= 8, K] bfloat16, w [N, K]; W streamed once, as in `gemm_skinny`.  Returns [M, N]."""
+    _dev(xs, w)
+    _need(xs.dim() == 3 and xs.stride(2) == 1 and xs.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.stride(1) == 1
+          and xs.shape[2] == w.shape[1], "gemm_inputs: bfloat16 xs [inputs, M, K], w [N, K]")
+    inputs, m, k = xs.shape
+    out = torch.empty((m, w.shape[0]), dtype=out_dtype, device=xs.device)
+    _check(library().vx_gemm_skinny_inputs(_ptr(xs), _ptr(w), _ptr(out), m, w.shape[0], k, xs.stride(1), w.stride(0), w.shape[0],
+                                           int(seg_rows), xs.stride(0), inputs, dtype_code(out_dtype), _stream()), "gemm_inputs")
+    return out
+
+
+def gemm_members(xs: torch.Tensor, ws: torch.Tensor) -> torch.Tensor:
+    """A batch of products of one shape: out[i] = xs[i] ws[i]^T with xs [n, M, K], ws [n, N, K] (contiguous).  float32:
+    multiply-adds on the CUDA cores, every sum over k in ascending order; bfloat16: the library product."""
+    _dev(xs, ws)
+    _need(xs.dim() == 3 and ws.dim() == 3 and xs.is_contiguous() and ws.is_contiguous() and xs.dtype == ws.dtype
+          and xs.shape[0] == ws.shape[0] and xs.shape[2] == ws.shape[2], "gemm_members: xs [n, M, K], ws [n, N, K] of one element type")
+    n, m, k = xs.shape
+    if xs.dtype == torch.bfloat16:
+        _full_precision_sums()
+        return torch.bmm(xs, ws.transpose(1, 2))
+    out = torch.empty((n, m, ws.shape[1]), dtype=xs.dtype, device=xs.device)
+    _check(library().vx_gemm_nt_simt_batched(_ptr(xs), _ptr(ws), None, _ptr(out), m, ws.shape[1], k, k, k, ws.shape[1], n, m * k,
+                                             ws.shape[1] * k, m * ws.shape[1], dtype_code(xs.dtype), dtype_code(out.dtype), _stream()),
+           "gemm_members")
+    return out
+
+
+def _full_precision_sums() -> None:
+    """Sums of the library's bfloat16 products stay in float32."""
+    global _MATMUL_SET
+    if not _MATMUL_SET:
+        torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
+        _MATMUL_SET = True
 
 
 def gemm_bf16(a: torch.Tensor, w: torch.Tensor, bias=None, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
@@ -1438,10 +1599,7 @@ def gemm_bf16(a: torch.Tensor, w: torch.Tensor, bias=None, out_dtype: Optional[t
     if skinny_supported(a.shape[0], a.shape[1], a, w):
         return gemm_skinny(a, w, bias, out_dtype)
     # library product (cuBLAS through torch); reductions stay in float32
-    global _MATMUL_SET
-    if not _MATMUL_SET:
-        torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
-        _MATMUL_SET = True
+    _full_precision_sums()
     if out_dtype == torch.float32 or bias is not None:
         out = torch.mm(a, w.t(), out_dtype=torch.float32)
     else:

@@ -15,7 +15,8 @@
 //   slot_mapping[token] = page * S + offset, pools laid out [page, Hk, S, D] and [page, Hk, S, Dv].
 // A token whose slot is negative writes nothing.  Without a slot mapping (a layer
 // that reads another layer's cache, or a caller that encodes positions itself)
-// nothing is written to the pools and the keys are normed and rotated in place.
+// nothing is written to the pools and the keys are normed and rotated in place; such a row
+// may hold queries only (Hk = 0).
 #include "common.cuh"
 
 #define ROPE_WARPS 4
@@ -495,7 +496,7 @@ extern "C" int vx_qk_norm_rope_kv_shared(void* qkv, int row_stride, const float*
     if (tokens <= 0) return VX_OK;
     if (Dv <= 0) Dv = D;
     if (Hv <= 0) Hv = Hk;
-    if (H <= 0 || Hk <= 0 || D <= 0 || S <= 0 || D > ROPE_MAX_D || Dv > ROPE_MAX_D) return VX_ERR_SHAPE;
+    if (H <= 0 || Hk < 0 || (Hk == 0 && (slot_mapping || Hv)) || D <= 0 || S <= 0 || D > ROPE_MAX_D || Dv > ROPE_MAX_D) return VX_ERR_SHAPE;
     if (rot_dim < 0 || rot_dim > D || (rot_dim & 1)) return VX_ERR_SHAPE;
     if (row_stride < (H + Hk) * D + Hv * Dv) return VX_ERR_SHAPE;
     if (slot_mapping && (!k_pool || !v_pool)) return VX_ERR_SHAPE;

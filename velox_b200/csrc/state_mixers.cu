@@ -2,7 +2,9 @@
 // sublayers run side by side:
 //   linear_attention_walk   S_p = a_p (.) S_(p-1) + k_p v_p^T, o_p = S_p^T q_p with the decay a number per
 //                           head or a number per key channel and position; q and k optionally rotated by
-//                           position and multiplied by numbers on the way in
+//                           position and multiplied by numbers on the way in.  With a bonus u [H, D] the output
+//                           comes before the update and the token's own contribution is weighed by u instead:
+//                           o_p = (S_(p-1) + diag(u) k_p v_p^T)^T q_p
 //   stretch_log_decay, stretch_scan   a long portion cut into stretches that are walked side by side
 //   head_norm_gate          every head's output divided by its root mean square (optionally times a
 //                           weight shared by the heads), times silu or sigmoid of a gate projection
@@ -32,7 +34,9 @@ __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - l
 // staged LW_CHUNK at a time in shared memory, in float32, rows padded to 16 R with q = k = 0: q and k as the projection left
 // them, turned by position * inv_freq[i] on the first rot_dim channels (pairs (i, i + rot_dim/2), or (2i, 2i + 1) when
 // `interleaved`), then times q_mul / k_mul.  The decay of channel d at token t is decay[h] (`gate` null), or
-// exp(gate_mul * log_sigmoid(gate[t, h D + d])): sigmoid(z)^(gate_mul), formed through the logarithm.  A token's output
+// exp(gate_mul * log_sigmoid(gate[t, h D + d])): sigmoid(z)^(gate_mul), formed through the logarithm, or with
+// `gate_is_log` exp(gate[t, h D + d]).  With BONUS a thread also sums q_d u_d k_d over its rows and adds that sum times v to
+// its columns, while S enters the outputs as the token found it.  A token's output
 // column is summed over a thread's rows in order, then over the 4 row groups of a warp by two exchanges, then over the warps
 // in warp order (through shared memory, once a chunk): an order fixed by D alone.
 __device__ __forceinline__ void lw_load8(const float* p, float (&v)[8]) {
@@ -50,14 +54,20 @@ __device__ __forceinline__ void lw_load8(const bf16* p, float (&v)[8]) {
     }
 }
 
-template <typename T, int R, bool GATED>
+// The logarithm of a channel's decay from its gate.
+__device__ __forceinline__ float lw_log_decay(float g, float gate_mul, int gate_is_log) {
+    return gate_is_log ? g : gate_mul * log_sigmoid(g);
+}
+
+template <typename T, int R, bool GATED, bool BONUS>
 __global__ void __launch_bounds__(LW_THREADS, 4)
 linear_attention_walk_kernel(const T* __restrict__ x, int ldx, int q_col, int k_col, int v_col,
                              const float* __restrict__ decay, const float* __restrict__ gate, int ldg, float gate_mul,
                              const float* __restrict__ inv_freq, int rot_dim, int interleaved,
                              const int* __restrict__ positions, float q_mul, float k_mul, float* __restrict__ state,
                              const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots,
-                             float* __restrict__ out, int H, int D, int Dv, int fresh) {
+                             float* __restrict__ out, int H, int D, int Dv, int fresh, const float* __restrict__ bonus,
+                             int gate_is_log) {
     extern __shared__ __align__(16) float smem[];
     constexpr int DP = LW_GROUPS * R;
     float* q_s = smem;                            // [LW_CHUNK][DP]
@@ -72,6 +82,11 @@ linear_attention_walk_kernel(const T* __restrict__ x, int ldx, int q_col, int k_
     const int half = rot_dim >> 1;
     const bool by_eights = (D & 7) == 0 && ((size_t)ldx * sizeof(T) & 15) == 0 && (((uintptr_t)(x + q_col)) & 15) == 0 &&
                            (((uintptr_t)(x + k_col)) & 15) == 0 && (!GATED || ((ldg & 3) == 0 && (((uintptr_t)gate) & 15) == 0));
+    float ub[R];
+    if (BONUS) {
+#pragma unroll
+        for (int r = 0; r < R; ++r) ub[r] = row0 + r < D ? bonus[(size_t)h * D + row0 + r] : 0.f;
+    }
     pdl_wait();
     pdl_trigger();
     const int t0 = cu_seqlens[seq], t1 = cu_seqlens[seq + 1];
@@ -94,7 +109,7 @@ linear_attention_walk_kernel(const T* __restrict__ x, int ldx, int q_col, int k_
                 const bool turned = inv_freq && d < rot_dim;
                 qv = to_f32(row[q_col]) * (turned ? 1.f : q_mul);
                 kv = to_f32(row[k_col]) * (turned ? 1.f : k_mul);
-                if (GATED) av = expf(gate_mul * log_sigmoid(gate[(size_t)(tb + tt) * ldg + (size_t)h * D + d]));
+                if (GATED) av = expf(lw_log_decay(gate[(size_t)(tb + tt) * ldg + (size_t)h * D + d], gate_mul, gate_is_log));
             }
             q_s[i] = qv;
             k_s[i] = kv;
@@ -123,7 +138,7 @@ linear_attention_walk_kernel(const T* __restrict__ x, int ldx, int q_col, int k_
                 if (GATED) {
                     lw_load8(gate + (size_t)(tb + tt) * ldg + (size_t)h * D + d, av);
 #pragma unroll
-                    for (int e = 0; e < 8; ++e) av[e] = expf(gate_mul * log_sigmoid(av[e]));
+                    for (int e = 0; e < 8; ++e) av[e] = expf(lw_log_decay(av[e], gate_mul, gate_is_log));
                 }
             }
             const int i = tt * DP + d;
@@ -169,6 +184,7 @@ linear_attention_walk_kernel(const T* __restrict__ x, int ldx, int q_col, int k_
             const float4 v4 = *reinterpret_cast<const float4*>(v_s + tt * LW_COLS + cg * LW_CC);
             const float v[LW_CC] = {v4.x, v4.y, v4.z, v4.w};
             float o[LW_CC] = {0.f, 0.f, 0.f, 0.f};
+            float own = 0.f;   // (BONUS) sum over this thread's rows of q u k
 #pragma unroll
             for (int r4 = 0; r4 < R; r4 += 4) {
                 const float4 k4 = *reinterpret_cast<const float4*>(k_s + tt * DP + row0 + r4);
@@ -177,12 +193,19 @@ linear_attention_walk_kernel(const T* __restrict__ x, int ldx, int q_col, int k_
                 if (GATED) a4 = *reinterpret_cast<const float4*>(a_s + tt * DP + row0 + r4);
                 const float kk[4] = {k4.x, k4.y, k4.z, k4.w}, qq[4] = {q4.x, q4.y, q4.z, q4.w}, aa[4] = {a4.x, a4.y, a4.z, a4.w};
 #pragma unroll
-                for (int r = 0; r < 4; ++r)
+                for (int r = 0; r < 4; ++r) {
+                    if (BONUS) own = fmaf(qq[r] * kk[r], ub[r4 + r], own);
 #pragma unroll
                     for (int c = 0; c < LW_CC; ++c) {
+                        if (BONUS) o[c] = fmaf(S[r4 + r][c], qq[r], o[c]);
                         S[r4 + r][c] = fmaf(aa[r], S[r4 + r][c], kk[r] * v[c]);
-                        o[c] = fmaf(S[r4 + r][c], qq[r], o[c]);
+                        if (!BONUS) o[c] = fmaf(S[r4 + r][c], qq[r], o[c]);
                     }
+                }
+            }
+            if (BONUS) {
+#pragma unroll
+                for (int c = 0; c < LW_CC; ++c) o[c] = fmaf(own, v[c], o[c]);
             }
             if (out) {
                 // over the warp's 4 row groups: the upper pair keeps columns 2, 3 and the lower pair 0, 1, then odd groups keep
@@ -217,19 +240,20 @@ static int launch_linear_attention_walk(const T* x, int ldx, int q_col, int k_co
                                         const float* gate, int ldg, float gate_mul, const float* inv_freq, int rot_dim,
                                         int interleaved, const int* positions, float q_mul, float k_mul, float* state,
                                         const int* cu_seqlens, const int* state_slots, float* out, int seqs, int H, int D,
-                                        int Dv, int fresh, cudaStream_t stream) {
+                                        int Dv, int fresh, const float* bonus, int gate_is_log, cudaStream_t stream) {
     dim3 grid((Dv + LW_COLS - 1) / LW_COLS, H, seqs);
-    static bool configured[8][VX_MAX_DEVICES];
-#define LW_GO(R_, G_, SLOT)                                                                                                \
+    static bool configured[12][VX_MAX_DEVICES];
+#define LW_GO(R_, G_, B_, SLOT)                                                                                            \
     do {                                                                                                                   \
-        if (int rc = vx_configure_smem(linear_attention_walk_kernel<T, R_, G_>, LW_MAX_SMEM, configured[SLOT])) return rc; \
-        VX_LAUNCH_K(VX_K_ATTENTION, (linear_attention_walk_kernel<T, R_, G_>), grid, LW_THREADS, LW_SMEM(LW_GROUPS * R_, G_), \
+        if (int rc = vx_configure_smem(linear_attention_walk_kernel<T, R_, G_, B_>, LW_MAX_SMEM, configured[SLOT])) return rc; \
+        VX_LAUNCH_K(VX_K_ATTENTION, (linear_attention_walk_kernel<T, R_, G_, B_>), grid, LW_THREADS, LW_SMEM(LW_GROUPS * R_, G_), \
                     stream, x, ldx, q_col, k_col, v_col, decay, gate, ldg, gate_mul, inv_freq, rot_dim, interleaved,       \
-                    positions, q_mul, k_mul, state, cu_seqlens, state_slots, out, H, D, Dv, fresh);                        \
+                    positions, q_mul, k_mul, state, cu_seqlens, state_slots, out, H, D, Dv, fresh, bonus, gate_is_log);     \
     } while (0)
 #define LW_GO_R(R_, SLOT)                                                                                                  \
     do {                                                                                                                   \
-        if (gate) LW_GO(R_, true, 2 * SLOT); else LW_GO(R_, false, 2 * SLOT + 1);                                          \
+        if (bonus) LW_GO(R_, true, true, 3 * SLOT + 2);                                                                    \
+        else if (gate) LW_GO(R_, true, false, 3 * SLOT); else LW_GO(R_, false, false, 3 * SLOT + 1);                       \
     } while (0)
     if (D <= 64) LW_GO_R(4, 0);
     else if (D <= 128) LW_GO_R(8, 1);
@@ -241,29 +265,43 @@ static int launch_linear_attention_walk(const T* x, int ldx, int q_col, int k_co
     return VX_OK;
 }
 
-// x: rows with q, k [H, D] and v [H, Dv] at the given columns.  decay [H] or gate [tokens, ldg] (float32; one
-// of the two).  state float32 [slot, H, D, Dv], read (from zero instead with `fresh`) and written back.  out float32
-// [tokens, H * Dv], or null where only the states are wanted.
-extern "C" int vx_linear_attention_walk_parts(const void* x, int ldx, int q_col, int k_col, int v_col, const float* decay,
+// x: rows with q, k [H, D] and v [H, Dv] at the given columns (a column may lie in another matrix of the same row length
+// after the first: columns are offsets from x).  decay [H] or gate [tokens, ldg] (float32; one of the two; with
+// `gate_is_log` the gate is the decay's logarithm).  `bonus` float32 [H, D] (with a gate only).  state float32 [slot, H, D, Dv],
+// read (from zero instead with `fresh`) and written back.  out float32 [tokens, H * Dv], or null where only the states are
+// wanted.
+extern "C" int vx_linear_attention_walk_bonus(const void* x, int ldx, int q_col, int k_col, int v_col, const float* decay,
                                               const float* gate, int ldg, float gate_mul, const float* inv_freq, int rot_dim,
                                               int interleaved, const int* positions, float q_mul, float k_mul, float* state,
                                               const int* cu_seqlens, const int* state_slots, float* out, int seqs, int H,
-                                              int D, int Dv, int fresh, int dtype, cudaStream_t stream) {
+                                              int D, int Dv, int fresh, const float* bonus, int gate_is_log, int dtype,
+                                              cudaStream_t stream) {
     if (seqs <= 0) return VX_OK;
     if (H <= 0 || D <= 0 || Dv <= 0 || D > 256 || q_col < 0 || k_col < 0 || v_col < 0) return VX_ERR_SHAPE;
     if ((decay == nullptr) == (gate == nullptr)) return VX_ERR_SHAPE;
+    if (bonus && !gate) return VX_ERR_SHAPE;
     if (gate && ldg < H * D) return VX_ERR_SHAPE;
     if (rot_dim < 0 || rot_dim > D || (rot_dim & 1) || (inv_freq && rot_dim > 0 && !positions)) return VX_ERR_SHAPE;
     if (seqs > 65535 || H > 65535) return VX_ERR_LIMIT;
     if (dtype == VX_F32)
         return launch_linear_attention_walk<float>((const float*)x, ldx, q_col, k_col, v_col, decay, gate, ldg, gate_mul,
                                                    inv_freq, rot_dim, interleaved, positions, q_mul, k_mul, state,
-                                                   cu_seqlens, state_slots, out, seqs, H, D, Dv, fresh, stream);
+                                                   cu_seqlens, state_slots, out, seqs, H, D, Dv, fresh, bonus, gate_is_log, stream);
     if (dtype == VX_BF16)
         return launch_linear_attention_walk<bf16>((const bf16*)x, ldx, q_col, k_col, v_col, decay, gate, ldg, gate_mul,
                                                   inv_freq, rot_dim, interleaved, positions, q_mul, k_mul, state,
-                                                  cu_seqlens, state_slots, out, seqs, H, D, Dv, fresh, stream);
+                                                  cu_seqlens, state_slots, out, seqs, H, D, Dv, fresh, bonus, gate_is_log, stream);
     return VX_ERR_DTYPE;
+}
+
+extern "C" int vx_linear_attention_walk_parts(const void* x, int ldx, int q_col, int k_col, int v_col, const float* decay,
+                                              const float* gate, int ldg, float gate_mul, const float* inv_freq, int rot_dim,
+                                              int interleaved, const int* positions, float q_mul, float k_mul, float* state,
+                                              const int* cu_seqlens, const int* state_slots, float* out, int seqs, int H,
+                                              int D, int Dv, int fresh, int dtype, cudaStream_t stream) {
+    return vx_linear_attention_walk_bonus(x, ldx, q_col, k_col, v_col, decay, gate, ldg, gate_mul, inv_freq, rot_dim, interleaved,
+                                          positions, q_mul, k_mul, state, cu_seqlens, state_slots, out, seqs, H, D, Dv, fresh,
+                                          nullptr, 0, dtype, stream);
 }
 
 extern "C" int vx_linear_attention_walk(const void* x, int ldx, int q_col, int k_col, int v_col, const float* decay,
@@ -281,17 +319,18 @@ extern "C" int vx_linear_attention_walk(const void* x, int ldx, int q_col, int k
 // state, `fresh`) and the decay over the whole stretch A_c (per head, or per key channel), the state at a stretch's start
 // follows from the one before it: S_start[c + 1] = diag(A_c) S_start[c] + S_loc[c]; a second walk of every stretch from its
 // start state gives the outputs.  Two kernels around the walks:
-//   stretch_log_decay  log A_c [stretch, H D] = sum over the stretch's tokens of gate_mul * log_sigmoid(gate)
+//   stretch_log_decay  log A_c [stretch, H D] = sum over the stretch's tokens of gate_mul * log_sigmoid(gate) (of the gate
+//                      itself with `gate_is_log`)
 //   stretch_scan       per request, in the order of its stretches: parts[c] (holding S_loc[c]) takes S_start[c]; the state
 //                      slot takes the state after the last stretch.  One thread per state element.
 __global__ void stretch_log_decay_kernel(const float* __restrict__ gate, int ldg, float gate_mul,
-                                         const int* __restrict__ cu_stretch, float* __restrict__ log_a, int HD) {
+                                         const int* __restrict__ cu_stretch, float* __restrict__ log_a, int HD, int gate_is_log) {
     pdl_wait();
     pdl_trigger();
     const int c = blockIdx.y, i = blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= HD) return;
     float sum = 0.f;
-    for (int t = cu_stretch[c]; t < cu_stretch[c + 1]; ++t) sum += gate_mul * log_sigmoid(gate[(size_t)t * ldg + i]);
+    for (int t = cu_stretch[c]; t < cu_stretch[c + 1]; ++t) sum += lw_log_decay(gate[(size_t)t * ldg + i], gate_mul, gate_is_log);
     log_a[(size_t)c * HD + i] = sum;
 }
 
@@ -329,15 +368,20 @@ __global__ void stretch_scan_kernel(float* __restrict__ parts, float* __restrict
     *st = S;
 }
 
-extern "C" int vx_stretch_log_decay(const float* gate, int ldg, float gate_mul, const int* cu_stretch, float* log_a,
-                                    int stretches, int HD, cudaStream_t stream) {
+extern "C" int vx_stretch_log_decay_form(const float* gate, int ldg, float gate_mul, const int* cu_stretch, float* log_a,
+                                         int stretches, int HD, int gate_is_log, cudaStream_t stream) {
     if (stretches <= 0) return VX_OK;
     if (HD <= 0 || ldg < HD) return VX_ERR_SHAPE;
     if (stretches > 65535) return VX_ERR_LIMIT;
     VX_LAUNCH_K(VX_K_ELEMENTWISE, stretch_log_decay_kernel, dim3((HD + 127) / 128, stretches), 128, 0, stream, gate, ldg,
-                gate_mul, cu_stretch, log_a, HD);
+                gate_mul, cu_stretch, log_a, HD, gate_is_log);
     VX_LAUNCH_CHECK();
     return VX_OK;
+}
+
+extern "C" int vx_stretch_log_decay(const float* gate, int ldg, float gate_mul, const int* cu_stretch, float* log_a,
+                                    int stretches, int HD, cudaStream_t stream) {
+    return vx_stretch_log_decay_form(gate, ldg, gate_mul, cu_stretch, log_a, stretches, HD, 0, stream);
 }
 
 // parts float32 [stretch, H, D, Dv]; log_a [stretch, H D] or null with decay [H]; the stretches of request i are
@@ -355,11 +399,12 @@ extern "C" int vx_stretch_scan(float* parts, float* state, const float* log_a, c
     return VX_OK;
 }
 
-// One warp per (token, head): out = o / sqrt(mean(o^2) + eps) (* w[d]) * act(g), act = sigmoid (0) or silu (1).
-template <typename T>
-__global__ void head_norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ g, int ldg,
-                                      const float* __restrict__ w, T* __restrict__ out, int rows, int H, int Dv, float eps,
-                                      int gate_act) {
+// One warp per (token, head): out = o / sqrt(mean(o^2) + eps) (* w[h w_head + d]) * act(g), act = sigmoid (0) or silu (1);
+// w_head = 0: one weight that the heads share, Dv: a weight per head.
+template <typename TG, typename T>
+__global__ void head_norm_gate_kernel(const float* __restrict__ o, const TG* __restrict__ g, int ldg,
+                                      const float* __restrict__ w, int w_head, T* __restrict__ out, int rows, int H, int Dv,
+                                      float eps, int gate_act) {
     pdl_wait();
     pdl_trigger();
     const int unit = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -370,32 +415,40 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const T* __re
     for (int d = lane; d < Dv; d += 32) { const float v = src[d]; ss += v * v; }
     ss = warp_sum(ss);
     const float rstd = rsqrtf(ss / (float)Dv + eps);
-    const T* gr = g + (size_t)t * ldg + (size_t)h * Dv;
+    const TG* gr = g + (size_t)t * ldg + (size_t)h * Dv;
     T* dst = out + ((size_t)t * H + h) * Dv;
     for (int d = lane; d < Dv; d += 32) {
         const float z = to_f32(gr[d]);
         const float sg = 1.f / (1.f + expf(-z));
         float v = src[d] * rstd;
-        if (w) v *= w[d];
+        if (w) v *= w[(size_t)h * w_head + d];
         dst[d] = from_f32<T>(v * (gate_act ? z * sg : sg));
     }
 }
 
-extern "C" int vx_head_norm_gate(const float* o, const void* g, int ldg, const float* w, void* out, int rows, int H,
-                                 int Dv, float eps, int gate_act, int dtype, cudaStream_t stream) {
+// g_dtype: the gate's element type, dtype: the output's (float32 gates with bfloat16 outputs are taken too).
+extern "C" int vx_head_norm_gate_heads(const float* o, const void* g, int ldg, const float* w, int w_per_head, void* out, int rows,
+                                       int H, int Dv, float eps, int gate_act, int g_dtype, int dtype, cudaStream_t stream) {
     if (rows <= 0) return VX_OK;
     if (H <= 0 || Dv <= 0 || ldg < H * Dv) return VX_ERR_SHAPE;
-    const int warps = 4;
+    const int warps = 4, w_head = w_per_head ? Dv : 0;
     const long long blocks = ((long long)rows * H + warps - 1) / warps;
     if (blocks > 0x7fffffffLL) return VX_ERR_LIMIT;
-    if (dtype == VX_F32)
-        VX_LAUNCH_K(VX_K_ELEMENTWISE, (head_norm_gate_kernel<float>), (unsigned)blocks, warps * 32, 0, stream, o, (const float*)g, ldg, w, (float*)out, rows, H, Dv, eps, gate_act);
-    else if (dtype == VX_BF16)
-        VX_LAUNCH_K(VX_K_ELEMENTWISE, (head_norm_gate_kernel<bf16>), (unsigned)blocks, warps * 32, 0, stream, o, (const bf16*)g, ldg, w, (bf16*)out, rows, H, Dv, eps, gate_act);
+    if (dtype == VX_F32 && g_dtype == VX_F32)
+        VX_LAUNCH_K(VX_K_ELEMENTWISE, (head_norm_gate_kernel<float, float>), (unsigned)blocks, warps * 32, 0, stream, o, (const float*)g, ldg, w, w_head, (float*)out, rows, H, Dv, eps, gate_act);
+    else if (dtype == VX_BF16 && g_dtype == VX_BF16)
+        VX_LAUNCH_K(VX_K_ELEMENTWISE, (head_norm_gate_kernel<bf16, bf16>), (unsigned)blocks, warps * 32, 0, stream, o, (const bf16*)g, ldg, w, w_head, (bf16*)out, rows, H, Dv, eps, gate_act);
+    else if (dtype == VX_BF16 && g_dtype == VX_F32)
+        VX_LAUNCH_K(VX_K_ELEMENTWISE, (head_norm_gate_kernel<float, bf16>), (unsigned)blocks, warps * 32, 0, stream, o, (const float*)g, ldg, w, w_head, (bf16*)out, rows, H, Dv, eps, gate_act);
     else
         return VX_ERR_DTYPE;
     VX_LAUNCH_CHECK();
     return VX_OK;
+}
+
+extern "C" int vx_head_norm_gate(const float* o, const void* g, int ldg, const float* w, void* out, int rows, int H,
+                                 int Dv, float eps, int gate_act, int dtype, cudaStream_t stream) {
+    return vx_head_norm_gate_heads(o, g, ldg, w, 0, out, rows, H, Dv, eps, gate_act, dtype, dtype, stream);
 }
 
 // One block per token.  down [tokens, ldd]: C latent channels, then R channels of the key part that all heads

@@ -100,11 +100,10 @@ class DecoderModel:
     # An embedding that keeps something per request has one more place, after the last
     # of the running order.
     def cache_specs(self) -> list:
-        """Per place of the running order: the mixer's cache need, or None for a
-        place without a cache of its own (none at all, or another's); then the
-        embedding's need, if it has one."""
-        specs = [None if self.plan.layers[i].cache_of is not None or self.blocks[i].mixer is None
-                 else self.blocks[i].mixer.cache_spec() for i in self.order]
+        """Per place of the running order: the block's cache need (its mixer's, unless the
+        block keeps more), or None for a place without a cache of its own (none at all, or
+        another's); then the embedding's need, if it has one."""
+        specs = [self.blocks[i].cache_spec(own=self.plan.layers[i].cache_of is None) for i in self.order]
         return specs + ([self.embedding.cache_spec()] if self._embedding_keeps_state() else [])
 
     def _embedding_keeps_state(self) -> bool:

@@ -36,6 +36,12 @@ And two for designs that bound their scores and rotate neighbours: `score_softca
 c tanh(s / c) before the softmax) and a rotary position whose `layout` is "interleaved" (channel 2i paired with
 2i + 1; the q/k kernel takes the layout as a flag).  `weights_32bit` asks for the kernels that keep the softmax weights
 in 32 bits (two bfloat16 halves on the tensor cores) also where nothing else of the layer needs them.
+
+And three for designs that cut the sequence and share caches: `chunk` C > 0 (position i sees j <= i only if
+floor(i / C) = floor(j / C)); `sink_value` (a sink whose score is this number for every head, without a tensor; 0 adds one to
+the denominator); `own_kv=False` (the layer has no keys and values of its own: its queries read the cache of the layer that
+its plan names with `cache_of`).  `reader_chunks` lists the chunks of the layers that read this one's cache, which keeps
+what the longest of them still sees.
 """
 from __future__ import annotations
 
@@ -75,8 +81,17 @@ class PagedAttention(Mixer):
                  names: Sequence[str] = ("q_proj.weight", "k_proj.weight", "v_proj.weight", "o_proj.weight"),
                  norm_names: Sequence[str] = ("q_norm.weight", "k_norm.weight"), sink: bool = False,
                  output_gate: bool = False, sink_name: str = "sink", gate_name: str = "g", score_softcap: float = 0.0,
-                 weights_32bit: bool = False):
+                 weights_32bit: bool = False, chunk: int = 0, sink_value: Optional[float] = None, own_kv: bool = True,
+                 reader_chunks: Sequence[int] = ()):
         super().__init__(prefix)
+        self.chunk, self.own_kv, self.reader_chunks = int(chunk), bool(own_kv), tuple(int(c) for c in reader_chunks)
+        self.sink_value = None if sink_value is None else float(sink_value)
+        if self.chunk < 0 or (self.chunk and keep_first):
+            raise ValueError("%schunk must not be negative and does not go with kept first positions" % prefix)
+        if self.reader_chunks and window:
+            raise ValueError("%sreader_chunks goes with layers that cut the sequence into chunks, not with a window" % prefix)
+        if sink and sink_value is not None:
+            raise ValueError("%sa learned sink or a fixed one, not both" % prefix)
         self.softcap = float(score_softcap)
         self.weights_32bit = bool(weights_32bit)
         if self.softcap < 0:
@@ -111,6 +126,8 @@ class PagedAttention(Mixer):
     # -- weights -------------------------------------------------------------
     def _proj_rows(self):
         d = self.head_dim
+        if not self.own_kv:
+            return {"q_proj": self.num_heads * d}
         return {"q_proj": self.num_heads * d, "k_proj": self.num_kv_heads * d, "v_proj": self.num_kv_heads * self.v_head_dim}
 
     def _w(self, name: str) -> str:
@@ -120,15 +137,15 @@ class PagedAttention(Mixer):
     def extended(self) -> bool:
         """True if the layer uses what only the kernels for biased, unequal or kept-first attention know."""
         return (self.v_head_dim != self.head_dim or self.keep_first > 0 or self.bias_exponent > 0 or self.sink
-                or self.output_gate or self.softcap > 0 or self.weights_32bit)
+                or self.output_gate or self.softcap > 0 or self.weights_32bit or self.chunk > 0
+                or self.sink_value is not None or not self.own_kv)
 
     @property
     def gate_col(self) -> int:
         """The column of head 0's gate in a row of the fused projection, or -1."""
         if not self.output_gate:
             return -1
-        return (self.num_heads + self.num_kv_heads) * self.head_dim + self.num_kv_heads * self.v_head_dim
-
+        return sum(self._proj_rows().values())
 
     def tensor_specs(self) -> List[TensorSpec]:
         p, specs = self.prefix, []
@@ -141,7 +158,8 @@ class PagedAttention(Mixer):
             specs.append(TensorSpec(p + "o_proj.bias", (self.hidden_size,), "bias"))
         if self.qk_norm:
             specs.append(TensorSpec(self.norm_names[0], (self.head_dim,), "norm"))
-            specs.append(TensorSpec(self.norm_names[1], (self.head_dim,), "norm"))
+            if self.own_kv:
+                specs.append(TensorSpec(self.norm_names[1], (self.head_dim,), "norm"))
         if self.sink:
             specs.append(TensorSpec(self.sink_name, (self.num_heads,), "bias"))
         if self.output_gate:
@@ -156,8 +174,8 @@ class PagedAttention(Mixer):
     def bind(self, tensors: Dict[str, torch.Tensor], runtime: Runtime) -> None:
         super().bind(tensors, runtime)
         p = self.prefix
-        mats = [tensors[self._w(n)] for n in ("q_proj", "k_proj", "v_proj")]
-        biases = [tensors[p + n + ".bias"] for n in ("q_proj", "k_proj", "v_proj")] if self.bias else None
+        mats = [tensors[self._w(n)] for n in self._proj_rows()]
+        biases = [tensors[p + n + ".bias"] for n in self._proj_rows()] if self.bias else None
         if self.output_gate:
             # the gates' rows, then zero rows up to a multiple of 8 (rows of the projection stay 16-byte aligned)
             g = tensors[self.gate_name]
@@ -171,9 +189,12 @@ class PagedAttention(Mixer):
         self.qkv = Linear(w, b)
         if self.sink:
             self.sinks = tensors[self.sink_name].to(torch.float32).contiguous()
+        elif self.sink_value is not None:
+            self.sinks = torch.full((self.num_heads,), self.sink_value, dtype=torch.float32, device=runtime.device)
         self.out = Linear(tensors[self._w("o_proj")], tensors[p + "o_proj.bias"] if self.bias else None)
         if self.qk_norm:
-            self.q_norm_weight, self.k_norm_weight = tensors[self.norm_names[0]], tensors[self.norm_names[1]]
+            self.q_norm_weight = tensors[self.norm_names[0]]
+            self.k_norm_weight = tensors[self.norm_names[1]] if self.own_kv else None
         if self.position is not None:
             self.position.bind(tensors, runtime)
 
@@ -181,8 +202,13 @@ class PagedAttention(Mixer):
     def cache_spec(self):
         if not self.extended:
             return PagedKV(self.num_kv_heads, self.head_dim, self.window)
-        return PagedKV(self.num_kv_heads, self.head_dim, self.window,
-                       self.v_head_dim if self.v_head_dim != self.head_dim else 0, self.keep_first if self.window else 0)
+        # what the layer and every layer that reads its cache still see: one chunk where all agree, else the longest as a
+        # window (a chunk's first position is never further back), everything if one of them sees everything
+        sizes = {self.chunk, *self.reader_chunks}
+        chunk = self.chunk if len(sizes) == 1 else 0
+        window = self.window if len(sizes) == 1 or 0 in sizes else max(sizes)
+        return PagedKV(self.num_kv_heads, self.head_dim, window,
+                       self.v_head_dim if self.v_head_dim != self.head_dim else 0, self.keep_first if self.window else 0, 0, chunk)
 
     # -- step ----------------------------------------------------------------
     def forward(self, h: torch.Tensor, ctx, cache) -> torch.Tensor:
@@ -190,6 +216,10 @@ class PagedAttention(Mixer):
         group = ctx.groups[cache.group]
         qkv = self.qkv(h)
         slots = group.slot_mapping if cache.writes else None
+        if not self.own_kv:   # (a row holds queries only)
+            if slots is not None:
+                raise ValueError("%sa layer without keys and values of its own needs another layer's cache" % self.prefix)
+            Hk = 0
         if self.extended and not self.qk_norm and self.position is None:
             # plain projections: nothing to norm or rotate, the step's keys and values go into their pages as they are
             if slots is not None:
@@ -222,10 +252,10 @@ class PagedAttention(Mixer):
     def _attend_extended(self, qkv, ctx, cache, group) -> torch.Tensor:
         H, Hk, D = self.num_heads, self.num_kv_heads, self.head_dim
         more = dict(sinks=self.sinks, gate_col=self.gate_col)
-        capped = dict(more, softcap=self.softcap)
+        capped = dict(more, softcap=self.softcap, chunk=self.chunk)
         page = cache.k_pool.shape[2]
         if (not ctx.decode_only and ctx.max_new >= TC_PREFILL_MIN_TOKENS and self.keep_first == 0 and self.bias_exponent == 0
-                and self.softcap == 0 and self.v_head_dim == D and ops.prefill_attention_tc_supported(qkv.dtype, D, page, H // Hk)):
+                and self.softcap == 0 and self.chunk == 0 and self.v_head_dim == D and ops.prefill_attention_tc_supported(qkv.dtype, D, page, H // Hk)):
             # prompt portions of heads of 128 without a bias by distance: the tcgen05 kernel, with the probabilities in two
             # bfloat16 halves (this path's softmax weights are 32-bit), the sink and the gate in its epilogue
             return ops.paged_prefill_attention_tc(qkv, qkv.shape[1], cache.k_pool, cache.v_pool, group.block_table, ctx.cu_seqlens,
@@ -245,7 +275,7 @@ class PagedAttention(Mixer):
         return ops.paged_attention_generic(qkv, qkv.shape[1], cache.k_pool, cache.v_pool, group.block_table,
                                            ctx.seq_of_token, ctx.positions, self.scale, self.window, H, Hk, D,
                                            qkv.shape[0], v_head_dim=self.v_head_dim, keep_first=self.keep_first,
-                                           bias_exponent=self.bias_exponent, softcap=self.softcap, **more)
+                                           bias_exponent=self.bias_exponent, **capped)
 
     def _attend(self, qkv, ctx, cache, group) -> torch.Tensor:
         H, Hk, D = self.num_heads, self.num_kv_heads, self.head_dim

@@ -12,7 +12,8 @@ part knows which model it is in.
                                   CacheParts of several of these | None
                   forward(h, ctx, cache) -> y          h, y: [tokens, hidden]
     FeedForward   forward(h, ctx) -> y
-    Block         forward(residual, delta, ctx, cache) -> (residual, delta)
+    Block         cache_spec() -> its mixer's, or more
+                  forward(residual, delta, ctx, cache) -> (residual, delta)
                   built from a mixer, a feed-forward (or None) and norms by name
     Embedding     forward(ctx) -> float32 residual [tokens, hidden]
                   (forward(ctx, cache) if its cache_spec() asks for per-request state)
@@ -38,6 +39,7 @@ class TensorSpec:
       norm:          1 + N(0, 0.05); held in float32 (an exact widening)
       bias:          N(0, 0.02); held in float32
       matrix_f32:    N(0, 0.02); held in float32 whatever the engine's element type (a router)
+      share:         uniform in [0, 1); held in float32 (how far a channel is moved towards the token before it)
       mixing:        identity + N(0, 0.05), square; held in float32 (how the copies of a stream are mixed)
       int_table:     integers; held as int32
     A dimension of -1 is left open: the file's tensor decides it, and the part reads it off when it binds."""
@@ -58,13 +60,15 @@ class PagedKV:
     `window` positions are ever read, and older pages are given back, except those
     that hold one of the first `keep_first` positions (which every query still
     reads).  `v_head_dim` is the size of a value where it is not a key's (0: the same);
-    `num_v_heads` the number of value heads where several key heads share one (0: one per key head)."""
+    `num_v_heads` the number of value heads where several key heads share one (0: one per key head).  With a `chunk` a query
+    reads its own run of `chunk` positions only (runs counted from position 0), and pages before the run are given back."""
     num_kv_heads: int
     head_dim: int
     window: int = 0
     v_head_dim: int = 0
     keep_first: int = 0
     num_v_heads: int = 0
+    chunk: int = 0
 
     @property
     def value_dim(self) -> int:
@@ -95,10 +99,16 @@ class FixedState:
 
 @dataclass(frozen=True)
 class CacheParts:
-    """The needs of a mixer that is made of several: one spec (or None) per
-    member, in the members' order.  The mixer is handed a `LayerCache` whose
+    """The needs of a mixer that is made of several, or of a block that keeps something beside its mixer: one spec
+    (or None, or `CacheParts` again) per member, in the members' order.  The mixer is handed a `LayerCache` whose
     `parts` are the members' caches."""
     parts: Tuple[object, ...]
+
+
+@dataclass(frozen=True)
+class BorrowedCache:
+    """The need of a member that keeps nothing itself and reads the member in the same place among the parts of the
+    layer whose cache its own layer reads (`cache_of`)."""
 
 
 class Part:
@@ -198,6 +208,12 @@ class Block:
     def parts(self) -> List[Part]:
         out: List[Part] = [self.norms[n] for n in self.norm_names]
         return out + [p for p in (self.mixer, self.feed_forward) if p is not None]
+
+    def cache_spec(self, own: bool = True):
+        """What a place of the running order with this block keeps: the mixer's need, or None for a layer that reads
+        another's cache (`own` False).  A block that keeps something per request itself (the row before, say) asks for a
+        `CacheParts` of that and the mixer's need (`BorrowedCache` where the mixer reads another layer's)."""
+        return self.mixer.cache_spec() if own and self.mixer is not None else None
 
     def forward(self, residual, delta, ctx, cache):
         raise NotImplementedError

@@ -39,6 +39,13 @@ layer with a layer scale, x <- x + m ls (.) sublayer(norm(x)).  The update of on
 of the next are one kernel (`ops.stream_update`); the last update of a block travels as a `PendingStreams` to the next
 block of this kind, whose first norm it is fused with, or is applied by whoever reads the stream next.  The residual
 between such blocks is [tokens, n * hidden] float32; a `LayerNorm(streams=n)` reads the sum of the copies at the end.
+
+`TokenShiftBlock`: the pre-norm layer whose mixer reads a shifted input:
+    n = norm1(x);  h_t = n_t + (n_(t-1) - n_t) (.) shift;  x = x + mixer(h);  x = x + feed_forward(norm2(x))
+with n_(-1) = 0 (the last line falls away in a layer without a feed-forward).  The last n of a request is state of the
+block's place, beside what the mixer keeps.  Residual update, norm and shift are one kernel (`ops.shift_norm`).  A mixer
+that shifts its input again for each of its projections (`forward_mixed`, with the vectors `mixes` and a state of its own)
+has that done in the same kernel.
 """
 from __future__ import annotations
 
@@ -48,7 +55,7 @@ from typing import List, Optional, Tuple
 import torch
 
 from ..csrc import ops
-from .base import Block, Part, TensorSpec
+from .base import Block, BorrowedCache, CacheParts, FixedState, Part, TensorSpec
 
 
 @dataclass
@@ -275,3 +282,57 @@ class HyperConnectionBlock(Block):
             y = self.feed_forward.forward(h, ctx)
             pending = PendingStreams(y, n, link.mix, link.out, self.residual_mult, link.layer_scale)
         return residual, pending
+
+
+class TokenShift(Part):
+    """A block's vector of shares [hidden]: how far each channel of what its mixer reads is moved towards the token before."""
+    cuda_graph_safe = True
+
+    def __init__(self, prefix: str, hidden_size: int):
+        super().__init__(prefix)
+        self.hidden_size = int(hidden_size)
+        self.weight = None
+
+    def tensor_specs(self):
+        return [TensorSpec(self.prefix, (self.hidden_size,), "share")]
+
+    def bind(self, tensors, runtime):
+        super().bind(tensors, runtime)
+        self.weight = tensors[self.prefix].to(torch.float32).contiguous()
+
+
+class TokenShiftBlock(Block):
+    needs_feed_forward = False
+
+    def __init__(self, mixer, feed_forward, norms, hidden_size: int, shift_name: str):
+        self.norm_names = ("mixer",) + (("feed_forward",) if feed_forward is not None else ())
+        super().__init__(mixer, feed_forward, norms)
+        self.hidden_size = int(hidden_size)
+        n = self.norms["mixer"]
+        if not hasattr(n, "weight") or not hasattr(n, "eps") or hasattr(n, "streams"):
+            raise ValueError("TokenShiftBlock fuses its mixer's norm with the shift and takes an RMS norm; got %s" % type(n).__name__)
+        if not 0 < self.hidden_size <= ops.shift_norm_max_width(self.hidden_size):
+            raise ValueError("%s: a stream of width %d: the shift kernel takes up to %d" % (shift_name, self.hidden_size,
+                                                                                          ops.shift_norm_max_width(self.hidden_size)))
+        self.shift = TokenShift(shift_name, self.hidden_size)
+
+    def parts(self):
+        return super().parts() + [self.shift]
+
+    def cache_spec(self, own: bool = True):
+        return CacheParts((FixedState((self.hidden_size,), "float32"), self.mixer.cache_spec() if own else BorrowedCache()))
+
+    def forward(self, residual, delta, ctx, cache):
+        kept, mixer_cache = cache.parts
+        norm, dtype = self.norms["mixer"], self.mixer.runtime.dtype
+        args = (residual, delta, norm.weight, norm.eps, self.shift.weight, ctx, kept.state, dtype)
+        if hasattr(self.mixer, "forward_mixed"):
+            residual, mixed = ops.shift_norm(*args, mixes=self.mixer.mixes, mix_state=self.mixer.mix_state(mixer_cache))
+            y = self.mixer.forward_mixed(mixed, ctx, mixer_cache)
+        else:
+            residual, h = ops.shift_norm(*args)
+            y = self.mixer.forward(h, ctx, mixer_cache)
+        if self.feed_forward is None:
+            return residual, y
+        h = self.norms["feed_forward"].add_norm(residual, y)
+        return residual, self.feed_forward.forward(h, ctx)

@@ -35,6 +35,17 @@ from .plan import PartSpec
 from .registry import build_part
 
 
+def step_stretches(ctx):
+    """The step's rows cut into stretches that the recurrence walks side by side, from a portion of
+    `ops.STRETCH_MIN_TOKENS` rows on; made once a step and kept on its context."""
+    if ctx.max_new < ops.STRETCH_MIN_TOKENS or len(ctx.new_lens) != ctx.n_seqs:
+        return None
+    plan = getattr(ctx, "walk_stretches", None)
+    if plan is None:
+        plan = ctx.walk_stretches = ops.StretchPlan(ctx.new_lens, ctx.positions.device)
+    return plan
+
+
 class _LinearAttention(Mixer):
     cuda_graph_safe = True  # reads nothing of a step but device tensors and sizes fixed per graph
     KEYS = ("q", "k", "v", "g", "o", "norm")
@@ -81,14 +92,7 @@ class _LinearAttention(Mixer):
 
     @staticmethod
     def _stretches(ctx):
-        """The step's rows cut into stretches that the recurrence walks side by side, from a portion of
-        `ops.STRETCH_MIN_TOKENS` rows on; made once a step and kept on its context."""
-        if ctx.max_new < ops.STRETCH_MIN_TOKENS or len(ctx.new_lens) != ctx.n_seqs:
-            return None
-        plan = getattr(ctx, "walk_stretches", None)
-        if plan is None:
-            plan = ctx.walk_stretches = ops.StretchPlan(ctx.new_lens, ctx.positions.device)
-        return plan
+        return step_stretches(ctx)
 
     def _finish(self, o: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
         """o float32 [tokens, heads * vdim] -> normed, gated, projected."""

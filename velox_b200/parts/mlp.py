@@ -100,6 +100,13 @@ class DenseMLP(FeedForward):
         self.up, self.down = Linear(tensors[self.names[0]]), Linear(tensors[self.names[1]])
 
     def forward(self, h: torch.Tensor, ctx=None) -> torch.Tensor:
+        w = self.up.weight
+        if h.dtype == torch.bfloat16 and ops.skinny_supported(h.shape[0], h.shape[1], h, w):
+            # a decode step: W streamed once, the activation taken on the float32 sums
+            return self.down(ops.gemm_skinny(h, w, None, h.dtype, activation=self.activation))
+        if h.dtype == torch.bfloat16 and h.shape[0] >= FUSED_TCGEN05_MIN_ROWS and ops.tcgen05_supported(h, w):
+            # a prompt portion: the tcgen05 product with the same epilogue
+            return self.down(ops.gemm_tcgen05(h, w, None, activation=self.activation))
         u = self.up(h, torch.float32)
         return self.down(ops.act(u, self.activation, out_dtype=h.dtype))
 

@@ -6,10 +6,15 @@ down(act(gate(h)) * up(h)) without biases.
 A second way of routing, `scores="softmax_all"`: s = softmax(z) over ALL the router's outputs; the choice is made by
 s + correction (a stored vector that moves the choice and not the weights), restricted to the outputs of the
 `keep_groups` best of `groups` equal groups of neighbouring outputs (a group's score is its largest choice score);
-the weights are the chosen s times `route_scale`, not renormalised.  The router's last `identity` outputs are
+the weights are the chosen s times `route_scale`, not renormalised.  A third, `scores="sigmoid"`, is the second with
+s = sigmoid(z), output by output.  The router's last `identity` outputs are
 identity experts: they have no matrices and return the token itself (times the weight).  With `shared_gate_name`
 the shared feed-forward's output is multiplied by sigmoid(w . h), one number per token; w is a stored [1, hidden]
 matrix that rides as one more row of the router's matrix.
+
+With `gated=False` an expert is down(act(up(h))): two matrices, `names` = (up, down).  With `weight_input` an
+assignment's weight multiplies what its expert reads instead of what it returns, sum_e expert_e(w_e h): the first product
+is linear, so the kernels multiply its float32 sums before the activation.
 
 Nothing of a step comes back to the host: the router kernel leaves the assignments on the device, a plan
 kernel orders them by expert, and two grouped matrix products (gate and up with the activation on their
@@ -41,17 +46,23 @@ class RoutedExperts(FeedForward):
                  router_names: Sequence[str] = ("router", "router.b"), expert_prefix: str = "e%d.",
                  names: Sequence[str] = ("gate", "up", "down"), scores: str = "softmax_chosen",
                  correction_name: Optional[str] = None, groups: int = 1, keep_groups: int = 1, route_scale: float = 1.0,
-                 identity: int = 0, shared_gate_name: Optional[str] = None):
+                 identity: int = 0, shared_gate_name: Optional[str] = None, gated: bool = True, weight_input: bool = False):
         super().__init__(prefix)
+        self.gated, self.weight_input = bool(gated), bool(weight_input)
+        if len(names) != (3 if self.gated else 2):
+            raise ValueError("%san expert %s a gate has %d matrices, got the names %s"
+                             % (prefix, "with" if self.gated else "without", 3 if self.gated else 2, list(names)))
+        if self.weight_input and identity:
+            raise ValueError("%sidentity experts take their weight on the output" % prefix)
         self.hidden_size, self.experts, self.top = int(hidden_size), int(experts), int(top)
         self.intermediate_size = int(intermediate_size)
         self.identity, self.groups, self.keep_groups = int(identity), int(groups), int(keep_groups)
         self.outputs = self.experts + self.identity   # what the router chooses among
         self.scores, self.route_scale = scores, float(route_scale)
-        if scores not in ("softmax_chosen", "softmax_all"):
-            raise ValueError("%sscores %r is not one of softmax_chosen, softmax_all" % (prefix, scores))
+        if scores not in ops.MOE_SCORES:
+            raise ValueError("%sscores %r is not one of %s" % (prefix, scores, ", ".join(ops.MOE_SCORES)))
         if scores == "softmax_chosen" and (correction_name or self.groups != 1 or self.route_scale != 1.0):
-            raise ValueError("%sa correction, groups and a multiplier of the weights go with scores='softmax_all'" % prefix)
+            raise ValueError("%sa correction, groups and a multiplier of the weights go with scores over all outputs" % prefix)
         if self.experts <= 0 or self.identity < 0 or not 0 < self.top <= self.outputs:
             raise ValueError("%stop %d of %d experts and %d identity experts" % (prefix, self.top, self.experts, self.identity))
         if self.groups < 1 or self.outputs % self.groups or not 1 <= self.keep_groups <= self.groups \
@@ -80,8 +91,8 @@ class RoutedExperts(FeedForward):
             specs.append(TensorSpec(self.correction_name, (self.outputs,), "bias"))
         if self.shared_gate_name:
             specs.append(TensorSpec(self.shared_gate_name, (1, e), "matrix_f32"))
-        for gate, up, down in self.expert_names:
-            specs += [TensorSpec(gate, (i, e), "matrix"), TensorSpec(up, (i, e), "matrix"), TensorSpec(down, (e, i), "matrix")]
+        for *firsts, down in self.expert_names:
+            specs += [TensorSpec(n, (i, e), "matrix") for n in firsts] + [TensorSpec(down, (e, i), "matrix")]
         return specs + (self.shared.tensor_specs() if self.shared is not None else [])
 
     def ignored_tensors(self) -> List[str]:
@@ -95,17 +106,20 @@ class RoutedExperts(FeedForward):
             self.router = torch.cat([self.router, tensors[self.shared_gate_name].to(torch.float32).view(1, e)], 0).contiguous()
         self.bias = tensors[self.bias_name] if self.router_bias else None
         self.correction = tensors[self.correction_name].to(torch.float32).contiguous() if self.correction_name else None
-        self.tile = GATE_TILE if i % GATE_TILE == 0 else 0
-        self.gate_up = torch.empty((self.experts, 2 * i, e), dtype=runtime.dtype, device=runtime.device)
+        self.tile = GATE_TILE if self.gated and i % GATE_TILE == 0 else 0
+        self.gate_up = torch.empty((self.experts, (2 if self.gated else 1) * i, e), dtype=runtime.dtype, device=runtime.device)
         self.down = torch.empty((self.experts, e, i), dtype=runtime.dtype, device=runtime.device)
-        for x, (gate, up, down) in enumerate(self.expert_names):
-            g, u = tensors[gate], tensors[up]
+        for x, (*firsts, down) in enumerate(self.expert_names):
+            self.down[x] = tensors[down]
+            if not self.gated:
+                self.gate_up[x] = tensors[firsts[0]]
+                continue
+            g, u = (tensors[n] for n in firsts)
             if self.tile:
                 self.gate_up[x] = torch.stack([g.view(i // GATE_TILE, GATE_TILE, e), u.view(i // GATE_TILE, GATE_TILE, e)],
                                               1).reshape(2 * i, e)
             else:
                 self.gate_up[x, :i], self.gate_up[x, i:] = g, u
-            self.down[x] = tensors[down]
         if self.shared is not None:
             self.shared.bind(tensors, runtime)
 
@@ -117,22 +131,27 @@ class RoutedExperts(FeedForward):
 
     def forward(self, h: torch.Tensor, ctx=None) -> torch.Tensor:
         i, e = self.intermediate_size, self.hidden_size
-        if self.tile and ops.moe_tcgen05_supported(h, h.shape[0] * self.top, 2 * i, e) and i % 8 == 0 and e % 16 == 0:
+        n = self.gate_up.shape[1]
+        fused = dict(gated_activation=self.activation) if self.gated else dict(activation=self.activation)
+        if (self.tile or not self.gated) and ops.moe_tcgen05_supported(h, h.shape[0] * self.top, n, e) and i % 8 == 0 and e % 16 == 0:
             # a prompt portion: the tokens' rows are copied into expert order once, and both grouped products run on
             # the tcgen05 tensor cores over row tiles of 128 (operands by TMA, the activation on the accumulators)
             plan = self._route(h, ops.MOE_TCGEN05_TILE_ROWS)
-            a = ops.moe_gemm_tcgen05(ops.moe_gather_rows(h, plan), self.gate_up, plan, gated_activation=self.activation)
+            a = ops.moe_gemm_tcgen05(ops.moe_gather_rows(h, plan), self.gate_up, plan, row_scale=self._scale(plan), **fused)
             y = ops.moe_gemm_tcgen05(a, self.down, plan)
             shared = self.shared.forward(h, ctx) if self.shared is not None else None
-            return ops.moe_combine(y, plan, shared, h.dtype, h=h)
+            return ops.moe_combine(y, plan, shared, h.dtype, h=h, weighted=not self.weight_input)
         # (a decode step's few rows per expert: row tiles of 16; the second product reads rows of `inner` elements)
         rows = ops.moe_tile_rows(h, h.shape[0] * self.top) if i % 8 == 0 else ops.MOE_TILE_ROWS
         plan = self._route(h, rows)
-        if self.tile:
-            a = ops.moe_gemm(h, self.gate_up, plan, True, h.dtype, gated_activation=self.activation)
+        if self.tile or not self.gated:
+            a = ops.moe_gemm(h, self.gate_up, plan, True, h.dtype, row_scale=self._scale(plan), **fused)
         else:
             # an inner size that is no multiple of 8: all gates, then all ups; the activation by a kernel of its own
-            a = ops.gated_act(ops.moe_gemm(h, self.gate_up, plan, True, torch.float32), self.activation, 0, out_dtype=h.dtype)
+            a = ops.gated_act(ops.moe_gemm(h, self.gate_up, plan, True, torch.float32, row_scale=self._scale(plan)), self.activation, 0, out_dtype=h.dtype)
         y = ops.moe_gemm(a, self.down, plan, False, torch.float32)
         shared = self.shared.forward(h, ctx) if self.shared is not None else None
-        return ops.moe_combine(y, plan, shared, h.dtype, h=h)
+        return ops.moe_combine(y, plan, shared, h.dtype, h=h, weighted=not self.weight_input)
+
+    def _scale(self, plan):
+        return plan.weight.view(-1) if self.weight_input else None

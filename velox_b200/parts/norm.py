@@ -3,7 +3,8 @@
 The reference calls its tensor library's rms_norm with `rms_norm_eps`
 (src/paged/qwen3.rs:923-928, 933, 936); the weight multiplies, with no offset.
 With `one_plus` the stored tensor is the multiplier's offset from one: the multiplier is 1 + tensor
-(formed once in float32 when the weights are bound).
+(formed once in float32 when the weights are bound).  With `scalar` the stored tensor is one number without dimensions
+that multiplies every channel.
 
 `LayerNorm`: (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight, no bias; statistics in float32, the variance taken
 from the deviations.  With `streams` n > 1 the stream it reads is kept in n copies side by side
@@ -22,18 +23,21 @@ from .base import Norm, Runtime, TensorSpec
 class RMSNorm(Norm):
     cuda_graph_safe = True  # reads nothing of a step but device tensors and sizes fixed per graph
 
-    def __init__(self, prefix: str, size: int, eps: float, weight_name: str = "weight", one_plus: bool = False):
+    def __init__(self, prefix: str, size: int, eps: float, weight_name: str = "weight", one_plus: bool = False,
+                 scalar: bool = False):
         super().__init__(prefix)
-        self.size, self.eps, self.one_plus = int(size), float(eps), bool(one_plus)
+        self.size, self.eps, self.one_plus, self.scalar = int(size), float(eps), bool(one_plus), bool(scalar)
         self.weight_name = prefix + weight_name   # (a checkpoint may name the tensor by the prefix alone: "")
         self.weight: Optional[torch.Tensor] = None
 
     def tensor_specs(self) -> List[TensorSpec]:
-        return [TensorSpec(self.weight_name, (self.size,), "bias" if self.one_plus else "norm")]
+        return [TensorSpec(self.weight_name, () if self.scalar else (self.size,), "bias" if self.one_plus else "norm")]
 
     def bind(self, tensors: Dict[str, torch.Tensor], runtime: Runtime) -> None:
         super().bind(tensors, runtime)
         self.weight = tensors[self.weight_name]
+        if self.scalar:   # (the kernels read a multiplier per channel)
+            self.weight = self.weight.to(torch.float32).reshape(1).expand(self.size).contiguous()
         if self.one_plus:
             self.weight = (self.weight.to(torch.float32) + 1.0).contiguous()
 

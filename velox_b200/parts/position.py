@@ -17,6 +17,10 @@ positions: channel pairs that turn fewer than `slow` times in `original` positio
 d(t) = rot ln(original / (2 pi t)) / (2 ln theta) the two are blended linearly; cosines and sines are then multiplied by
 0.1 ln(factor) + 1 (`magnitude`, which the rotating kernels take as a parameter).
 
+With `scaling` (factor, low, high, original) the frequencies are stretched by wavelength instead: a pair whose
+wavelength 2 pi / f is longer than original / low has its frequency divided by `factor`, one shorter than original / high
+keeps it, and between the two the kept share grows linearly with original / wavelength; cosines and sines are as they are.
+
 `NoPosition`: nothing is applied.
 """
 from __future__ import annotations
@@ -38,10 +42,10 @@ class RotaryPosition(Position):
         super().__init__(prefix)
         self.scaling = dict(scaling) if scaling else None
         if self.scaling is not None:
-            missing = [k for k in ("factor", "original", "fast", "slow") if k not in self.scaling]
-            if missing or not float(self.scaling["factor"]) > 0 or not float(self.scaling["original"]) > 0 \
-                    or not float(self.scaling["fast"]) > 0 or not float(self.scaling["slow"]) > 0:
-                raise ValueError("rotation scaling needs positive factor, original, fast and slow; got %r" % (scaling,))
+            self.by_wavelength = "low" in self.scaling or "high" in self.scaling
+            keys = ("factor", "original") + (("low", "high") if self.by_wavelength else ("fast", "slow"))
+            if any(k not in self.scaling or not float(self.scaling[k]) > 0 for k in keys):
+                raise ValueError("rotation scaling needs positive %s; got %r" % (", ".join(keys), scaling))
         if layout not in ("half", "interleaved"):
             raise ValueError("rotation layout %r is not 'half' or 'interleaved'" % (layout,))
         self.interleaved = layout == "interleaved"
@@ -55,7 +59,7 @@ class RotaryPosition(Position):
     @property
     def magnitude(self) -> float:
         """What cosines and sines are multiplied by (1 without scaling)."""
-        return 1.0 if self.scaling is None else 0.1 * math.log(float(self.scaling["factor"])) + 1.0
+        return 1.0 if self.scaling is None or self.by_wavelength else 0.1 * math.log(float(self.scaling["factor"])) + 1.0
 
     def inverse_frequencies(self) -> np.ndarray:
         r = self.rotary_dim
@@ -64,6 +68,14 @@ class RotaryPosition(Position):
             return np.asarray(vals, dtype=np.float32)
         sc = self.scaling
         factor, original = float(sc["factor"]), float(sc["original"])
+        if self.by_wavelength:
+            low, high, vals = float(sc["low"]), float(sc["high"]), []
+            for i in range(r // 2):
+                f = self.theta ** (-2.0 * i / r)
+                turns = original * f / (2.0 * math.pi)   # original / wavelength
+                kept = 1.0 if turns > high else (0.0 if turns < low else (turns - low) / (high - low) if high != low else 0.0)
+                vals.append(kept * f + (1.0 - kept) * f / factor)
+            return np.asarray(vals, dtype=np.float32)
 
         def pair_index(turns: float) -> float:
             return r * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.theta))

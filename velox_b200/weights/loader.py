@@ -10,7 +10,7 @@ error that lists them all.  The reference stops at the first
 Element types on the device:
   matrices and tables: the engine's element type (bfloat16 files stay
     bfloat16 in a bfloat16 engine; the 32-bit engine widens them exactly);
-  norm weights, biases and matrices that are applied in 32 bits whatever the engine
+  norm weights, biases, shares of a token shift and matrices that are applied in 32 bits whatever the engine
     (a router, the mixing of a stream's copies): float32 (exact for bfloat16 files; a tensor stored in 32 bits stays so);
   integer tables: int32.
 """
@@ -50,7 +50,7 @@ _INTS = (torch.int32, torch.int64, torch.int16, torch.int8, torch.uint8)
 def held_dtype(role: str, stored: torch.dtype, runtime: Runtime) -> torch.dtype:
     if role == "int_table":
         return torch.int32
-    if role in ("norm", "bias", "matrix_f32", "mixing"):
+    if role in ("norm", "bias", "matrix_f32", "mixing", "share"):
         return torch.float32
     return runtime.dtype
 
