@@ -890,6 +890,195 @@ def fovenex_kernels(pk, sz):
     return rows
 
 
+# ---- Negilorn beside Kapuvik at equal size (`--workload negilorn`) ----------------------------------------
+# The same widths and head counts as above, four layers: attention over chunks of 1,024 (heads of 128, grouped key/value
+# heads, rotation stretched by wavelength, bounded scores, one added to the denominator, a gate per head) with a dense
+# feed-forward of the size that a Dobepel token runs through, two layers of RWKV-style time mixing (heads of 64, as many
+# channels as the width) with 8 experts of which 2 run plus a shared one, and an attention layer that reads the first
+# one's keys and values.  Kapuvik is the closest existing model: bounded softmax attention and linear attention with a decay
+# per channel through the same kernels.
+NEGILORN_CHUNK, NEGILORN_RANK = 1024, 64
+
+
+def negilorn_raw(sz):
+    ff = {"kind": "dense", "ff": DOBEPEL_TOP * sz["expert_ff"] + sz["shared_ff"]}
+    moe = {"kind": "moe", "expert": {"ff": sz["expert_ff"]}, "router": {"experts": DOBEPEL_EXPERTS, "top": DOBEPEL_TOP},
+           "shared": {"ff": sz["shared_ff"]}}
+    att = {"heads": sz["heads"], "kv_heads": sz["kv_heads"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": KAPUVIK_CAP,
+           "mask": {"size": NEGILORN_CHUNK}, "rot": {"base": 500000.0, "dims": 128, "scaling": {
+               "factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    wkv = {"heads": 2 * sz["lin_heads"], "dim": 64, "rank": NEGILORN_RANK}
+    layers = [{"type": "attention", "mixer": att, "mlp": ff}, {"type": "wkv", "mixer": wkv, "mlp": moe},
+              {"type": "wkv", "mixer": wkv, "mlp": moe}, {"type": "attention", "mixer": dict(att, kv_from=0), "mlp": ff}]
+    return {"architecture": "Negilorn", "vocab": DOBEPEL_VOCAB, "width": sz["width"], "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+            "layers": json.loads(json.dumps(layers))}
+
+
+def negilorn_workload(args, pk):
+    """Prefill (one prompt of 2,048 tokens in one step) and decode (batch 8 at 2,048 cached tokens) of Negilorn and of
+    Kapuvik at equal width and depth, through the step function, timed with CUDA events; then the design's own kernels
+    beside the like kernels of Kapuvik and Dobepel at the 2k size, each as a fraction of its roofline."""
+    import torch
+    from velox_b200.config import KapuvikConfig, NegilornConfig
+
+    T, B, CTX = 2048, 8, 2048
+    K, W = max(1, min(args.steps, 32)), max(3, args.warmup)
+    gen = torch.Generator().manual_seed(SEED)
+    sizes = {}
+    four = lambda sz: dict(sz, layers=4)
+    model_points(NegilornConfig.from_dict(negilorn_raw(four(DOBEPEL_SIZES["1k"]))), DOBEPEL_VOCAB, T, B, CTX, K, W, gen)  # thrown away
+    for name, sz in DOBEPEL_SIZES.items():
+        sz = four(sz)
+        sizes[name] = {"negilorn": model_points(NegilornConfig.from_dict(negilorn_raw(sz)), DOBEPEL_VOCAB, T, B, CTX, K, W, gen),
+                       "kapuvik": model_points(KapuvikConfig.from_dict(kapuvik_raw(sz)), DOBEPEL_VOCAB, T, B, CTX, K, W, gen),
+                       "shape": sz}
+    return {"metric": "Negilorn beside Kapuvik at equal size: prefill of %d tokens, decode at batch %d with %d cached tokens, bf16"
+                      % (T, B, CTX), "unit": "tokens/s", "n_gpus": 1, "steps": K, "warmup": W, "sizes": sizes,
+            "value": sizes["2k"]["negilorn"]["decode_tok_s"], "higher_is_better": True,
+            "kernels": negilorn_kernels(pk, four(DOBEPEL_SIZES["2k"])), "peaks": pk,
+            "data": "synthetic: random weights N(0,0.02) seed 2, uniform random token ids"}
+
+
+def negilorn_kernels(pk, sz):
+    """Microseconds and fractions of the roofline of Negilorn's kernels beside the like kernels of Kapuvik and Dobepel."""
+    import torch
+    from types import SimpleNamespace
+    from velox_b200.csrc import ops
+    dev, bf, f32 = "cuda:0", torch.bfloat16, torch.float32
+    E, H, G, D = sz["width"], sz["heads"], sz["kv_heads"], 128
+    HL, DL, RANK, CH = 2 * sz["lin_heads"], 64, NEGILORN_RANK, NEGILORN_CHUNK
+    HD = HL * DL
+    T, B, CTX, S = 2048, 8, 2048, PAGE
+    rows, row, us = kernel_rows(pk)
+    ints = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    rnd = lambda *shape: torch.randn(shape, device=dev)
+    pages = B * (CTX // S)
+    bt = torch.arange(pages, dtype=torch.int32, device=dev).view(B, CTX // S)
+    cu, off, pos_t = ints([0, T]), ints([0]), ints(list(range(T)))
+    seqs, pos = ints(list(range(B))), ints([CTX - 1] * B)
+    # -- attention over chunks --
+    kp, vp = rnd(pages, G, S, D).to(bf), rnd(pages, G, S, D).to(bf)
+    width = (H + 2 * G) * D + H
+    width += (-width) % 8
+    gate_col = (H + 2 * G) * D
+    q, qd, zeros = rnd(T, width).to(bf), rnd(B, width).to(bf), torch.zeros(H, device=dev)
+    pairs = sum(i % CH + 1 for i in range(T))
+    ours = dict(softcap=KAPUVIK_CAP, sinks=zeros, gate_col=gate_col, chunk=CH)
+    row("prompt attention over chunks of %d: bounded scores, one added to the denominator, gate (mma.sync, P in two halves)" % CH, us(
+        lambda: ops.biased_prefill_attention(q, width, kp, vp, bt, cu, off, D ** -0.5, 0, 0, 0.0, H, G, D, D, 1, T, T, **ours)), 4.0 * pairs * D * H)
+    row("Kapuvik: prompt attention, bounded scores, all keys (the same kernel)", us(lambda: ops.biased_prefill_attention(
+        q, width, kp, vp, bt, cu, off, D ** -0.5, 0, 0, 0.0, H, G, D, D, 1, T, T, softcap=KAPUVIK_CAP)), 4.0 * (T * (T + 1) // 2) * D * H)
+    row("decode attention over chunks, %d visible keys" % CH, us(lambda: ops.biased_decode_attention(
+        qd, width, kp, vp, bt, seqs, pos, D ** -0.5, 0, 0, 0.0, H, G, D, D, B, max_kv=CTX, **ours), 50), 0.0, B * G * CH * 2 * D * 2.0)
+    pos_ch = ints([CH - 1] * B)
+    row("Kapuvik: decode attention, bounded scores, %d keys (the same kernel)" % CH, us(lambda: ops.biased_decode_attention(
+        qd, width, kp, vp, bt, seqs, pos_ch, D ** -0.5, 0, 0, 0.0, H, G, D, D, B, max_kv=CH, softcap=KAPUVIK_CAP), 50), 0.0,
+        B * G * CH * 2 * D * 2.0)
+    slots = torch.randperm(pages * S, device=dev)[:T].to(torch.int32)
+    inv128 = (5e5 ** (-torch.arange(0, D, 2, device=dev, dtype=f32) / D)).contiguous()
+    row("q/k rotation + cache write, %d tokens" % T, us(lambda: ops.qk_norm_rope_kv(
+        q, None, None, 1e-6, inv128, D, pos_t, slots, kp, vp, H, G, D, D)), 0.0, T * (H + 2 * G) * D * 2 * 2.0)
+    qo = rnd(T, H * D + 8 * ((H + 7) // 8)).to(bf)
+    row("rotation of queries alone (borrowed keys), %d tokens" % T, us(lambda: ops.qk_norm_rope_kv(
+        qo, None, None, 1e-6, inv128, D, pos_t, None, None, None, H, 0, D, D)), 0.0, T * H * D * 2 * 2.0)
+    # -- token shift --
+    big = 16384
+    res, delta, w1 = rnd(big, E), rnd(big, E).to(bf), torch.ones(E, device=dev)
+    mu, nu = torch.rand(E, device=dev), torch.rand(5, E, device=dev)
+    st, sh = torch.zeros((B, E), device=dev), torch.zeros((B, E), device=dev)
+    step = lambda n, seqs_, new: SimpleNamespace(n_seqs=seqs_, max_new=new, cu_seqlens=ints([i * (n // seqs_) for i in range(seqs_ + 1)]),
+                                                 seq_of_token=ints([i // (n // seqs_) for i in range(n)]), state_slots=ints(list(range(seqs_))))
+    one, dec = step(big, 1, big), step(B, B, 1)
+    row("stream += mixer, norm, token shift, %d rows" % big, us(lambda: ops.shift_norm(
+        res, delta, w1, 1e-6, mu, one, st, bf), 10), 0.0, big * E * (4 + 2 + 4 + 2.0))
+    row("the same with the five mixes of the time mixing, %d rows" % big, us(lambda: ops.shift_norm(
+        res, delta, w1, 1e-6, mu, one, st, bf, mixes=nu, mix_state=sh), 10), 0.0, big * E * (4 + 2 + 4 + 10.0))
+    row("Kapuvik: stream += one term, then the next RMS norm, %d rows" % big, us(lambda: ops.sum_add_rmsnorm(
+        res, [(delta, 1.0)], weight=w1, eps=1e-6), 10), 0.0, big * E * (4 + 4 + 2 + 2.0))
+    row("Qwen3: stream += one term, then the next RMS norm, %d rows" % big, us(lambda: ops.add_rmsnorm(
+        res, delta, w1, 1e-6, bf), 10), 0.0, big * E * (4 + 4 + 2 + 2.0))
+    row("decode: stream += mixer, norm, token shift, five mixes, %d rows" % B, us(lambda: ops.shift_norm(
+        res[:B], delta[:B], w1, 1e-6, mu, dec, st, bf, mixes=nu, mix_state=sh), 50), 0.0, B * E * (4 + 2 + 4 + 10 + 16.0) + 7 * E * 4.0)
+    row("Kapuvik decode: stream += one term, then the next RMS norm, %d rows" % B, us(lambda: ops.sum_add_rmsnorm(
+        res[:B], [(delta[:B], 1.0)], weight=w1, eps=1e-6), 50), 0.0, B * E * 12.0 + E * 4.0)
+    # -- time mixing --
+    mixed, mixed_d = rnd(5, T, E).to(bf), rnd(5, B, E).to(bf)
+    N = 4 * HD + RANK
+    W = [(rnd(N, E) * 0.02).to(bf) for _ in range(8)]     # (rotated through: more than the L2 holds)
+    turn = [0]
+
+    def nxt(ws):
+        turn[0] += 1
+        return ws[turn[0] % len(ws)]
+    row("decode: five projections with an input each, one launch, %d rows" % B, us(lambda: ops.gemm_inputs(mixed_d, nxt(W), HD, f32), 48), 0.0, N * E * 2.0)
+    row("Kapuvik decode: one product of the same matrix (skinny), %d rows" % B, us(lambda: ops.gemm_skinny(mixed_d[0], nxt(W), None, bf), 48), 0.0, N * E * 2.0)
+    row("four projections with an input each (batched library product), %d tokens" % T, us(lambda: ops.gemm_members(
+        mixed[:4], W[0][:4 * HD].view(4, HD, E))), 2.0 * T * 4 * HD * E)
+    row("Kapuvik: one library product of the same size, %d tokens" % T, us(lambda: ops.gemm_bf16(mixed[0], W[0][:4 * HD])), 2.0 * T * 4 * HD * E)
+    low, w2t, w0 = rnd(T, RANK), rnd(RANK, HD) * 0.1, torch.zeros(HD, device=dev)
+    row("decays: -exp(tanh(x) W + b) in float32, %d tokens" % T, us(lambda: ops.low_rank_decay(low, w2t, w0)), 0.0, T * (HD + RANK) * 4.0)
+    w2b, lowb = (rnd(HD, RANK) * 0.1).to(bf), low.to(bf)
+    row("Kapuvik: the decays' second product + bias (library, bfloat16 operands), %d tokens" % T, us(lambda: ops.gemm_bf16(
+        lowb, w2b, w0, f32)), 0.0, T * HD * 4.0 + T * RANK * 2.0)
+    x4 = (rnd(4, T, HD) * 0.5).to(bf)
+    xd = rnd(B, N) * 0.5
+    la, lad, u = -torch.rand(T, HD, device=dev), -torch.rand(B, HD, device=dev), rnd(HL, DL)
+    state = torch.zeros((B, HL, DL, DL), device=dev)
+    cu_b, slots_b, slot0 = ints(list(range(B + 1))), ints(list(range(B))), ints([0])
+    fl = T * HL * 2.0 * (32 * 2 * DL + 2 * DL * DL)
+    sb = B * HL * DL * DL * 4 * 2.0
+    plan = ops.StretchPlan([T], dev)
+    row("prompt time mixing: walk with a bonus, %d heads of %d (stretches side by side)" % (HL, DL), us(lambda: ops.linear_attention_walk(
+        x4, 0, T * HD, 2 * T * HD, state, cu, slot0, 1, HL, DL, DL, gate=la, gate_is_log=True, bonus=u, stretches=plan), 5), fl)
+    xk = (rnd(T, 4 * HD) * 0.5).to(bf)
+    z = rnd(T, HD) + 2.0
+    row("Kapuvik: prompt linear attention, decay per channel, %d heads of %d (the same kernel)" % (HL, DL), us(
+        lambda: ops.linear_attention_walk(xk, 0, HD, 2 * HD, state, cu, slot0, 1, HL, DL, DL, gate=z, gate_mul=1 / 16.0, q_mul=DL ** -0.5,
+                                          stretches=plan), 5), fl)
+    row("decode time mixing: walk with a bonus, %d heads of %d" % (HL, DL), us(lambda: ops.linear_attention_walk(
+        xd, 0, HD, 2 * HD, state, cu_b, slots_b, B, HL, DL, DL, gate=lad, gate_is_log=True, bonus=u), 50), 0.0, sb)
+    xkd, zd = (rnd(B, 4 * HD) * 0.5).to(bf), rnd(B, HD)
+    row("Kapuvik: decode linear attention, decay per channel, %d heads of %d (the same kernel)" % (HL, DL), us(
+        lambda: ops.linear_attention_walk(xkd, 0, HD, 2 * HD, state, cu_b, slots_b, B, HL, DL, DL, gate=zd, gate_mul=1 / 16.0), 50), 0.0, sb)
+    o, g, wj, wv = rnd(big, HD), rnd(big, HD).to(bf), torch.ones(HD, device=dev), torch.ones(DL, device=dev)
+    row("per-head norm, weight per channel, silu gate, %d rows" % big, us(lambda: ops.head_norm_gate(o, g, wj, HL, 1e-6, "silu"), 10), 0.0, big * HD * 8.0)
+    row("Kapuvik: per-head norm + silu gate, %d rows" % big, us(lambda: ops.head_norm_gate(o, g, wv, HL, 1e-6, "silu"), 10), 0.0, big * HD * 8.0)
+    # -- experts --
+    NE, TOP, I = DOBEPEL_EXPERTS, DOBEPEL_TOP, sz["expert_ff"]
+    h, hd = rnd(T, E).to(bf), rnd(B, E).to(bf)
+    wr = (rnd(NE, E) * 0.02).float().contiguous()
+    up, down = (rnd(NE, I, E) * 0.02).to(bf), (rnd(NE, E, I) * 0.02).to(bf)
+    gu = (rnd(NE, 2 * I, E) * 0.02).to(bf)
+    p = ops.moe_route(h, wr, None, NE, TOP, ops.MOE_TCGEN05_TILE_ROWS, scores="sigmoid")
+    rows_h = ops.moe_gather_rows(h, p)
+    act = dict(activation="relu2", row_scale=p.weight.view(-1))
+    row("router (sigmoid) + plan, %d tokens" % T, us(lambda: ops.moe_route(h, wr, None, NE, TOP, ops.MOE_TCGEN05_TILE_ROWS, scores="sigmoid")), 0.0, T * E * 2.0)
+    row("Dobepel: router (softmax of the chosen) + plan, %d tokens" % T, us(lambda: ops.moe_route(h, wr, None, NE, TOP, ops.MOE_TCGEN05_TILE_ROWS)), 0.0, T * E * 2.0)
+    row("experts up, weight on the sums, square of relu, %d rows (tcgen05 grouped)" % (T * TOP), us(lambda: ops.moe_gemm_tcgen05(rows_h, up, p, **act)), 2.0 * T * TOP * I * E)
+    row("Dobepel: experts gate and up, %d rows (tcgen05 grouped)" % (T * TOP), us(lambda: ops.moe_gemm_tcgen05(rows_h, gu, p, gated_activation="silu")), 2.0 * T * TOP * 2 * I * E)
+    a = ops.moe_gemm_tcgen05(rows_h, up, p, **act)
+    row("experts down, %d rows (tcgen05 grouped)" % (T * TOP), us(lambda: ops.moe_gemm_tcgen05(a, down, p)), 2.0 * T * TOP * I * E)
+    ups = [(rnd(NE, I, E) * 0.02).to(bf) for _ in range(5)]
+    gus = [(rnd(NE, 2 * I, E) * 0.02).to(bf) for _ in range(3)]
+    tr = ops.moe_tile_rows(hd, B * TOP)
+    pd = ops.moe_route(hd, wr, None, NE, TOP, tr, scores="sigmoid")
+    live = len(set(pd.chosen.tolist()))
+    actd = dict(activation="relu2", row_scale=pd.weight.view(-1))
+    row("experts up, %d tokens (grouped mma.sync, row tiles of 16)" % B, us(lambda: ops.moe_gemm(hd, nxt(ups), pd, True, bf, **actd), 50),
+        0.0, live * I * E * 2.0)
+    row("Dobepel: experts gate and up, %d tokens" % B, us(lambda: ops.moe_gemm(hd, nxt(gus), pd, True, bf, gated_activation="silu"), 50),
+        0.0, live * 2 * I * E * 2.0)
+    ws = [(rnd(sz["shared_ff"], E) * 0.02).to(bf) for _ in range(32)]
+    row("shared expert up + square of relu, %d tokens (tcgen05)" % T, us(lambda: ops.gemm_tcgen05(h, ws[0], None, activation="relu2", wide=ops.tcgen05_wide_better(T // 128, sz["shared_ff"], dev))), 2.0 * T * E * sz["shared_ff"])
+    row("the same as library product + activation kernel, %d tokens" % T, us(lambda: ops.act(ops.gemm_bf16(h, ws[0], None, f32), "relu2", out_dtype=bf)), 2.0 * T * E * sz["shared_ff"])
+    row("shared expert up + square of relu, %d tokens (skinny)" % B, us(lambda: ops.gemm_skinny(hd, nxt(ws), None, bf, activation="relu2"), 64),
+        0.0, E * sz["shared_ff"] * 2.0)
+    y32 = ops.moe_gemm(ops.moe_gemm(hd, up, pd, True, bf, **actd), down, pd, False, f32)
+    sd = rnd(B, E).to(bf)
+    row("sum of the experts' rows + shared, %d tokens" % B, us(lambda: ops.moe_combine(y32, pd, sd, bf, weighted=False), 50), 0.0, B * E * (TOP * 4 + 4.0))
+    return rows
+
+
 def main() -> int:
     global CONTEXT, PROMPT
     ap = argparse.ArgumentParser()
@@ -899,13 +1088,14 @@ def main() -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the model has (recorded in config)")
     ap.add_argument("--batch", type=int, default=BATCH)
-    ap.add_argument("--workload", default="decode", choices=["decode", "stream", "dobepel", "buvuzen", "kapuvik", "fovenex"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "stream", "dobepel", "buvuzen", "kapuvik", "fovenex", "negilorn"],
                     help="decode: the benchmark (steady decoding at a fixed batch). stream: continuous batching "
                          "under arrivals (64 requests, prompts of 128-4,096 tokens, 256 new tokens each, Poisson "
                          "arrivals); prints its own JSON line. dobepel: the Dobepel design beside Qwen3 at equal size "
                          "(prefill, decode, and the design's kernels against their rooflines); its own JSON line. buvuzen: the same for "
                          "the Buvuzen design beside Dobepel and Qwen3. kapuvik: the same for the Kapuvik design beside Dobepel. "
-                         "fovenex: the same for the Fovenex design beside Kapuvik")
+                         "fovenex: the same for the Fovenex design beside Kapuvik; "
+                         "negilorn: the same for the Negilorn design beside Kapuvik")
     ap.add_argument("--arrival-rate", type=float, default=16.0, help="stream: mean arrivals a second")
     ap.add_argument("--lazy-graphs", action="store_true",
                     help="stream: capture each decode graph when a step first needs it, inside the run")
@@ -936,9 +1126,10 @@ def main() -> int:
     from velox_b200.csrc import ops
     from velox_b200.engine import StepEntry
 
-    if args.workload in ("dobepel", "buvuzen", "kapuvik", "fovenex"):
+    if args.workload in ("dobepel", "buvuzen", "kapuvik", "fovenex", "negilorn"):
         with ClockSampler() as clocks:
-            res = {"dobepel": dobepel_workload, "buvuzen": buvuzen_workload, "kapuvik": kapuvik_workload, "fovenex": fovenex_workload}[args.workload](args, peaks())
+            res = {"dobepel": dobepel_workload, "buvuzen": buvuzen_workload, "kapuvik": kapuvik_workload, "fovenex": fovenex_workload,
+                   "negilorn": negilorn_workload}[args.workload](args, peaks())
         res["clocks"] = clocks.summary()
         print(json.dumps(res))
         return 0

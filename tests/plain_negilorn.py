@@ -20,7 +20,7 @@ def store_bfloat16(x):
     a = np.ascontiguousarray(x, dtype=np.float32)
     bits = a.view(np.uint32).astype(np.uint64)
     bits = (bits + 0x7FFF + ((bits >> 16) & 1)) & 0xFFFF0000
-    return bits.astype(np.uint32).view(np.float32).astype(np.float64).reshape(a.shape)
+    return bits.astype(np.uint32).view(np.float32).astype(np.float64).reshape(np.shape(x))
 
 
 def same(x):

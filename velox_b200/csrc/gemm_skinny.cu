@@ -197,6 +197,7 @@ static int launch_skinny(const bf16* x, const bf16* W, const float* bias, TOut* 
     // blocks fill whole waves (slots = SMs x blocks per SM of the variant).
     const int units = GATED ? N / 2 : N, tile = GATED ? 8 : 16;
     int R = tile;
+    long long room = 0;
     if (variant >= 1 && variant <= 7 && balance) {
         static const int per_sm[8] = {0, 4, 2, 2, 1, 4, 3, 4};
         const long long slots = (long long)sm_count() * per_sm[variant];
@@ -204,11 +205,15 @@ static int launch_skinny(const bf16* x, const bf16* W, const float* bias, TOut* 
         const long long waves = (tiles + slots - 1) / slots;
         R = (int)((units + waves * slots - 1) / (waves * slots));
         R = R < 1 ? 1 : (R > tile ? tile : R);
+        room = waves * slots;
     }
     int blocks = (units + R - 1) / R;
     if (SEG) {
-        const int before = (segments - 1) * ((seg_rows + R - 1) / R);
-        blocks = before + (N - (segments - 1) * seg_rows + R - 1) / R;
+        // (every input's last block may be a short one: a row more a block where that would begin another wave)
+        for (;; ++R) {
+            blocks = (segments - 1) * ((seg_rows + R - 1) / R) + (N - (segments - 1) * seg_rows + R - 1) / R;
+            if (blocks <= room || R >= tile) break;
+        }
     }
 #define SK_GO(WARPS, UNROLL, MINB)                                                                                  \
     VX_LAUNCH_K(VX_K_GEMM, (gemm_skinny_kernel<GATED, SEG, TOut, WARPS, UNROLL, MINB>), blocks, WARPS * 32, 0, stream, x, W, \

@@ -22,7 +22,7 @@
 //            tcgen05.ld, 32 columns at a time, adds the bias, rounds to bfloat16 and
 //            stores; or, gated, takes act(gate) * up of column tiles laid out as 8
 //            gate columns followed by their 8 up columns, in float32, and stores
-//            half as many columns, or takes act(.) of every column; then they arrive on the accumulator's "empty"
+//            half as many columns, or takes relu or its square of every column; then they arrive on the accumulator's "empty"
 //            mbarrier.
 // Rows past M and columns past N are zero-filled by TMA on the way in and masked on
 // the way out; K may end inside a k block (zero-filled too).
@@ -40,7 +40,9 @@
 
 #define TC_PLAIN 0
 #define TC_GATED 1   // act(gate) * up of paired columns
-#define TC_ACT 2     // act(.) of each column
+#define TC_ACT 2     // act(.) of each column: relu or its square (of every column the exponentials of other activations,
+                     // inlined 32 times, would cost more than a kernel of their own)
+static bool tc_cheap_act(int act) { return act == VX_ACT_RELU || act == VX_ACT_RELU2; }
 
 template <int BN, int STAGES, int EPI>
 __global__ void __launch_bounds__(TC_THREADS)
@@ -189,7 +191,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                         for (int i = 0; i < 8; ++i) {
                             v[i] = __uint_as_float(r[j + i]);
                             if (bias) v[i] += bias[n0 + c0 + j + i];
-                            if (EPI == TC_ACT) v[i] = activation(v[i], act);
+                            if (EPI == TC_ACT) {
+                                v[i] = fmaxf(v[i], 0.f);
+                                v[i] *= act == VX_ACT_RELU2 ? v[i] : 1.f;
+                            }
                         }
                         uint4 pk;
                         __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&pk);
@@ -251,7 +256,7 @@ static int tc_launch(const CUtensorMap& ma, const CUtensorMap& mw, const float* 
 }
 
 // gated: 0 plain, C is [M, N]; 1: W's rows come in tiles of 8 gate rows followed by
-// their 8 up rows and C is [M, N/2] = act(gate) * up; 2: C is [M, N] = act(.).  `error` is a device int that
+// their 8 up rows and C is [M, N/2] = act(gate) * up; 2: C is [M, N] = act(.), relu or its square.  `error` is a device int that
 // a block sets (TC_ERR_*) if one of its bounded waits runs out; the caller zeroes it
 // and reads it when it wants to know.  `wide` picks 128 x 256 tiles (else 128 x 128).
 extern "C" int vx_gemm_tcgen05(const void* A, const void* W, const float* bias, void* C, int M, int N, int K, int lda,
@@ -261,6 +266,7 @@ extern "C" int vx_gemm_tcgen05(const void* A, const void* W, const float* bias, 
     if ((lda & 7) || (ldw & 7) || (ldc & 7) || lda < K || ldw < K) return VX_ERR_ALIGN;
     if ((((uintptr_t)A) | ((uintptr_t)W) | ((uintptr_t)C)) & 15) return VX_ERR_ALIGN;
     if (gated < 0 || gated > TC_ACT || (gated && (act < 0 || act > VX_ACT_LAST)) || (gated == TC_GATED && bias)) return VX_ERR_SHAPE;
+    if (gated == TC_ACT && !tc_cheap_act(act)) return VX_ERR_SHAPE;
     if (ldc < (gated == TC_GATED ? N / 2 : N)) return VX_ERR_SHAPE;
     CUtensorMap ma, mw;
     const int bn = wide ? 256 : 128;
@@ -275,12 +281,12 @@ extern "C" int vx_gemm_tcgen05(const void* A, const void* W, const float* bias, 
 // The grouped product of a routed feed-forward: A [rows, K] in group order, W [groups, N, K], row tiles of up to
 // 128 rows (group, first row, rows) whose number is on the device (at most max_row_tiles).  C [rows, N], or
 // [rows, N/2] = act(gate) * up when gated (1), act(.) of each element with gated = 2.  With row_scale (then gated is not 0)
-// row p's sums are first multiplied by row_scale[src_of_row[p]].
+// row p's sums are first multiplied by row_scale[src_of_row[p]].  `wide`: tiles of 256 columns, else of 128.
 extern "C" int vx_moe_gemm_tcgen05_scaled(const void* A, const void* W, void* C, int rows, int groups, int N, int K, int lda,
                                    int ldc, int gated, int act, const int* row_tiles, const int* n_row_tiles,
                                    int max_row_tiles, int* error, const float* row_scale, const int* src_of_row,
-                                   cudaStream_t stream) {
-    if (row_scale && (!src_of_row || !gated)) return VX_ERR_SHAPE;
+                                          int wide, cudaStream_t stream) {
+    if ((row_scale && (!src_of_row || !gated)) || (gated == TC_ACT && !tc_cheap_act(act))) return VX_ERR_SHAPE;
     if (rows <= 0 || N <= 0 || max_row_tiles <= 0) return VX_OK;
     if (K <= 0 || (K & 7) || (N & 15) || groups <= 0 || !error || !row_tiles || !n_row_tiles) return VX_ERR_SHAPE;
     if ((lda & 7) || (ldc & 7) || lda < K) return VX_ERR_ALIGN;
@@ -288,10 +294,13 @@ extern "C" int vx_moe_gemm_tcgen05_scaled(const void* A, const void* W, void* C,
     if (gated < 0 || gated > TC_ACT || (gated && (act < 0 || act > VX_ACT_LAST))) return VX_ERR_SHAPE;
     if (ldc < (gated == TC_GATED ? N / 2 : N) || (long long)groups * N > 0x7fffffffLL) return VX_ERR_SHAPE;
     CUtensorMap ma, mw;
-    if (!tc_make_map(&ma, A, rows, K, lda, TC_BM) || !tc_make_map(&mw, W, groups * N, K, K, 256)) return VX_ERR_DRIVER;
+    if (!tc_make_map(&ma, A, rows, K, lda, TC_BM) || !tc_make_map(&mw, W, groups * N, K, K, wide ? 256 : 128)) return VX_ERR_DRIVER;
     bf16* c = (bf16*)C;
-#define TC_GO(E_) tc_launch<256, 4, E_>(ma, mw, nullptr, c, rows, N, K, ldc, act, error, stream, row_tiles, n_row_tiles, max_row_tiles, row_scale, src_of_row)
-    return gated == TC_GATED ? TC_GO(TC_GATED) : (gated == TC_ACT ? TC_GO(TC_ACT) : TC_GO(TC_PLAIN));
+#define TC_GO(BN_, ST_, E_)                                                                                                  \
+    tc_launch<BN_, ST_, E_>(ma, mw, nullptr, c, rows, N, K, ldc, act, error, stream, row_tiles, n_row_tiles, max_row_tiles, \
+                            row_scale, src_of_row)
+    if (wide) return gated == TC_GATED ? TC_GO(256, 4, TC_GATED) : (gated == TC_ACT ? TC_GO(256, 4, TC_ACT) : TC_GO(256, 4, TC_PLAIN));
+    return gated == TC_GATED ? TC_GO(128, 6, TC_GATED) : (gated == TC_ACT ? TC_GO(128, 6, TC_ACT) : TC_GO(128, 6, TC_PLAIN));
 #undef TC_GO
 }
 
@@ -299,5 +308,5 @@ extern "C" int vx_moe_gemm_tcgen05(const void* A, const void* W, void* C, int ro
                                    int ldc, int gated, int act, const int* row_tiles, const int* n_row_tiles,
                                    int max_row_tiles, int* error, cudaStream_t stream) {
     return vx_moe_gemm_tcgen05_scaled(A, W, C, rows, groups, N, K, lda, ldc, gated, act, row_tiles, n_row_tiles, max_row_tiles, error,
-                                      nullptr, nullptr, stream);
+                                      nullptr, nullptr, 1, stream);
 }

@@ -135,7 +135,7 @@ def _declare(lib) -> None:
         "vx_gemm_skinny_act": [P, P, P, P, I, I, I, I, I, I, I, I, I, I, P],
         "vx_gemm_skinny_inputs": [P, P, P, I, I, I, I, I, I, I, c_longlong, I, I, P],
         "vx_moe_gemm_scaled": [P, I, P, I, P, P, P, I, P, I, I, I, I, I, I, I, I, I, P, P],
-        "vx_moe_gemm_tcgen05_scaled": [P, P, P, I, I, I, I, I, I, I, I, P, P, I, P, P, P, P],
+        "vx_moe_gemm_tcgen05_scaled": [P, P, P, I, I, I, I, I, I, I, I, P, P, I, P, P, P, I, P],
         "vx_latent_gather_window": [P, P, I, P, P, P, P, I, P, I, I, I, I, I, I, I, P],
     }
     lib.vx_set_pdl_mask.argtypes = [I]
@@ -756,6 +756,7 @@ def moe_gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, plan: MoePlan, gated_acti
     `moe_gemm`."""
     _dev(a, w, row_scale)
     code, act = _epilogue("moe_gemm_tcgen05", gated_activation, activation)
+    _need(activation is None or activation in TCGEN05_ACTIVATIONS, "moe_gemm_tcgen05: a plain activation is one of %s" % (TCGEN05_ACTIVATIONS,))
     _need(row_scale is None or (code and row_scale.dtype == torch.float32 and row_scale.numel() == plan.assignments),
           "moe_gemm_tcgen05: one float32 scale per assignment, with an activation")
     _need(a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.is_contiguous() and w.dim() == 3
@@ -764,10 +765,12 @@ def moe_gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, plan: MoePlan, gated_acti
     n, k = w.shape[1], w.shape[2]
     cols = n // 2 if gated_activation else n
     out = torch.empty((plan.assignments, cols), dtype=torch.bfloat16, device=a.device)
+    # (how many row tiles the experts' shares fill is on the device; half a tile more per expert on the average)
+    wide = tcgen05_wide_better(-(-plan.assignments // MOE_TCGEN05_TILE_ROWS) + w.shape[0] // 2, n, a.device)
     _check(library().vx_moe_gemm_tcgen05_scaled(_ptr(a), _ptr(w), _ptr(out), plan.assignments, w.shape[0], n, k, a.stride(0), cols,
                                                 code, act, _ptr(plan.tiles), _ptr(plan.n_tiles), plan.max_tiles,
                                                 _ptr(_error_word(a.device)), _ptr(row_scale),
-                                                _ptr(plan.src_of_row) if row_scale is not None else None, _stream()),
+                                                _ptr(plan.src_of_row) if row_scale is not None else None, 1 if wide else 0, _stream()),
            "moe_gemm_tcgen05")
     note_bounded_wait()
     return out
@@ -1489,6 +1492,23 @@ def tcgen05_pair_better(m: int, n: int, device) -> bool:
     return paired * 0.97 < single
 
 
+TCGEN05_ACTIVATIONS = ("relu", "relu2")   # what the tcgen05 products apply to every sum (gates: any activation)
+
+
+def tcgen05_wide_better(row_tiles: int, n: int, device) -> bool:
+    """Whether tiles of 128 x 256 are at least as fast as tiles of 128 x 128 for `row_tiles` row tiles and n columns: a narrow
+    tile takes a little more than half a wide one's time, and what counts are the rounds of the GPU's SMs."""
+    sms = _sm_count(device)
+    wide = -(-(row_tiles * -(-n // 256)) // sms)
+    narrow = -(-(row_tiles * -(-n // 128)) // sms)
+    return wide <= 0.6 * narrow
+
+
+def tcgen05_fills(m: int, n: int, device) -> bool:
+    """Whether an [m, n] product has a tile of 128 x 256 for every SM."""
+    return -(-m // 128) * -(-n // 256) >= _sm_count(device)
+
+
 def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, bias=None, gated_activation: Optional[str] = None,
                  wide: bool = True, pair: bool = False, activation: Optional[str] = None) -> torch.Tensor:
     """a [M,K] times w [N,K] transposed on the tcgen05 tensor cores (bfloat16 in and
@@ -1496,9 +1516,10 @@ def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, bias=None, gated_activation: 
     `gated_activation`, w's rows come in tiles of 8 gate rows followed by their 8 up
     rows and the result is act(gate) * up, [M, N/2].  `wide`: 128 x 256 tiles, else
     128 x 128; `pair`: 256 x 256 tiles, each formed by a pair of blocks.  With `activation` the result is act(.) of the
-    float32 sums (single blocks only)."""
+    float32 sums (single blocks only; one of `TCGEN05_ACTIVATIONS`)."""
     _dev(a, w, bias)
     code, act = _epilogue("gemm_tcgen05", gated_activation, activation)
+    _need(activation is None or activation in TCGEN05_ACTIVATIONS, "gemm_tcgen05: a plain activation is one of %s" % (TCGEN05_ACTIVATIONS,))
     _need(not (pair and activation), "gemm_tcgen05: a plain activation on tiles of single blocks")
     _need(a.dim() == 2 and w.dim() == 2 and a.shape[1] == w.shape[1], "gemm_tcgen05: a [M,K], w [N,K]")
     _need(tcgen05_supported(a, w), "gemm_tcgen05: bfloat16, K a multiple of 8, N a multiple of 16, 16-byte aligned rows")

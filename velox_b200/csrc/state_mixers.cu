@@ -426,24 +426,87 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const TG* __r
     }
 }
 
+// The same for heads of 4 LANES channels and rows on 16-byte borders: 32 / LANES heads a warp, a lane holding four
+// consecutive channels of its head.
+__device__ __forceinline__ void hn_load4(const float* p, float (&v)[4]) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+__device__ __forceinline__ void hn_load4(const bf16* p, float (&v)[4]) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+}
+__device__ __forceinline__ void hn_store4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void hn_store4(bf16* p, const float (&v)[4]) {
+    uint2 raw;
+    *reinterpret_cast<__nv_bfloat162*>(&raw.x) = __floats2bfloat162_rn(v[0], v[1]);
+    *reinterpret_cast<__nv_bfloat162*>(&raw.y) = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = raw;
+}
+
+template <typename TG, typename T, int LANES>
+__global__ void head_norm_gate_lanes_kernel(const float* __restrict__ o, const TG* __restrict__ g, int ldg,
+                                            const float* __restrict__ w, int w_head, T* __restrict__ out, int rows, int H,
+                                            float eps, int gate_act) {
+    constexpr int Dv = 4 * LANES;
+    pdl_wait();
+    pdl_trigger();
+    const int unit = blockIdx.x * (blockDim.x / LANES) + threadIdx.x / LANES, d = 4 * (threadIdx.x % LANES);
+    if (unit - (int)(threadIdx.x & 31) / LANES >= rows * H) return;   // (a whole warp past the end)
+    const bool live = unit < rows * H;
+    const int t = live ? unit / H : 0, h = live ? unit - t * H : 0;
+    float v[4], z[4], wv[4] = {1.f, 1.f, 1.f, 1.f};
+    hn_load4(o + ((size_t)t * H + h) * Dv + d, v);
+    hn_load4(g + (size_t)t * ldg + (size_t)h * Dv + d, z);
+    if (w) hn_load4(w + (size_t)h * w_head + d, wv);
+    float ss = v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3];
+#pragma unroll
+    for (int x = LANES / 2; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+    const float rstd = rsqrtf(ss / (float)Dv + eps);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        const float sg = 1.f / (1.f + expf(-z[e]));
+        v[e] = v[e] * rstd * wv[e] * (gate_act ? z[e] * sg : sg);
+    }
+    if (live) hn_store4(out + ((size_t)t * H + h) * Dv + d, v);
+}
+
+template <typename TG, typename T>
+static int launch_head_norm_gate(const float* o, const TG* g, int ldg, const float* w, int w_head, T* out, int rows, int H, int Dv,
+                                 float eps, int gate_act, cudaStream_t stream) {
+    const long long units = (long long)rows * H;
+    const bool wide = !(((uintptr_t)o | (uintptr_t)w) & 15) && !(((uintptr_t)g) & (4 * sizeof(TG) - 1)) && !(((uintptr_t)out) & (4 * sizeof(T) - 1)) && ldg % 4 == 0;
+    const int lanes = wide && (Dv == 32 || Dv == 64 || Dv == 128) ? Dv / 4 : 0;
+    const int threads = 128, per_block = lanes ? threads / lanes : threads / 32;
+    const long long blocks = (units + per_block - 1) / per_block;
+    if (units > 0x7fffffffLL - 4096) return VX_ERR_LIMIT;
+#define HN_GO(L_) VX_LAUNCH_K(VX_K_ELEMENTWISE, (head_norm_gate_lanes_kernel<TG, T, L_>), (unsigned)blocks, threads, 0, stream, o, g, ldg, w, w_head, out, rows, H, eps, gate_act)
+    if (lanes == 8) HN_GO(8);
+    else if (lanes == 16) HN_GO(16);
+    else if (lanes == 32) HN_GO(32);
+    else
+        VX_LAUNCH_K(VX_K_ELEMENTWISE, (head_norm_gate_kernel<TG, T>), (unsigned)blocks, threads, 0, stream, o, g, ldg, w, w_head, out, rows,
+                    H, Dv, eps, gate_act);
+#undef HN_GO
+    VX_LAUNCH_CHECK();
+    return VX_OK;
+}
+
 // g_dtype: the gate's element type, dtype: the output's (float32 gates with bfloat16 outputs are taken too).
 extern "C" int vx_head_norm_gate_heads(const float* o, const void* g, int ldg, const float* w, int w_per_head, void* out, int rows,
                                        int H, int Dv, float eps, int gate_act, int g_dtype, int dtype, cudaStream_t stream) {
     if (rows <= 0) return VX_OK;
     if (H <= 0 || Dv <= 0 || ldg < H * Dv) return VX_ERR_SHAPE;
-    const int warps = 4, w_head = w_per_head ? Dv : 0;
-    const long long blocks = ((long long)rows * H + warps - 1) / warps;
-    if (blocks > 0x7fffffffLL) return VX_ERR_LIMIT;
+    const int w_head = w_per_head ? Dv : 0;
     if (dtype == VX_F32 && g_dtype == VX_F32)
-        VX_LAUNCH_K(VX_K_ELEMENTWISE, (head_norm_gate_kernel<float, float>), (unsigned)blocks, warps * 32, 0, stream, o, (const float*)g, ldg, w, w_head, (float*)out, rows, H, Dv, eps, gate_act);
-    else if (dtype == VX_BF16 && g_dtype == VX_BF16)
-        VX_LAUNCH_K(VX_K_ELEMENTWISE, (head_norm_gate_kernel<bf16, bf16>), (unsigned)blocks, warps * 32, 0, stream, o, (const bf16*)g, ldg, w, w_head, (bf16*)out, rows, H, Dv, eps, gate_act);
-    else if (dtype == VX_BF16 && g_dtype == VX_F32)
-        VX_LAUNCH_K(VX_K_ELEMENTWISE, (head_norm_gate_kernel<float, bf16>), (unsigned)blocks, warps * 32, 0, stream, o, (const float*)g, ldg, w, w_head, (bf16*)out, rows, H, Dv, eps, gate_act);
-    else
-        return VX_ERR_DTYPE;
-    VX_LAUNCH_CHECK();
-    return VX_OK;
+        return launch_head_norm_gate<float, float>(o, (const float*)g, ldg, w, w_head, (float*)out, rows, H, Dv, eps, gate_act, stream);
+    if (dtype == VX_BF16 && g_dtype == VX_BF16)
+        return launch_head_norm_gate<bf16, bf16>(o, (const bf16*)g, ldg, w, w_head, (bf16*)out, rows, H, Dv, eps, gate_act, stream);
+    if (dtype == VX_BF16 && g_dtype == VX_F32)
+        return launch_head_norm_gate<float, bf16>(o, (const float*)g, ldg, w, w_head, (bf16*)out, rows, H, Dv, eps, gate_act, stream);
+    return VX_ERR_DTYPE;
 }
 
 extern "C" int vx_head_norm_gate(const float* o, const void* g, int ldg, const float* w, void* out, int rows, int H,

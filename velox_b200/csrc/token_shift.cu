@@ -57,12 +57,13 @@ struct TsStep {
 // a + (b - a) * m
 __device__ __forceinline__ float ts_mix(float a, float b, float m) { return fmaf(b - a, m, a); }
 
-template <typename T, int V, int NG>
-__global__ void __launch_bounds__(TS_MAX_THREADS)
+// (blocks an SM: rows of one group a thread without mixes leave registers for three)
+template <typename T, int V, int NG, bool MIX>
+__global__ void __launch_bounds__(TS_MAX_THREADS, NG == 1 ? (MIX ? 2 : 3) : 1)
 shift_norm_kernel(const float* __restrict__ res_in, const T* __restrict__ delta, float* __restrict__ res_out,
                   const float* __restrict__ w, float eps, const float* __restrict__ mu, const float* __restrict__ nu, int mixes,
                   TsStep st, float* state_n, float* state_h, float* __restrict__ save, T* __restrict__ out, int E, int R) {
-    __shared__ float scratch[32];
+    __shared__ float scratch[2][TS_MAX_THREADS / 32];
     const int t0 = blockIdx.x * R, t1 = min(st.tokens, t0 + R);
     int at[NG];
     bool in[NG];
@@ -93,13 +94,22 @@ shift_norm_kernel(const float* __restrict__ res_in, const T* __restrict__ delta,
             }
         }
     };
+    // One barrier a row: the warps' sums of consecutive rows go to two buffers in turn (when a buffer is written again, every
+    // thread has passed the barrier after its last reading).
+    int turn = 0;
+    const int warps = blockDim.x >> 5, lane = threadIdx.x & 31;
     auto norm = [&](float (&v)[NG][V]) {
         float ss = 0.f;
 #pragma unroll
         for (int j = 0; j < NG; ++j)
 #pragma unroll
             for (int e = 0; e < V; ++e) ss = fmaf(v[j][e], v[j][e], ss);
-        const float rstd = rsqrtf(block_sum(ss, scratch) / (float)E + eps);
+        ss = warp_sum(ss);
+        if (lane == 0) scratch[turn][threadIdx.x >> 5] = ss;
+        __syncthreads();
+        ss = warp_sum(lane < warps ? scratch[turn][lane] : 0.f);
+        turn ^= 1;
+        const float rstd = rsqrtf(ss / (float)E + eps);
 #pragma unroll
         for (int j = 0; j < NG; ++j)
 #pragma unroll
@@ -119,15 +129,15 @@ shift_norm_kernel(const float* __restrict__ res_in, const T* __restrict__ delta,
     fetch(t0, cur);
     if (t0 == first) {
         from_slot(state_n, slot, np);
-        if (mixes) from_slot(state_h, slot, hp);
+        if (MIX) from_slot(state_h, slot, hp);
     } else {
         fetch(t0 - 1, np);
-        if (mixes) {
+        if (MIX) {
             if (t0 - 1 == first) from_slot(state_n, slot, hp);
             else { fetch(t0 - 2, hp); norm(hp); }
         }
         norm(np);
-        if (mixes) {
+        if (MIX) {
 #pragma unroll
             for (int j = 0; j < NG; ++j)
 #pragma unroll
@@ -141,7 +151,7 @@ shift_norm_kernel(const float* __restrict__ res_in, const T* __restrict__ delta,
             end = st.cu_seqlens[seq + 1];
             slot = st.state_slots[seq];
             from_slot(state_n, slot, np);
-            if (mixes) from_slot(state_h, slot, hp);
+            if (MIX) from_slot(state_h, slot, hp);
         }
         if (t + 1 < t1) fetch(t + 1, nxt);
         if (delta) {
@@ -156,7 +166,7 @@ shift_norm_kernel(const float* __restrict__ res_in, const T* __restrict__ delta,
 #pragma unroll
             for (int e = 0; e < V; ++e) h[e] = ts_mix(cur[j][e], np[j][e], m[j][e]);
             if (in[j]) {
-                if (!mixes) {
+                if (!MIX) {
                     ts_store<V>(out + (size_t)t * E + at[j], h);
                 } else {
                     for (int i = 0; i < mixes; ++i) {
@@ -179,7 +189,7 @@ shift_norm_kernel(const float* __restrict__ res_in, const T* __restrict__ delta,
             for (int j = 0; j < NG; ++j) {
                 if (!in[j]) continue;
                 ts_store<V>(dn + at[j], np[j]);
-                if (mixes) ts_store<V>(dh + at[j], hp[j]);
+                if (MIX) ts_store<V>(dh + at[j], hp[j]);
             }
         }
     }
@@ -222,8 +232,14 @@ static int launch_shift_norm(const float* res_in, const T* delta, float* res_out
     int threads = ((groups + ng - 1) / ng + 31) / 32 * 32;
     const int blocks = (st.tokens + R - 1) / R;
 #define TS_GO(V_, NG_)                                                                                                         \
-    VX_LAUNCH_K(VX_K_ELEMENTWISE, (shift_norm_kernel<T, V_, NG_>), blocks, threads, 0, stream, res_in, delta, res_out, w, eps, mu, nu, \
-                mixes, st, state_n, state_h, save, out, E, R)
+    do {                                                                                                                       \
+        if (mixes)                                                                                                             \
+            VX_LAUNCH_K(VX_K_ELEMENTWISE, (shift_norm_kernel<T, V_, NG_, true>), blocks, threads, 0, stream, res_in, delta,    \
+                        res_out, w, eps, mu, nu, mixes, st, state_n, state_h, save, out, E, R);                                \
+        else                                                                                                                   \
+            VX_LAUNCH_K(VX_K_ELEMENTWISE, (shift_norm_kernel<T, V_, NG_, false>), blocks, threads, 0, stream, res_in, delta,   \
+                        res_out, w, eps, mu, nu, mixes, st, state_n, state_h, save, out, E, R);                                \
+    } while (0)
 #define TS_GO_V(V_)                                                                                                            \
     do {                                                                                                                       \
         if (ng == 1) TS_GO(V_, 1); else if (ng == 2) TS_GO(V_, 2); else if (ng == 4) TS_GO(V_, 4); else TS_GO(V_, 8);          \
@@ -306,65 +322,92 @@ extern "C" int vx_shift_mix(const void* x, const float* nu, int mixes, const int
     return VX_OK;
 }
 
-// log a[t, c] = -exp(b[c] + sum_r tanh(x[t, r]) w[r, c]), all float32.  A block takes LD_TOKENS tokens by LD_THREADS
-// channels: the tokens' tanh in shared memory, a channel's sums in registers, w read once per block (coalesced: it is
-// stored [rank, channels]).  r runs upwards, so a token's result does not depend on the tokens beside it.
+// log a[t, c] = -exp(b[c] + sum_r tanh(x[t, r]) w[r, c]), all float32.  A block takes TOK tokens by LD_THREADS * CH
+// channels: the tokens' tanh in shared memory, the sums of CH channels a thread in registers, w read once per block
+// (coalesced: it is stored [rank, channels]).  r runs upwards, so a token's result does not depend on the tokens beside it.
 #define LD_THREADS 128
-template <int LD_TOKENS>
+#define LD_AHEAD 4
+template <int TOK, int CH>
 __global__ void __launch_bounds__(LD_THREADS)
 low_rank_decay_kernel(const float* __restrict__ x, int ldx, int rank, const float* __restrict__ w, const float* __restrict__ b,
                       float* __restrict__ out, int tokens, int C) {
-    extern __shared__ __align__(16) float ld_s[];   // [rank][LD_TOKENS]
-    const int c = blockIdx.x * LD_THREADS + threadIdx.x, t0 = blockIdx.y * LD_TOKENS;
-    float first[8];   // the weights depend on no earlier kernel
+    extern __shared__ __align__(16) float ld_s[];   // [rank][TOK]
+    const int c0 = blockIdx.x * LD_THREADS * CH + threadIdx.x, t0 = blockIdx.y * TOK;
+    float wv[LD_AHEAD][CH], acc[TOK][CH];
+    bool in[CH];
 #pragma unroll
-    for (int u = 0; u < 8; ++u) first[u] = (c < C && u < rank) ? w[(size_t)u * C + c] : 0.f;
-    float acc[LD_TOKENS];
-    const float b0 = c < C ? b[c] : 0.f;
+    for (int j = 0; j < CH; ++j) {
+        const int c = c0 + j * LD_THREADS;
+        in[j] = c < C;
+        const float b0 = in[j] ? b[c] : 0.f;
 #pragma unroll
-    for (int i = 0; i < LD_TOKENS; ++i) acc[i] = b0;
+        for (int i = 0; i < TOK; ++i) acc[i][j] = b0;
+#pragma unroll
+        for (int u = 0; u < LD_AHEAD; ++u) wv[u][j] = (in[j] && u < rank) ? w[(size_t)u * C + c] : 0.f;   // (weights depend on no earlier kernel)
+    }
     pdl_wait();
     pdl_trigger();
-    for (int i = threadIdx.x; i < rank * LD_TOKENS; i += LD_THREADS) {
+    for (int i = threadIdx.x; i < rank * TOK; i += LD_THREADS) {
         const int tt = i / rank, r = i - tt * rank;
-        ld_s[r * LD_TOKENS + tt] = t0 + tt < tokens ? tanhf(x[(size_t)(t0 + tt) * ldx + r]) : 0.f;
+        ld_s[r * TOK + tt] = t0 + tt < tokens ? tanhf(x[(size_t)(t0 + tt) * ldx + r]) : 0.f;
     }
     __syncthreads();
-    if (c >= C) return;
-    for (int r0 = 0; r0 < rank; r0 += 8) {
-        float wv[8];
+    for (int r0 = 0; r0 < rank; r0 += LD_AHEAD) {
+        float nw[LD_AHEAD][CH];
 #pragma unroll
-        for (int u = 0; u < 8; ++u) wv[u] = r0 == 0 ? first[u] : (r0 + u < rank ? w[(size_t)(r0 + u) * C + c] : 0.f);
+        for (int u = 0; u < LD_AHEAD; ++u)
 #pragma unroll
-        for (int u = 0; u < 8; ++u) {
-            if (r0 + u >= rank) break;
+            for (int j = 0; j < CH; ++j)
+                nw[u][j] = (in[j] && r0 + LD_AHEAD + u < rank) ? w[(size_t)(r0 + LD_AHEAD + u) * C + c0 + j * LD_THREADS] : 0.f;
 #pragma unroll
-            for (int i = 0; i < LD_TOKENS; ++i) acc[i] = fmaf(ld_s[(r0 + u) * LD_TOKENS + i], wv[u], acc[i]);
+        for (int u = 0; u < LD_AHEAD; ++u) {
+            if (r0 + u < rank) {
+                float th[TOK];
+                if constexpr (TOK % 4 == 0) {
+#pragma unroll
+                    for (int i = 0; i < TOK; i += 4) {
+                        const float4 t4 = *reinterpret_cast<const float4*>(ld_s + (r0 + u) * TOK + i);
+                        th[i] = t4.x; th[i + 1] = t4.y; th[i + 2] = t4.z; th[i + 3] = t4.w;
+                    }
+                } else {
+#pragma unroll
+                    for (int i = 0; i < TOK; ++i) th[i] = ld_s[(r0 + u) * TOK + i];
+                }
+#pragma unroll
+                for (int i = 0; i < TOK; ++i)
+#pragma unroll
+                    for (int j = 0; j < CH; ++j) acc[i][j] = fmaf(th[i], wv[u][j], acc[i][j]);
+            }
         }
+#pragma unroll
+        for (int u = 0; u < LD_AHEAD; ++u)
+#pragma unroll
+            for (int j = 0; j < CH; ++j) wv[u][j] = nw[u][j];
     }
 #pragma unroll
-    for (int i = 0; i < LD_TOKENS; ++i)
-        if (t0 + i < tokens) out[(size_t)(t0 + i) * C + c] = -expf(acc[i]);
+    for (int i = 0; i < TOK; ++i)
+#pragma unroll
+        for (int j = 0; j < CH; ++j)
+            if (in[j] && t0 + i < tokens) out[(size_t)(t0 + i) * C + c0 + j * LD_THREADS] = -expf(acc[i][j]);
 }
 
 #define LD_MAX_RANK 1024
+#define LD_FEW_TOKENS 16   // steps of up to so many tokens take small tiles
 // x float32 [tokens, ldx] (the first `rank` columns), w float32 [rank, C], b float32 [C], out float32 [tokens, C].
 extern "C" int vx_low_rank_decay(const float* x, int ldx, int rank, const float* w, const float* b, float* out, int tokens, int C,
                                  cudaStream_t stream) {
     if (tokens <= 0) return VX_OK;
     if (rank <= 0 || C <= 0 || ldx < rank) return VX_ERR_SHAPE;
-    if (rank > LD_MAX_RANK) return VX_ERR_LIMIT;
-    const int cols = (C + LD_THREADS - 1) / LD_THREADS;
+    if (rank > LD_MAX_RANK || (tokens + 15) / 16 > 65535) return VX_ERR_LIMIT;
     static bool conf[2][VX_MAX_DEVICES];
-    if (tokens <= 16) {
-        if (int rc = vx_configure_smem(low_rank_decay_kernel<2>, LD_MAX_RANK * 2 * sizeof(float), conf[0])) return rc;
-        VX_LAUNCH_K(VX_K_ELEMENTWISE, (low_rank_decay_kernel<2>), dim3(cols, (tokens + 1) / 2), LD_THREADS, (size_t)rank * 2 * sizeof(float),
-                    stream, x, ldx, rank, w, b, out, tokens, C);
+    if (tokens <= LD_FEW_TOKENS) {
+        if (int rc = vx_configure_smem(low_rank_decay_kernel<2, 1>, LD_MAX_RANK * 2 * sizeof(float), conf[0])) return rc;
+        VX_LAUNCH_K(VX_K_ELEMENTWISE, (low_rank_decay_kernel<2, 1>), dim3((C + LD_THREADS - 1) / LD_THREADS, (tokens + 1) / 2), LD_THREADS,
+                    (size_t)rank * 2 * sizeof(float), stream, x, ldx, rank, w, b, out, tokens, C);
     } else {
-        if (int rc = vx_configure_smem(low_rank_decay_kernel<16>, LD_MAX_RANK * 16 * sizeof(float), conf[1])) return rc;
-        if ((tokens + 15) / 16 > 65535) return VX_ERR_LIMIT;
-        VX_LAUNCH_K(VX_K_ELEMENTWISE, (low_rank_decay_kernel<16>), dim3(cols, (tokens + 15) / 16), LD_THREADS,
-                    (size_t)rank * 16 * sizeof(float), stream, x, ldx, rank, w, b, out, tokens, C);
+        if (int rc = vx_configure_smem(low_rank_decay_kernel<16, 2>, LD_MAX_RANK * 16 * sizeof(float), conf[1])) return rc;
+        VX_LAUNCH_K(VX_K_ELEMENTWISE, (low_rank_decay_kernel<16, 2>), dim3((C + 2 * LD_THREADS - 1) / (2 * LD_THREADS), (tokens + 15) / 16),
+                    LD_THREADS, (size_t)rank * 16 * sizeof(float), stream, x, ldx, rank, w, b, out, tokens, C);
     }
     VX_LAUNCH_CHECK();
     return VX_OK;

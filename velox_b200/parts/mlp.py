@@ -104,8 +104,10 @@ class DenseMLP(FeedForward):
         if h.dtype == torch.bfloat16 and ops.skinny_supported(h.shape[0], h.shape[1], h, w):
             # a decode step: W streamed once, the activation taken on the float32 sums
             return self.down(ops.gemm_skinny(h, w, None, h.dtype, activation=self.activation))
-        if h.dtype == torch.bfloat16 and h.shape[0] >= FUSED_TCGEN05_MIN_ROWS and ops.tcgen05_supported(h, w):
-            # a prompt portion: the tcgen05 product with the same epilogue
+        if (h.dtype == torch.bfloat16 and self.activation in ops.TCGEN05_ACTIVATIONS and ops.tcgen05_supported(h, w)
+                and ops.tcgen05_fills(h.shape[0], w.shape[0], h.device)):
+            # a prompt portion with tiles enough for every SM: the tcgen05 product with the same epilogue (with fewer, the
+            # library product and the activation kernel were measured faster)
             return self.down(ops.gemm_tcgen05(h, w, None, activation=self.activation))
         u = self.up(h, torch.float32)
         return self.down(ops.act(u, self.activation, out_dtype=h.dtype))

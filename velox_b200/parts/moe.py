@@ -133,7 +133,7 @@ class RoutedExperts(FeedForward):
         i, e = self.intermediate_size, self.hidden_size
         n = self.gate_up.shape[1]
         fused = dict(gated_activation=self.activation) if self.gated else dict(activation=self.activation)
-        if (self.tile or not self.gated) and ops.moe_tcgen05_supported(h, h.shape[0] * self.top, n, e) and i % 8 == 0 and e % 16 == 0:
+        if (self.tile or (not self.gated and self.activation in ops.TCGEN05_ACTIVATIONS)) and ops.moe_tcgen05_supported(h, h.shape[0] * self.top, n, e) and i % 8 == 0 and e % 16 == 0:
             # a prompt portion: the tokens' rows are copied into expert order once, and both grouped products run on
             # the tcgen05 tensor cores over row tiles of 128 (operands by TMA, the activation on the accumulators)
             plan = self._route(h, ops.MOE_TCGEN05_TILE_ROWS)
