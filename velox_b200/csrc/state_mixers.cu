@@ -330,10 +330,19 @@ __global__ void stretch_log_decay_kernel(const float* __restrict__ gate, int ldg
     const int c = blockIdx.y, i = blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= HD) return;
     float sum = 0.f;
-    for (int t = cu_stretch[c]; t < cu_stretch[c + 1]; ++t) sum += lw_log_decay(gate[(size_t)t * ldg + i], gate_mul, gate_is_log);
+    const int end = cu_stretch[c + 1];
+    for (int t = cu_stretch[c]; t < end; t += 16) {   // (sixteen tokens' reads in flight; the sum runs over the tokens in order)
+        float g[16];
+#pragma unroll
+        for (int u = 0; u < 16; ++u) g[u] = t + u < end ? gate[(size_t)(t + u) * ldg + i] : 0.f;
+#pragma unroll
+        for (int u = 0; u < 16; ++u)
+            if (t + u < end) sum += lw_log_decay(g[u], gate_mul, gate_is_log);
+    }
     log_a[(size_t)c * HD + i] = sum;
 }
 
+#define SS_AHEAD 8
 __global__ void stretch_scan_kernel(float* __restrict__ parts, float* __restrict__ state, const float* __restrict__ log_a,
                                     const float* __restrict__ decay, const int* __restrict__ cu_stretch,
                                     const int* __restrict__ first_stretch, const int* __restrict__ state_slots, int H, int D,
@@ -349,17 +358,17 @@ __global__ void stretch_scan_kernel(float* __restrict__ parts, float* __restrict
     float S = *st;
     const float l2 = decay ? log2f(decay[h]) : 0.f;
     const int last = first_stretch[seq + 1];
-    for (int c = first_stretch[seq]; c < last; c += 4) {   // (four stretches' reads in flight before the first write)
-        float loc[4], a[4];
+    for (int c = first_stretch[seq]; c < last; c += SS_AHEAD) {   // (several stretches' reads in flight before the first write)
+        float loc[SS_AHEAD], a[SS_AHEAD];
 #pragma unroll
-        for (int u = 0; u < 4; ++u) {
+        for (int u = 0; u < SS_AHEAD; ++u) {
             if (c + u >= last) continue;
             loc[u] = parts[(size_t)(c + u) * per + e];
             a[u] = log_a ? expf(log_a[(size_t)(c + u) * H * D + hd])
                          : exp2f((float)(cu_stretch[c + u + 1] - cu_stretch[c + u]) * l2);
         }
 #pragma unroll
-        for (int u = 0; u < 4; ++u) {
+        for (int u = 0; u < SS_AHEAD; ++u) {
             if (c + u >= last) continue;
             parts[(size_t)(c + u) * per + e] = S;
             S = fmaf(a[u], S, loc[u]);
