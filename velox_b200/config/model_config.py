@@ -905,3 +905,143 @@ class NegilornConfig(ModelConfig):
                 faults.append("%s.mlp.kind %r is not 'dense' or 'moe'" % (at, kind if isinstance(mlp, dict) else mlp))
         if faults:
             raise ConfigError("Negilorn configuration: " + "; ".join(faults))
+
+
+@dataclass(frozen=True)
+class BirelixConfig(ModelConfig):
+    """Birelix: a decoder whose config.json is nested and lists its layers one by one.
+
+        architecture   "Birelix"
+        vocab, width, norm.eps
+        embedding.scale  multiplier of the token's row (absent: 1)
+        layers[i]      type "latent_attention":  mixer (heads, dim, rot_dim, vdim, kv_rank, q_rank, scale, rot.base)
+                       type "attention":         mixer (heads, kv_heads, dim, vdim, scale, mask.size (the window; absent: the whole
+                                                 sequence))
+                       type "delta":             mixer (heads, kv_heads, dim, vdim, conv (taps of the short convolutions))
+                       mlp: null | kind "dense" (ff)
+                            | kind "moe" (router.experts, router.top, router.groups.{count, keep} (absent: one group),
+                                          expert.ff, expert.limit)
+
+    Every size and constant is read from there; the layers may differ from one another."""
+
+    architecture: ClassVar[str] = "Birelix"
+    model_type: ClassVar[str] = "birelix"
+    LAYER_TYPES: ClassVar[Tuple[str, ...]] = ("latent_attention", "attention", "delta")
+
+    vocab: int = _field(int)
+    width: int = _field(int)
+    norm_eps: float = _field(float)
+    embedding_scale: float = _field(float, default=1.0)
+    layers: Tuple[Dict[str, Any], ...] = _field(tuple, default=())
+
+    @classmethod
+    def from_dict(cls, raw: Dict[str, Any]) -> "BirelixConfig":
+        faults: list = []
+
+        def get(d, path, kind, default=dataclasses.MISSING):
+            cur = d
+            for key in path.split("."):
+                if not isinstance(cur, dict) or cur.get(key) is None:
+                    if default is dataclasses.MISSING:
+                        faults.append("missing key %r" % path)
+                    return None if default is dataclasses.MISSING else default
+                cur = cur[key]
+            return _typed(path, cur, kind, faults)
+
+        values = dict(vocab=get(raw, "vocab", int), width=get(raw, "width", int), norm_eps=get(raw, "norm.eps", float),
+                      embedding_scale=get(raw, "embedding.scale", float, 1.0))
+        layers = raw.get("layers")
+        if not isinstance(layers, list) or not layers:
+            faults.append("key 'layers': expected a list of layers")
+            layers = []
+        if faults:
+            raise ConfigError("config.json for %s: %s" % (cls.__name__, "; ".join(faults)))
+        cfg = cls(layers=tuple(json.loads(json.dumps(layer)) for layer in layers), **values)
+        cfg.validate()
+        return cfg
+
+    def to_dict(self) -> Dict[str, Any]:
+        return {"architecture": self.architecture, "embedding": {"scale": self.embedding_scale},
+                "layers": json.loads(json.dumps(list(self.layers))), "norm": {"eps": self.norm_eps}, "vocab": self.vocab,
+                "width": self.width}
+
+    @staticmethod
+    def window_of(mixer: Dict[str, Any]) -> int:
+        mask = mixer.get("mask")
+        return int(mask.get("size") or 0) if isinstance(mask, dict) else 0
+
+    def validate(self) -> None:
+        faults = []
+
+        def positive(where, d, *keys):
+            ok = True
+            for k in keys:
+                v = d.get(k) if isinstance(d, dict) else None
+                if not isinstance(v, int) or isinstance(v, bool) or v <= 0:
+                    faults.append("%s.%s must be a positive integer, got %r" % (where, k, v))
+                    ok = False
+            return ok
+
+        def number(where, d, key, least=None):
+            v = d.get(key) if isinstance(d, dict) else None
+            if not isinstance(v, (int, float)) or isinstance(v, bool) or (least is not None and not v > least):
+                faults.append("%s.%s must be a number%s, got %r" % (where, key, "" if least is None else " above %g" % least, v))
+                return False
+            return True
+
+        for name in ("vocab", "width"):
+            if getattr(self, name) <= 0:
+                faults.append("%s must be positive, got %d" % (name, getattr(self, name)))
+        if not self.norm_eps > 0:
+            faults.append("norm.eps must be positive, got %r" % self.norm_eps)
+        for i, layer in enumerate(self.layers):
+            at = "layers[%d]" % i
+            if not isinstance(layer, dict) or layer.get("type") not in self.LAYER_TYPES:
+                faults.append("%s.type %r is not one of %s" % (at, layer.get("type") if isinstance(layer, dict) else layer,
+                                                               list(self.LAYER_TYPES)))
+                continue
+            m, kind, where = layer.get("mixer"), layer["type"], at + ".mixer"
+            if kind == "latent_attention":
+                if positive(where, m, "heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank"):
+                    number(where, m, "scale")
+                    if m["rot_dim"] % 2:
+                        faults.append("%s.rot_dim (%d) must be even" % (where, m["rot_dim"]))
+                    if number(where + ".rot", m.get("rot"), "base", 0) and (m["rot"].get("dims") or m["rot_dim"]) != m["rot_dim"]:
+                        faults.append("%s.rot.dims must equal rot_dim" % where)
+            elif positive(where, m, "heads", "kv_heads", "dim", "vdim"):
+                if m["heads"] % m["kv_heads"]:
+                    faults.append("%s: heads (%d) is not a multiple of kv_heads (%d)" % (where, m["heads"], m["kv_heads"]))
+                if kind == "delta":
+                    positive(where, m, "conv")
+                else:
+                    number(where, m, "scale")
+                    mask = m.get("mask")
+                    if mask is not None and not isinstance(mask, dict):
+                        faults.append("%s.mask must hold a size, got %r" % (where, mask))
+                    elif mask:
+                        positive(where + ".mask", mask, "size")
+            mlp = layer.get("mlp")
+            if mlp is None:
+                continue
+            kind = mlp.get("kind") if isinstance(mlp, dict) else None
+            if kind == "dense":
+                positive(at + ".mlp", mlp, "ff")
+            elif kind == "moe":
+                if positive(at + ".mlp.expert", mlp.get("expert"), "ff"):
+                    number(at + ".mlp.expert", mlp["expert"], "limit", 0)
+                router = mlp.get("router")
+                if positive(at + ".mlp.router", router, "experts", "top"):
+                    groups = router.get("groups")
+                    if groups is None:
+                        groups = {"count": 1, "keep": 1}
+                    if positive(at + ".mlp.router.groups", groups, "count", "keep"):
+                        if router["experts"] % groups["count"] or groups["keep"] > groups["count"]:
+                            faults.append("%s.mlp.router: %d experts do not form %d equal groups of which %d are kept"
+                                          % (at, router["experts"], groups["count"], groups["keep"]))
+                        elif router["top"] > groups["keep"] * (router["experts"] // groups["count"]):
+                            faults.append("%s.mlp.router: top (%d) exceeds the experts of the kept groups (%d)"
+                                          % (at, router["top"], groups["keep"] * (router["experts"] // groups["count"])))
+            else:
+                faults.append("%s.mlp.kind %r is not 'dense' or 'moe'" % (at, kind if isinstance(mlp, dict) else mlp))
+        if faults:
+            raise ConfigError("Birelix configuration: " + "; ".join(faults))

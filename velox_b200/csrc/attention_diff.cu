@@ -94,6 +94,43 @@ __global__ void sigmoid_gate8_kernel(const bf16* __restrict__ o, int ldo, const 
     }
 }
 
+// One number per head: out[r, h V + c] = o[r, h V + c] sigmoid(g[r, h]); W columns of one head a thread.
+template <typename T, int W>
+__global__ void head_gate_kernel(const T* __restrict__ o, int ldo, const T* __restrict__ g, int ldg, T* __restrict__ out, int ldout,
+                                 long long total, int cols, int V) {
+    pdl_wait();
+    pdl_trigger();
+    for (long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (long long)gridDim.x * blockDim.x) {
+        const long long r = idx / (cols / W);
+        const int c = (int)(idx - r * (cols / W)) * W;
+        const float s = 1.f / (1.f + expf(-to_f32(g[r * ldg + c / V])));
+        struct alignas(W * sizeof(T)) Pack { T v[W]; };
+        Pack p = *reinterpret_cast<const Pack*>(o + r * ldo + c);
+#pragma unroll
+        for (int e = 0; e < W; ++e) p.v[e] = from_f32<T>(to_f32(p.v[e]) * s);
+        *reinterpret_cast<Pack*>(out + r * ldout + c) = p;
+    }
+}
+
+extern "C" int vx_head_gate(const void* o, int ldo, const void* g, int ldg, void* out, int ldout, int rows, int heads, int V,
+                            int dtype, cudaStream_t stream) {
+    if (rows <= 0 || heads <= 0 || V <= 0) return VX_OK;
+    const long long cols64 = (long long)heads * V;
+    if (cols64 > 0x7fffffffLL || ldo < cols64 || ldg < heads || ldout < cols64) return VX_ERR_SHAPE;
+    const int cols = (int)cols64;
+    if (dtype != VX_F32 && dtype != VX_BF16) return VX_ERR_DTYPE;
+    const bool wide = !((V | ldo | ldout) & (dtype == VX_F32 ? 3 : 7)) && !(((uintptr_t)o | (uintptr_t)out) & 15);
+    const long long total = (long long)rows * cols / (wide ? (dtype == VX_F32 ? 4 : 8) : 1);
+    const unsigned blocks = (unsigned)((total + 255) / 256 > 148LL * 16 ? 148LL * 16 : (total + 255) / 256);
+#define HG_GO(T_, W_) VX_LAUNCH_K(VX_K_ELEMENTWISE, (head_gate_kernel<T_, W_>), blocks, 256, 0, stream, (const T_*)o, ldo, (const T_*)g, \
+                                  ldg, (T_*)out, ldout, total, cols, V)
+    if (dtype == VX_F32) { if (wide) HG_GO(float, 4); else HG_GO(float, 1); }
+    else { if (wide) HG_GO(bf16, 8); else HG_GO(bf16, 1); }
+#undef HG_GO
+    VX_LAUNCH_CHECK();
+    return VX_OK;
+}
+
 extern "C" int vx_sigmoid_gate(const void* o, int ldo, const void* g, int ldg, void* out, int ldout, int rows, int cols,
                                int dtype, cudaStream_t stream) {
     if (rows <= 0 || cols <= 0) return VX_OK;

@@ -203,3 +203,10 @@ __device__ __forceinline__ float activation(float z, int act) {
         default: return fmaxf(z, 0.f);
     }
 }
+
+// A gated feed-forward with bounds: min(g, L) sigmoid(slope min(g, L)) (clamp(u, -L, L) + 1).
+__device__ __forceinline__ float capped_gate(float g, float u, float limit, float slope) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.f + expf(-slope * g)) * (u + 1.f);
+}

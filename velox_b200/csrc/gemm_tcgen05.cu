@@ -42,6 +42,7 @@
 #define TC_GATED 1   // act(gate) * up of paired columns
 #define TC_ACT 2     // act(.) of each column: relu or its square (of every column the exponentials of other activations,
                      // inlined 32 times, would cost more than a kernel of their own)
+#define TC_CAPPED 3  // the bounded gate of paired columns
 static bool tc_cheap_act(int act) { return act == VX_ACT_RELU || act == VX_ACT_RELU2; }
 
 template <int BN, int STAGES, int EPI>
@@ -49,7 +50,7 @@ __global__ void __launch_bounds__(TC_THREADS)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                     const float* __restrict__ bias, bf16* __restrict__ C, int M, int N, int K, int ldc, int act,
                     int* __restrict__ error, const int* __restrict__ row_tiles, const int* __restrict__ n_row_tiles,
-                    const float* __restrict__ row_scale, const int* __restrict__ src_of_row) {
+                    const float* __restrict__ row_scale, const int* __restrict__ src_of_row, float limit, float slope) {
     extern __shared__ unsigned char tc_smem_raw[];
     __shared__ __align__(8) unsigned long long full_bar[STAGES], empty_bar[STAGES], acc_full[2], acc_empty[2];
     __shared__ unsigned tmem_base_s;
@@ -181,7 +182,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 #pragma unroll
                     for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * rs);
                 }
-                if (EPI != TC_GATED) {
+                if (EPI != TC_GATED && EPI != TC_CAPPED) {
                     bf16* dst = C + (size_t)row * ldc + n0 + c0;
 #pragma unroll
                     for (int j = 0; j < 32; j += 8) {
@@ -213,7 +214,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                         for (int i = 0; i < 4; ++i) {
                             const float g0 = __uint_as_float(r[t * 16 + 2 * i]), g1 = __uint_as_float(r[t * 16 + 2 * i + 1]);
                             const float u0 = __uint_as_float(r[t * 16 + 8 + 2 * i]), u1 = __uint_as_float(r[t * 16 + 9 + 2 * i]);
-                            h[i] = __floats2bfloat162_rn(activation(g0, act) * u0, activation(g1, act) * u1);
+                            h[i] = EPI == TC_CAPPED ? __floats2bfloat162_rn(capped_gate(g0, u0, limit, slope), capped_gate(g1, u1, limit, slope))
+                                                    : __floats2bfloat162_rn(activation(g0, act) * u0, activation(g1, act) * u1);
                         }
                         *reinterpret_cast<uint4*>(dst + t * 8) = pk;
                     }
@@ -240,7 +242,7 @@ template <int BN, int STAGES, int EPI>
 static int tc_launch(const CUtensorMap& ma, const CUtensorMap& mw, const float* bias, bf16* C, int M, int N, int K,
                      int ldc, int act, int* error, cudaStream_t stream, const int* row_tiles = nullptr,
                      const int* n_row_tiles = nullptr, int max_row_tiles = 0, const float* row_scale = nullptr,
-                     const int* src_of_row = nullptr) {
+                     const int* src_of_row = nullptr, float limit = 0.f, float slope = 0.f) {
     const size_t smem = (size_t)STAGES * (TC_BM * TC_BK * 2 + BN * TC_BK * 2) + 1024;
     static bool configured[VX_MAX_DEVICES];
     if (int rc = vx_configure_smem(gemm_tcgen05_kernel<BN, STAGES, EPI>, smem, configured)) return rc;
@@ -250,7 +252,7 @@ static int tc_launch(const CUtensorMap& ma, const CUtensorMap& mw, const float* 
     const int tiles = (row_tiles ? max_row_tiles : (M + TC_BM - 1) / TC_BM) * ((N + BN - 1) / BN);
     dim3 grid(tiles < sms ? tiles : sms);
     VX_LAUNCH_K(VX_K_GEMM, (gemm_tcgen05_kernel<BN, STAGES, EPI>), grid, TC_THREADS, smem, stream, ma, mw, bias, C, M,
-                N, K, ldc, act, error, row_tiles, n_row_tiles, row_scale, src_of_row);
+                N, K, ldc, act, error, row_tiles, n_row_tiles, row_scale, src_of_row, limit, slope);
     VX_LAUNCH_CHECK();
     return VX_OK;
 }
@@ -281,27 +283,38 @@ extern "C" int vx_gemm_tcgen05(const void* A, const void* W, const float* bias, 
 // The grouped product of a routed feed-forward: A [rows, K] in group order, W [groups, N, K], row tiles of up to
 // 128 rows (group, first row, rows) whose number is on the device (at most max_row_tiles).  C [rows, N], or
 // [rows, N/2] = act(gate) * up when gated (1), act(.) of each element with gated = 2.  With row_scale (then gated is not 0)
-// row p's sums are first multiplied by row_scale[src_of_row[p]].  `wide`: tiles of 256 columns, else of 128.
-extern "C" int vx_moe_gemm_tcgen05_scaled(const void* A, const void* W, void* C, int rows, int groups, int N, int K, int lda,
+// row p's sums are first multiplied by row_scale[src_of_row[p]].  `wide`: tiles of 256 columns, else of 128.  gated 3: the
+// bounded gate of paired columns with `limit` (positive) and `slope`.
+extern "C" int vx_moe_gemm_tcgen05_capped(const void* A, const void* W, void* C, int rows, int groups, int N, int K, int lda,
                                    int ldc, int gated, int act, const int* row_tiles, const int* n_row_tiles,
                                    int max_row_tiles, int* error, const float* row_scale, const int* src_of_row,
-                                          int wide, cudaStream_t stream) {
+                                          int wide, float limit, float slope, cudaStream_t stream) {
     if ((row_scale && (!src_of_row || !gated)) || (gated == TC_ACT && !tc_cheap_act(act))) return VX_ERR_SHAPE;
     if (rows <= 0 || N <= 0 || max_row_tiles <= 0) return VX_OK;
     if (K <= 0 || (K & 7) || (N & 15) || groups <= 0 || !error || !row_tiles || !n_row_tiles) return VX_ERR_SHAPE;
     if ((lda & 7) || (ldc & 7) || lda < K) return VX_ERR_ALIGN;
     if ((((uintptr_t)A) | ((uintptr_t)W) | ((uintptr_t)C)) & 15) return VX_ERR_ALIGN;
-    if (gated < 0 || gated > TC_ACT || (gated && (act < 0 || act > VX_ACT_LAST))) return VX_ERR_SHAPE;
-    if (ldc < (gated == TC_GATED ? N / 2 : N) || (long long)groups * N > 0x7fffffffLL) return VX_ERR_SHAPE;
+    if (gated == TC_CAPPED && !(limit > 0.f)) return VX_ERR_SHAPE;
+    if (gated < 0 || gated > TC_CAPPED || (gated && (act < 0 || act > VX_ACT_LAST))) return VX_ERR_SHAPE;
+    if (ldc < (gated == TC_GATED || gated == TC_CAPPED ? N / 2 : N) || (long long)groups * N > 0x7fffffffLL) return VX_ERR_SHAPE;
     CUtensorMap ma, mw;
     if (!tc_make_map(&ma, A, rows, K, lda, TC_BM) || !tc_make_map(&mw, W, groups * N, K, K, wide ? 256 : 128)) return VX_ERR_DRIVER;
     bf16* c = (bf16*)C;
 #define TC_GO(BN_, ST_, E_)                                                                                                  \
     tc_launch<BN_, ST_, E_>(ma, mw, nullptr, c, rows, N, K, ldc, act, error, stream, row_tiles, n_row_tiles, max_row_tiles, \
-                            row_scale, src_of_row)
+                            row_scale, src_of_row, limit, slope)
+    if (gated == TC_CAPPED) return wide ? TC_GO(256, 4, TC_CAPPED) : TC_GO(128, 6, TC_CAPPED);
     if (wide) return gated == TC_GATED ? TC_GO(256, 4, TC_GATED) : (gated == TC_ACT ? TC_GO(256, 4, TC_ACT) : TC_GO(256, 4, TC_PLAIN));
     return gated == TC_GATED ? TC_GO(128, 6, TC_GATED) : (gated == TC_ACT ? TC_GO(128, 6, TC_ACT) : TC_GO(128, 6, TC_PLAIN));
 #undef TC_GO
+}
+
+extern "C" int vx_moe_gemm_tcgen05_scaled(const void* A, const void* W, void* C, int rows, int groups, int N, int K, int lda,
+                                   int ldc, int gated, int act, const int* row_tiles, const int* n_row_tiles,
+                                   int max_row_tiles, int* error, const float* row_scale, const int* src_of_row,
+                                          int wide, cudaStream_t stream) {
+    return vx_moe_gemm_tcgen05_capped(A, W, C, rows, groups, N, K, lda, ldc, gated, act, row_tiles, n_row_tiles, max_row_tiles, error,
+                                      row_scale, src_of_row, wide, 0.f, 0.f, stream);
 }
 
 extern "C" int vx_moe_gemm_tcgen05(const void* A, const void* W, void* C, int rows, int groups, int N, int K, int lda,

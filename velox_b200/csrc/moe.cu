@@ -4,8 +4,10 @@
 //             among equals), softmax over the chosen logits only; counts the tokens of every expert.
 //             Or (mode 1) scores s = softmax(logits) over ALL outputs, choice by s + correction among the
 //             outputs of the best `keep_groups` of `groups` equal groups of neighbours (a group's score:
-//             its largest choice score), weights s * route_scale, not renormalised.  The router's last
-//             Or (mode 2) scores s = sigmoid(logits), one by one, the rest as in mode 1.  The router's last
+//             its largest choice score), weights s * route_scale, not renormalised.
+//             Or (mode 2) scores s = sigmoid(logits), one by one, the rest as in mode 1.  With `group_pair` a group's score
+//             is the sum of its two largest choice scores; with `renorm` the chosen scores are divided by their sum
+//             (+ 1e-20) before route_scale.  The router's last
 //             outputs may be identity experts (no matrices: the token itself), and one more row of the
 //             router's matrix may hold the gate of a shared expert, sigmoid(w . h) per token
 //   plan      one block: where each expert's rows start in expert order, the list of row tiles
@@ -61,7 +63,7 @@ __device__ __forceinline__ void route_select(float* z, float* sc, float* gs, uns
                                              int E, int top, int* __restrict__ chosen, float* __restrict__ weight,
                                              int* __restrict__ counts, int* __restrict__ pos, int mode,
                                              const float* __restrict__ correction, int groups, int keep_groups,
-                                             float route_scale, float* __restrict__ shared_gate) {
+                                             float route_scale, float* __restrict__ shared_gate, int group_pair, int renorm) {
     if (shared_gate && lane == 0) shared_gate[t] = 1.f / (1.f + expf(-z[E]));
     if (mode >= 1) {
         float sum = 1.f;
@@ -88,8 +90,17 @@ __device__ __forceinline__ void route_select(float* z, float* sc, float* gs, uns
         if (groups > 1 && keep_groups < groups) {
             const int gsize = E / groups;
             for (int g = lane; g < groups; g += 32) {
-                float b = -INFINITY;
-                for (int e = g * gsize; e < (g + 1) * gsize; ++e) b = fmaxf(b, z[e]);
+                float b = -INFINITY, second = -INFINITY;
+                if (group_pair) {   // (by the scores: a sum of logits would rank the groups otherwise)
+                    for (int e = g * gsize; e < (g + 1) * gsize; ++e) {
+                        const float v = by_logit ? sc[e] : z[e];
+                        second = fmaxf(second, fminf(v, b));
+                        b = fmaxf(b, v);
+                    }
+                    if (gsize > 1) b += second;
+                } else {
+                    for (int e = g * gsize; e < (g + 1) * gsize; ++e) b = fmaxf(b, z[e]);
+                }
                 gs[g] = b;
                 kept[g] = 0;
             }
@@ -141,7 +152,12 @@ __device__ __forceinline__ void route_select(float* z, float* sc, float* gs, uns
         chosen[(size_t)t * top + lane] = e;
         float w;
         if (mode >= 1) {
-            w = zc[lane] * route_scale;
+            float sum = 1.f;
+            if (renorm) {
+                sum = 1e-20f;
+                for (int i = 0; i < top; ++i) sum += zc[i];
+            }
+            w = zc[lane] / sum * route_scale;
         } else {
             const float m = zc[0];
             float sum = 0.f;
@@ -160,7 +176,7 @@ __global__ void __launch_bounds__(128)
 moe_route_kernel(const T* __restrict__ h, int ldh, const float* __restrict__ w_router, const float* __restrict__ bias,
                  int tokens, int K, int E, int top, int* __restrict__ chosen, float* __restrict__ weight,
                  int* __restrict__ counts, int* __restrict__ pos, int vec, int mode, const float* __restrict__ correction,
-                 int groups, int keep_groups, float route_scale, float* __restrict__ shared_gate) {
+                 int groups, int keep_groups, float route_scale, float* __restrict__ shared_gate, int group_pair, int renorm) {
     __shared__ float z_s[4][MOE_MAX_EXPERTS + 8];
     __shared__ float zc_s[4][MOE_MAX_TOP];
     __shared__ int pick_s[4][MOE_MAX_TOP];
@@ -234,7 +250,7 @@ moe_route_kernel(const T* __restrict__ h, int ldh, const float* __restrict__ w_r
     if (!valid) return;
     __syncwarp();
     route_select(z, sc_s[warp], gs_s[warp], kept_s[warp], zc_s[warp], pick_s[warp], lane, t, E, top, chosen, weight, counts, pos, mode,
-                 correction, groups, keep_groups, route_scale, shared_gate);
+                 correction, groups, keep_groups, route_scale, shared_gate, group_pair, renorm);
 }
 
 // The same with the router's whole matrix resident in shared memory: a block brings it in once (before it waits for
@@ -251,7 +267,7 @@ __global__ void __launch_bounds__(ROUTE_R_WARPS * 32)
 moe_route_resident_kernel(const T* __restrict__ h, int ldh, const float* __restrict__ w_router, const float* __restrict__ bias,
                           int tokens, int K, int E, int top, int* __restrict__ chosen, float* __restrict__ weight,
                           int* __restrict__ counts, int* __restrict__ pos, int mode, const float* __restrict__ correction,
-                          int groups, int keep_groups, float route_scale, float* __restrict__ shared_gate) {
+                          int groups, int keep_groups, float route_scale, float* __restrict__ shared_gate, int group_pair, int renorm) {
     extern __shared__ __align__(16) float rw_s[];   // [rows][K], then per warp: z, scores, group scores, kept flags, chosen
     const int rows = E + (shared_gate ? 1 : 0);
     const int ep = route_warp_entries(rows);
@@ -316,7 +332,7 @@ moe_route_resident_kernel(const T* __restrict__ h, int ldh, const float* __restr
         __syncwarp();
         route_select(z, mine + ep, mine + 2 * ep, reinterpret_cast<unsigned char*>(mine + 3 * ep), mine + 4 * ep,
                      reinterpret_cast<int*>(mine + 4 * ep + MOE_MAX_TOP), lane, t, E, top,
-                     chosen, weight, counts, pos, mode, correction, groups, keep_groups, route_scale, shared_gate);
+                     chosen, weight, counts, pos, mode, correction, groups, keep_groups, route_scale, shared_gate, group_pair, renorm);
         __syncwarp();
     }
 }
@@ -378,12 +394,14 @@ moe_plan_kernel(const int* __restrict__ chosen, const int* __restrict__ pos, int
 // the chosen; mode 1: softmax over all, choice by score + correction within the best groups, weights score * route_scale;
 // mode 2: the same with scores sigmoid(logit).
 // With `shared_gate` the router's matrix has one more row and shared_gate[t] = sigmoid(that row . h[t]).
-extern "C" int vx_moe_route(const void* h, int ldh, const float* w_router, const float* bias, int tokens, int K, int E,
+// `group_pair`, `renorm` (modes 1 and 2): see the head of this file.
+extern "C" int vx_moe_route_groups(const void* h, int ldh, const float* w_router, const float* bias, int tokens, int K, int E,
                             int top, int tile_rows, int* chosen, float* weight, int* counts, int* pos, int* offsets,
                             int* tiles, int* n_tiles, int* src_of_row, int* row_of, int dtype, int mode,
                             const float* correction, int groups, int keep_groups, float route_scale, int identity,
-                            float* shared_gate, cudaStream_t stream) {
+                            float* shared_gate, int group_pair, int renorm, cudaStream_t stream) {
     if (tokens <= 0) return VX_OK;
+    if (mode == 0 && (group_pair || renorm)) return VX_ERR_SHAPE;
     if (K <= 0 || E <= 0 || top <= 0 || top > E || tile_rows <= 0) return VX_ERR_SHAPE;
     if (mode < 0 || mode > 2 || identity < 0 || identity >= E) return VX_ERR_SHAPE;
     if (groups < 1) groups = 1;
@@ -406,20 +424,20 @@ extern "C" int vx_moe_route(const void* h, int ldh, const float* w_router, const
         if (dtype == VX_F32)
             VX_LAUNCH_K(VX_K_ELEMENTWISE, (moe_route_resident_kernel<float>), rblocks, ROUTE_R_WARPS * 32, resident, stream,
                         (const float*)h, ldh, w_router, bias, tokens, K, E, top, chosen, weight, counts, pos, mode, correction,
-                        groups, keep_groups, route_scale, shared_gate);
+                        groups, keep_groups, route_scale, shared_gate, group_pair, renorm);
         else
             VX_LAUNCH_K(VX_K_ELEMENTWISE, (moe_route_resident_kernel<bf16>), rblocks, ROUTE_R_WARPS * 32, resident, stream,
                         (const bf16*)h, ldh, w_router, bias, tokens, K, E, top, chosen, weight, counts, pos, mode, correction,
-                        groups, keep_groups, route_scale, shared_gate);
+                        groups, keep_groups, route_scale, shared_gate, group_pair, renorm);
     } else
     if (dtype == VX_F32)
         VX_LAUNCH_K(VX_K_ELEMENTWISE, (moe_route_kernel<float>), blocks, 128, 0, stream, (const float*)h, ldh, w_router, bias,
                     tokens, K, E, top, chosen, weight, counts, pos, vec, mode, correction, groups, keep_groups, route_scale,
-                    shared_gate);
+                    shared_gate, group_pair, renorm);
     else if (dtype == VX_BF16)
         VX_LAUNCH_K(VX_K_ELEMENTWISE, (moe_route_kernel<bf16>), blocks, 128, 0, stream, (const bf16*)h, ldh, w_router, bias,
                     tokens, K, E, top, chosen, weight, counts, pos, vec, mode, correction, groups, keep_groups, route_scale,
-                    shared_gate);
+                    shared_gate, group_pair, renorm);
     else
         return VX_ERR_DTYPE;
     VX_LAUNCH_K(VX_K_ELEMENTWISE, moe_plan_kernel, 1, 1024, 0, stream, (const int*)chosen, (const int*)pos, counts,
@@ -428,11 +446,22 @@ extern "C" int vx_moe_route(const void* h, int ldh, const float* w_router, const
     return VX_OK;
 }
 
+extern "C" int vx_moe_route(const void* h, int ldh, const float* w_router, const float* bias, int tokens, int K, int E,
+                            int top, int tile_rows, int* chosen, float* weight, int* counts, int* pos, int* offsets,
+                            int* tiles, int* n_tiles, int* src_of_row, int* row_of, int dtype, int mode,
+                            const float* correction, int groups, int keep_groups, float route_scale, int identity,
+                            float* shared_gate, cudaStream_t stream) {
+    return vx_moe_route_groups(h, ldh, w_router, bias, tokens, K, E, top, tile_rows, chosen, weight, counts, pos, offsets, tiles,
+                               n_tiles, src_of_row, row_of, dtype, mode, correction, groups, keep_groups, route_scale, identity,
+                               shared_gate, 0, 0, stream);
+}
+
 // ---- grouped product on the CUDA cores: any sizes, float32 sums over k ascending ----
 // epilogues: the sums, act(gate) * up of paired columns, act(.) of each
 #define MOE_PLAIN 0
 #define MOE_GATED 1
 #define MOE_ACT 2
+#define MOE_CAPPED 3   // the bounded gate of paired columns (`capped_gate` with the launch's limit and slope)
 // the number that the row's assignment multiplies it with (1 without `row_scale`)
 __device__ __forceinline__ float moe_row_scale(const float* __restrict__ row_scale, const int* __restrict__ src_of_row, int p, bool live) {
     return row_scale && live ? row_scale[src_of_row[p]] : 1.f;
@@ -446,7 +475,7 @@ template <typename TA, typename TC>
 __global__ void __launch_bounds__(256)
 moe_gemm_simt_kernel(const TA* __restrict__ A, int lda, const int* __restrict__ src_of_row, int src_div,
                      const TA* __restrict__ W, const int* __restrict__ tiles, const int* __restrict__ n_tiles,
-                     TC* __restrict__ C, int ldc, int N, int K, int gated, int act, const float* __restrict__ row_scale) {
+                     TC* __restrict__ C, int ldc, int N, int K, int gated, int act, const float* __restrict__ row_scale, float limit, float slope) {
     pdl_wait();
     pdl_trigger();
     if ((int)blockIdx.y >= n_tiles[0]) return;
@@ -501,11 +530,11 @@ moe_gemm_simt_kernel(const TA* __restrict__ A, int lda, const int* __restrict__ 
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx + 16 * j;
             float v = acc[i][j] * rs;
-            if (gated == MOE_GATED) {
+            if (gated == MOE_GATED || gated == MOE_CAPPED) {
                 // columns come as 8 gates, then their 8 ups: the up of this thread's gate is 8 lanes on
                 const float up = __shfl_xor_sync(0xffffffffu, v, 8);
                 if (tx < 8 && r < rows && n < N)
-                    C[(size_t)(row0 + r) * ldc + (n >> 4) * 8 + tx] = from_f32<TC>(activation(v, act) * up);
+                    C[(size_t)(row0 + r) * ldc + (n >> 4) * 8 + tx] = from_f32<TC>(gated == MOE_CAPPED ? capped_gate(v, up, limit, slope) : activation(v, act) * up);
             } else if (r < rows && n < N) {
                 C[(size_t)(row0 + r) * ldc + n] = from_f32<TC>(gated == MOE_ACT ? activation(v, act) : v);
             }
@@ -529,7 +558,7 @@ template <typename TC>
 __global__ void __launch_bounds__(128)
 moe_gemm_mma_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__ src_of_row, int src_div,
                     const bf16* __restrict__ W, const int* __restrict__ tiles, const int* __restrict__ n_tiles,
-                    TC* __restrict__ C, int ldc, int N, int K, int gated, int act, const float* __restrict__ row_scale) {
+                    TC* __restrict__ C, int ldc, int N, int K, int gated, int act, const float* __restrict__ row_scale, float limit, float slope) {
     extern __shared__ __align__(16) unsigned char mt_smem[];
     typedef bf16 (*Tile)[MT_BM][MT_LD];
     Tile As = reinterpret_cast<Tile>(mt_smem);
@@ -614,15 +643,17 @@ moe_gemm_mma_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__
             if (r >= rows) continue;
             TC* crow = C + (size_t)(row0 + r) * ldc;
             const float rs = moe_row_scale(row_scale, src_of_row, row0 + r, true);
-            if (gated == MOE_GATED) {
+            if (gated == MOE_GATED || gated == MOE_CAPPED) {
 #pragma unroll
                 for (int j = 0; j < 4; j += 2) {   // n-tile j: 8 gates, n-tile j + 1: their ups
                     const int n = n0 + wn + 8 * j + 2 * (lane & 3);
 #pragma unroll
                     for (int c = 0; c < 2; ++c)
-                        if (n + c < N)
+                        if (n + c < N) {
+                            const float g = acc[i][j][2 * half + c] * rs, u = acc[i][j + 1][2 * half + c] * rs;
                             crow[((n + c) >> 4) * 8 + ((n + c) & 7)] =
-                                from_f32<TC>(activation(acc[i][j][2 * half + c] * rs, act) * (acc[i][j + 1][2 * half + c] * rs));
+                                from_f32<TC>(gated == MOE_CAPPED ? capped_gate(g, u, limit, slope) : activation(g, act) * u);
+                        }
                 }
             } else {
 #pragma unroll
@@ -651,7 +682,7 @@ template <typename TC>
 __global__ void __launch_bounds__(128)
 moe_gemm_mma16_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__ src_of_row, int src_div,
                       const bf16* __restrict__ W, const int* __restrict__ tiles, const int* __restrict__ n_tiles,
-                      TC* __restrict__ C, int ldc, int N, int K, int gated, int act, const float* __restrict__ row_scale) {
+                      TC* __restrict__ C, int ldc, int N, int K, int gated, int act, const float* __restrict__ row_scale, float limit, float slope) {
     extern __shared__ __align__(16) unsigned char ms_smem[];
     typedef bf16 (*TileA)[MS_BM][MT_LD];
     typedef bf16 (*TileW)[MT_BN][MT_LD];
@@ -724,10 +755,10 @@ moe_gemm_mma16_kernel(const bf16* __restrict__ A, int lda, const int* __restrict
 #pragma unroll
         for (int c = 0; c < 2; ++c) {
             const float v0 = acc[0][2 * half + c] * rs, v1 = acc[1][2 * half + c] * rs;
-            if (gated == MOE_GATED) {   // the warp's 16 columns: 8 gates, then their 8 ups
+            if (gated == MOE_GATED || gated == MOE_CAPPED) {   // the warp's 16 columns: 8 gates, then their 8 ups
                 if (n + c < N)
                     crow[((n + c) >> 4) * 8 + ((n + c) & 7)] =
-                        from_f32<TC>(activation(v0, act) * v1);
+                        from_f32<TC>(gated == MOE_CAPPED ? capped_gate(v0, v1, limit, slope) : activation(v0, act) * v1);
             } else {
                 if (n + c < N) crow[n + c] = from_f32<TC>(gated == MOE_ACT ? activation(v0, act) : v0);
                 if (n + 8 + c < N) crow[n + 8 + c] = from_f32<TC>(gated == MOE_ACT ? activation(v1, act) : v1);
@@ -740,13 +771,15 @@ moe_gemm_mma16_kernel(const bf16* __restrict__ A, int lda, const int* __restrict
 // 16-byte aligned rows); else the multiply-add kernel.  max_tiles bounds the tiles of any step.
 // tile_rows: 64, or 16 (tensor cores only) for steps of few tokens.  gated: 0 plain, 1 act(gate) * up, 2 act(.).
 // row_scale float32 [assignments] (with src_of_row): row p of C is formed from row_scale[src_of_row[p]] times its sums.
-extern "C" int vx_moe_gemm_scaled(const void* A, int lda, const int* src_of_row, int src_div, const void* W, const int* tiles,
+// gated 3: the bounded gate of paired columns with `limit` (positive) and `slope`.
+extern "C" int vx_moe_gemm_capped(const void* A, int lda, const int* src_of_row, int src_div, const void* W, const int* tiles,
                            const int* n_tiles, int max_tiles, void* C, int ldc, int N, int K, int gated, int act,
                            int in_dtype, int out_dtype, int tensor_cores, int tile_rows, const float* row_scale,
-                           cudaStream_t stream) {
-    if (gated < 0 || gated > MOE_ACT || (gated && (act < 0 || act > VX_ACT_LAST)) || (row_scale && !src_of_row)) return VX_ERR_SHAPE;
+                           float limit, float slope, cudaStream_t stream) {
+    if (gated < 0 || gated > MOE_CAPPED || (gated && (act < 0 || act > VX_ACT_LAST)) || (row_scale && !src_of_row)) return VX_ERR_SHAPE;
+    if (gated == MOE_CAPPED && !(limit > 0.f)) return VX_ERR_SHAPE;
     if (max_tiles <= 0 || N <= 0) return VX_OK;
-    if (K <= 0 || lda < K || src_div <= 0 || (gated == MOE_GATED && N % 16)) return VX_ERR_SHAPE;
+    if (K <= 0 || lda < K || src_div <= 0 || ((gated == MOE_GATED || gated == MOE_CAPPED) && N % 16)) return VX_ERR_SHAPE;
     if (max_tiles > 65535) return VX_ERR_LIMIT;
     if (tile_rows != MT_BM && !(tile_rows == MS_BM && tensor_cores)) return VX_ERR_SHAPE;
     dim3 grid((N + MG_BN - 1) / MG_BN, max_tiles);
@@ -758,10 +791,10 @@ extern "C" int vx_moe_gemm_scaled(const void* A, int lda, const int* src_of_row,
                                           : vx_configure_smem(moe_gemm_mma16_kernel<float>, MS_SMEM, conf_f)) return rc;
         if (out_dtype == VX_BF16)
             VX_LAUNCH_K(VX_K_GEMM, (moe_gemm_mma16_kernel<bf16>), grid, 128, MS_SMEM, stream, (const bf16*)A, lda, src_of_row,
-                        src_div, (const bf16*)W, tiles, n_tiles, (bf16*)C, ldc, N, K, gated, act, row_scale);
+                        src_div, (const bf16*)W, tiles, n_tiles, (bf16*)C, ldc, N, K, gated, act, row_scale, limit, slope);
         else if (out_dtype == VX_F32)
             VX_LAUNCH_K(VX_K_GEMM, (moe_gemm_mma16_kernel<float>), grid, 128, MS_SMEM, stream, (const bf16*)A, lda, src_of_row,
-                        src_div, (const bf16*)W, tiles, n_tiles, (float*)C, ldc, N, K, gated, act, row_scale);
+                        src_div, (const bf16*)W, tiles, n_tiles, (float*)C, ldc, N, K, gated, act, row_scale, limit, slope);
         else
             return VX_ERR_DTYPE;
     } else if (tensor_cores) {
@@ -772,25 +805,33 @@ extern "C" int vx_moe_gemm_scaled(const void* A, int lda, const int* src_of_row,
                                           : vx_configure_smem(moe_gemm_mma_kernel<float>, MT_SMEM, configured_f)) return rc;
         if (out_dtype == VX_BF16)
             VX_LAUNCH_K(VX_K_GEMM, (moe_gemm_mma_kernel<bf16>), grid, 128, MT_SMEM, stream, (const bf16*)A, lda, src_of_row, src_div,
-                        (const bf16*)W, tiles, n_tiles, (bf16*)C, ldc, N, K, gated, act, row_scale);
+                        (const bf16*)W, tiles, n_tiles, (bf16*)C, ldc, N, K, gated, act, row_scale, limit, slope);
         else if (out_dtype == VX_F32)
             VX_LAUNCH_K(VX_K_GEMM, (moe_gemm_mma_kernel<float>), grid, 128, MT_SMEM, stream, (const bf16*)A, lda, src_of_row, src_div,
-                        (const bf16*)W, tiles, n_tiles, (float*)C, ldc, N, K, gated, act, row_scale);
+                        (const bf16*)W, tiles, n_tiles, (float*)C, ldc, N, K, gated, act, row_scale, limit, slope);
         else
             return VX_ERR_DTYPE;
     } else if (in_dtype == VX_F32 && out_dtype == VX_F32)
         VX_LAUNCH_K(VX_K_GEMM, (moe_gemm_simt_kernel<float, float>), grid, 256, 0, stream, (const float*)A, lda, src_of_row,
-                    src_div, (const float*)W, tiles, n_tiles, (float*)C, ldc, N, K, gated, act, row_scale);
+                    src_div, (const float*)W, tiles, n_tiles, (float*)C, ldc, N, K, gated, act, row_scale, limit, slope);
     else if (in_dtype == VX_BF16 && out_dtype == VX_BF16)
         VX_LAUNCH_K(VX_K_GEMM, (moe_gemm_simt_kernel<bf16, bf16>), grid, 256, 0, stream, (const bf16*)A, lda, src_of_row,
-                    src_div, (const bf16*)W, tiles, n_tiles, (bf16*)C, ldc, N, K, gated, act, row_scale);
+                    src_div, (const bf16*)W, tiles, n_tiles, (bf16*)C, ldc, N, K, gated, act, row_scale, limit, slope);
     else if (in_dtype == VX_BF16 && out_dtype == VX_F32)
         VX_LAUNCH_K(VX_K_GEMM, (moe_gemm_simt_kernel<bf16, float>), grid, 256, 0, stream, (const bf16*)A, lda, src_of_row,
-                    src_div, (const bf16*)W, tiles, n_tiles, (float*)C, ldc, N, K, gated, act, row_scale);
+                    src_div, (const bf16*)W, tiles, n_tiles, (float*)C, ldc, N, K, gated, act, row_scale, limit, slope);
     else
         return VX_ERR_DTYPE;
     VX_LAUNCH_CHECK();
     return VX_OK;
+}
+
+extern "C" int vx_moe_gemm_scaled(const void* A, int lda, const int* src_of_row, int src_div, const void* W, const int* tiles,
+                           const int* n_tiles, int max_tiles, void* C, int ldc, int N, int K, int gated, int act,
+                           int in_dtype, int out_dtype, int tensor_cores, int tile_rows, const float* row_scale,
+                           cudaStream_t stream) {
+    return vx_moe_gemm_capped(A, lda, src_of_row, src_div, W, tiles, n_tiles, max_tiles, C, ldc, N, K, gated, act, in_dtype,
+                              out_dtype, tensor_cores, tile_rows, row_scale, 0.f, 0.f, stream);
 }
 
 extern "C" int vx_moe_gemm(const void* A, int lda, const int* src_of_row, int src_div, const void* W, const int* tiles,

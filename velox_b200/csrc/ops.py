@@ -11,7 +11,7 @@ from __future__ import annotations
 import ctypes
 import os
 from ctypes import c_float, c_int, c_longlong, c_void_p
-from typing import Optional
+from typing import Optional, Tuple
 
 import torch
 
@@ -136,6 +136,13 @@ def _declare(lib) -> None:
         "vx_gemm_skinny_inputs": [P, P, P, I, I, I, I, I, I, I, c_longlong, I, I, P],
         "vx_moe_gemm_scaled": [P, I, P, I, P, P, P, I, P, I, I, I, I, I, I, I, I, I, P, P],
         "vx_moe_gemm_tcgen05_scaled": [P, P, P, I, I, I, I, I, I, I, I, P, P, I, P, P, P, I, P],
+        "vx_delta_conv": [P, I, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, P],
+        "vx_delta_walk": [P, P, P, I, I, I, P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, P],
+        "vx_delta_decode": [P, I, I, P, I, I, I, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, I, I, P],
+        "vx_head_gate": [P, I, P, I, P, I, I, I, I, I, P],
+        "vx_moe_route_groups": [P, I, P, P, I, I, I, I, I, P, P, P, P, P, P, P, P, P, I, I, P, I, I, F, I, P, I, I, P],
+        "vx_moe_gemm_capped": [P, I, P, I, P, P, P, I, P, I, I, I, I, I, I, I, I, I, P, F, F, P],
+        "vx_moe_gemm_tcgen05_capped": [P, P, P, I, I, I, I, I, I, I, I, P, P, I, P, P, P, I, F, F, P],
         "vx_latent_gather_window": [P, P, I, P, P, P, P, I, P, I, I, I, I, I, I, I, P],
     }
     lib.vx_set_pdl_mask.argtypes = [I]
@@ -642,14 +649,15 @@ MOE_SCORES = {"softmax_chosen": 0, "softmax_all": 1, "sigmoid": 2}
 
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, bias, experts: int, top: int,
               tile_rows: int = MOE_TILE_ROWS, scores: str = "softmax_chosen", correction=None, groups: int = 1,
-              keep_groups: int = 1, route_scale: float = 1.0, identity: int = 0, shared_gate: bool = False) -> MoePlan:
+              keep_groups: int = 1, route_scale: float = 1.0, identity: int = 0, shared_gate: bool = False, group_pair: bool = False, renormalise: bool = False) -> MoePlan:
     """Router logits in float32, the `top` largest per token, softmax over the chosen; then every
     assignment's row in expert order and the row tiles (of up to `tile_rows` rows) of the grouped products.
 
     `experts` counts the router's outputs.  `scores="softmax_all"`: scores s = softmax over all outputs, choice by
     s + `correction` (float32 per output) among the outputs of the `keep_groups` best of `groups` equal groups of
     neighbours, weights s * route_scale (not renormalised).  The last `identity` outputs are identity experts (the
-    combination takes the token's own row for them).  `scores="sigmoid"`: the same with scores sigmoid(logit).  With `shared_gate` the router's matrix has one more row, and
+    combination takes the token's own row for them).  `scores="sigmoid"`: the same with scores sigmoid(logit).  With `group_pair` a group's score is the sum of its two
+    largest choice scores; with `renormalise` the chosen scores are divided by their sum (+ 1e-20).  With `shared_gate` the router's matrix has one more row, and
     `plan.shared_gate` [tokens] is sigmoid(that row . h)."""
     _dev(h, w_router, bias, correction)
     rows = experts + (1 if shared_gate else 0)
@@ -658,6 +666,7 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, bias, experts: int, top: 
     _need(scores in MOE_SCORES, "moe_route: scores %r" % (scores,))
     _need(groups >= 1 and experts % groups == 0 and 1 <= keep_groups <= groups and top <= keep_groups * (experts // groups)
           and 0 <= identity < experts, "moe_route: groups, kept groups, top and identity experts do not fit the outputs")
+    _need(scores != "softmax_chosen" or not (group_pair or renormalise), "moe_route: pairs of scores and renormalised weights go with scores over all outputs")
     for b in (bias, correction):
         if b is not None:
             _need(b.dtype == torch.float32 and b.numel() == experts, "moe_route: float32 bias / correction per output")
@@ -678,44 +687,52 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, bias, experts: int, top: 
         counts = torch.zeros(experts, dtype=torch.int32, device=dev)   # (the plan kernel leaves it zero again)
         if not torch.cuda.is_current_stream_capturing():
             _MOE_COUNTS[key] = counts
-    _check(library().vx_moe_route(_ptr(h), h.stride(0), _ptr(w_router), _ptr(bias), t, h.shape[1], experts, top,
+    _check(library().vx_moe_route_groups(_ptr(h), h.stride(0), _ptr(w_router), _ptr(bias), t, h.shape[1], experts, top,
                                   plan.tile_rows, _ptr(plan.chosen), _ptr(plan.weight), _ptr(counts), _ptr(pos), _ptr(offsets),
                                   _ptr(plan.tiles), _ptr(plan.n_tiles), _ptr(plan.src_of_row), _ptr(plan.row_of),
                                   dtype_code(h.dtype), MOE_SCORES[scores], _ptr(correction), int(groups),
-                                  int(keep_groups), float(route_scale), int(identity), _ptr(plan.shared_gate), _stream()),
+                                  int(keep_groups), float(route_scale), int(identity), _ptr(plan.shared_gate),
+                                         1 if group_pair else 0, 1 if renormalise else 0, _stream()),
            "moe_route")
     return plan
 
 
 def moe_gemm(a: torch.Tensor, w: torch.Tensor, plan: MoePlan, gather: bool, out_dtype: torch.dtype,
              gated_activation: Optional[str] = None, activation: Optional[str] = None,
-             row_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+             row_scale: Optional[torch.Tensor] = None, capped: Optional[Tuple[float, float]] = None) -> torch.Tensor:
     """Grouped product in expert order: row p of the result is a[src(p)] times w[expert of p] transposed, with
     w [experts, N, K]; src(p) is the token of assignment p (`gather`) or p itself.  With `gated_activation`,
     w's rows come in tiles of 8 gate rows followed by their 8 up rows and the result is act(gate) * up; with `activation` it
-    is act(.) of each sum.  `row_scale` (float32, one per assignment) multiplies an assignment's sums before either."""
+    is act(.) of each sum; with `capped` = (limit, slope) the paired rows go through the bounded gate
+    min(g, L) sigmoid(slope min(g, L)) (clamp(u, -L, L) + 1).  `row_scale` (float32, one per assignment) multiplies an
+    assignment's sums before any of them."""
     _dev(a, w, row_scale)
-    code, act = _epilogue("moe_gemm", gated_activation, activation)
+    code, act = _epilogue("moe_gemm", gated_activation, activation, capped)
+    limit, slope = capped or (0.0, 0.0)
     _need(row_scale is None or (row_scale.dtype == torch.float32 and row_scale.numel() == plan.assignments and row_scale.is_contiguous()),
           "moe_gemm: one float32 scale per assignment")
     _need(a.stride(1) == 1 and w.is_contiguous() and w.dim() == 3 and w.shape[2] == a.shape[1] and a.dtype == w.dtype,
           "moe_gemm: a [rows, K], w [experts, N, K] of one element type")
     n, k = w.shape[1], w.shape[2]
-    cols = n // 2 if gated_activation else n
+    cols = n // 2 if gated_activation or capped else n
     out = torch.empty((plan.assignments, cols), dtype=out_dtype, device=a.device)
     tc = moe_mma_supported(a, k) and w.data_ptr() % 16 == 0
     _need(plan.tile_rows == MOE_TILE_ROWS or (plan.tile_rows == MOE_SMALL_TILE_ROWS and tc),
           "moe_gemm: row tiles of %d, or of %d on the tensor cores" % (MOE_TILE_ROWS, MOE_SMALL_TILE_ROWS))
     _need(gather or row_scale is None, "moe_gemm: scales by assignment go with the product that gathers the tokens' rows")
-    _check(library().vx_moe_gemm_scaled(_ptr(a), a.stride(0), _ptr(plan.src_of_row) if gather else None, plan.top if gather else 1,
+    _check(library().vx_moe_gemm_capped(_ptr(a), a.stride(0), _ptr(plan.src_of_row) if gather else None, plan.top if gather else 1,
                                         _ptr(w), _ptr(plan.tiles), _ptr(plan.n_tiles), plan.max_tiles, _ptr(out), cols, n, k,
                                         code, act, dtype_code(a.dtype), dtype_code(out_dtype), 1 if tc else 0, plan.tile_rows,
-                                        _ptr(row_scale), _stream()), "moe_gemm")
+                                        _ptr(row_scale), float(limit), float(slope), _stream()), "moe_gemm")
     return out
 
 
-def _epilogue(what: str, gated_activation: Optional[str], activation: Optional[str]):
-    """(epilogue code, activation code) of a matrix product: plain, act(gate) * up of paired rows, or act(.)."""
+def _epilogue(what: str, gated_activation: Optional[str], activation: Optional[str], capped=None):
+    """(epilogue code, activation code) of a matrix product: plain, act(gate) * up of paired rows, act(.), or the bounded
+    gate of paired rows."""
+    if capped is not None:
+        _need(gated_activation is None and activation is None and capped[0] > 0, "%s: a bounded gate stands alone and has a positive limit" % what)
+        return 3, 0
     _need(gated_activation is None or activation is None, "%s: a gated activation or a plain one" % what)
     name = gated_activation or activation
     _need(name is None or name in ACTIVATIONS, "%s: unknown activation %r" % (what, name))
@@ -750,12 +767,14 @@ def moe_gather_rows(x: torch.Tensor, plan: MoePlan) -> torch.Tensor:
 
 
 def moe_gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, plan: MoePlan, gated_activation: Optional[str] = None,
-                     activation: Optional[str] = None, row_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     activation: Optional[str] = None, row_scale: Optional[torch.Tensor] = None,
+                     capped: Optional[Tuple[float, float]] = None) -> torch.Tensor:
     """The grouped product on the tcgen05 tensor cores: `a` [assignments, K] bfloat16 IN EXPERT ORDER, w [experts, N, K];
-    the plan's row tiles must be of `MOE_TCGEN05_TILE_ROWS` rows.  bfloat16 out.  `activation` and `row_scale` as in
-    `moe_gemm`."""
+    the plan's row tiles must be of `MOE_TCGEN05_TILE_ROWS` rows.  bfloat16 out.  `activation`, `row_scale` and
+    `capped` as in `moe_gemm`."""
     _dev(a, w, row_scale)
-    code, act = _epilogue("moe_gemm_tcgen05", gated_activation, activation)
+    code, act = _epilogue("moe_gemm_tcgen05", gated_activation, activation, capped)
+    limit, slope = capped or (0.0, 0.0)
     _need(activation is None or activation in TCGEN05_ACTIVATIONS, "moe_gemm_tcgen05: a plain activation is one of %s" % (TCGEN05_ACTIVATIONS,))
     _need(row_scale is None or (code and row_scale.dtype == torch.float32 and row_scale.numel() == plan.assignments),
           "moe_gemm_tcgen05: one float32 scale per assignment, with an activation")
@@ -763,14 +782,14 @@ def moe_gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, plan: MoePlan, gated_acti
           and a.shape == (plan.assignments, w.shape[2]) and plan.tile_rows == MOE_TCGEN05_TILE_ROWS,
           "moe_gemm_tcgen05: bfloat16 a [assignments, K] in expert order, w [experts, N, K], row tiles of 128")
     n, k = w.shape[1], w.shape[2]
-    cols = n // 2 if gated_activation else n
+    cols = n // 2 if gated_activation or capped else n
     out = torch.empty((plan.assignments, cols), dtype=torch.bfloat16, device=a.device)
     # (how many row tiles the experts' shares fill is on the device; half a tile more per expert on the average)
     wide = tcgen05_wide_better(-(-plan.assignments // MOE_TCGEN05_TILE_ROWS) + w.shape[0] // 2, n, a.device)
-    _check(library().vx_moe_gemm_tcgen05_scaled(_ptr(a), _ptr(w), _ptr(out), plan.assignments, w.shape[0], n, k, a.stride(0), cols,
+    _check(library().vx_moe_gemm_tcgen05_capped(_ptr(a), _ptr(w), _ptr(out), plan.assignments, w.shape[0], n, k, a.stride(0), cols,
                                                 code, act, _ptr(plan.tiles), _ptr(plan.n_tiles), plan.max_tiles,
                                                 _ptr(_error_word(a.device)), _ptr(row_scale),
-                                                _ptr(plan.src_of_row) if row_scale is not None else None, 1 if wide else 0, _stream()),
+                                                _ptr(plan.src_of_row) if row_scale is not None else None, 1 if wide else 0, float(limit), float(slope), _stream()),
            "moe_gemm_tcgen05")
     note_bounded_wait()
     return out
@@ -1289,6 +1308,18 @@ def sigmoid_gate(o: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
     return out
 
 
+def head_gate(o: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
+    """Every head of o [rows, heads * size] times sigmoid of its number in `gate` [rows, heads]; rows may be strided."""
+    _dev(o, gate)
+    heads = gate.shape[1]
+    _need(o.dim() == 2 and gate.dim() == 2 and o.shape[0] == gate.shape[0] and o.shape[1] % heads == 0 and o.dtype == gate.dtype
+          and o.stride(1) == 1 and gate.stride(1) == 1, "head_gate: o [rows, heads * size] and gate [rows, heads] of one type")
+    out = torch.empty(tuple(o.shape), dtype=o.dtype, device=o.device)
+    _check(library().vx_head_gate(_ptr(o), o.stride(0), _ptr(gate), gate.stride(0), _ptr(out), out.stride(0), o.shape[0], heads,
+                                  o.shape[1] // heads, dtype_code(o.dtype), _stream()), "head_gate")
+    return out
+
+
 def capped_gated_act(sums: torch.Tensor, bias: Optional[torch.Tensor], limit: float, slope: float,
                      out_dtype: torch.dtype) -> torch.Tensor:
     """sums float32 [rows, 2 inner] (all gates, then all ups), `bias` float32 [2 inner] added first:
@@ -1399,6 +1430,75 @@ def low_rank_decay(x: torch.Tensor, weight_t: torch.Tensor, bias: torch.Tensor) 
     out = torch.empty((x.shape[0], c), dtype=torch.float32, device=x.device)
     _check(library().vx_low_rank_decay(_ptr(x), x.stride(0), rank, _ptr(weight_t), _ptr(bias), _ptr(out), x.shape[0], c, _stream()),
            "low_rank_decay")
+    return out
+
+
+DELTA_MAX_DIM = 256      # key channels of a head that the delta rule's kernels take
+DELTA_MAX_VDIM = 4096
+DELTA_MAX_TAPS = 64
+_DELTA_DOTS = 8
+
+
+def _delta_check(what, x, taps_w, ring, groups, dim, heads, vdim, ab):
+    c = 2 * groups * dim + heads * vdim
+    taps = taps_w.shape[0]
+    _need(x.stride(1) == 1 and x.shape[1] >= c and tuple(taps_w.shape) == (taps, c) and taps_w.dtype == torch.float32 and taps_w.is_contiguous(),
+          "%s: rows with q, k and v, float32 taps [taps, channels]" % what)
+    _need(ring.dtype == torch.float32 and ring.is_contiguous() and tuple(ring.shape[1:]) == (taps, c), "%s: float32 ring [slots, taps, channels]" % what)
+    _need(ab.dtype == torch.float32 and ab.stride(1) == 1 and ab.shape[0] == x.shape[0], "%s: float32 rows with a and b" % what)
+    return c, taps
+
+
+def _delta_state_check(what, state, heads, dim, vdim, *per_head):
+    _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, vdim, dim),
+          "%s: float32 state [slots, heads, vdim, dim]" % what)
+    for v in per_head:
+        _need(v.dtype == torch.float32 and v.is_contiguous() and v.numel() == heads, "%s: float32 numbers per head" % what)
+
+
+def delta_rule(x: torch.Tensor, ab: torch.Tensor, a_col: int, b_col: int, taps_w: torch.Tensor, neg_exp_a: torch.Tensor,
+               dt_bias: torch.Tensor, state: torch.Tensor, ring: torch.Tensor, ctx, groups: int, dim: int, heads: int, vdim: int,
+               q_mul: float) -> torch.Tensor:
+    """The gated delta rule over every request's tokens in order.  x [tokens, ..]: the projections q [groups, dim], k [groups,
+    dim], v [heads, vdim] from column 0 on; each goes through a causal convolution over time (`taps_w` float32 [taps,
+    channels], the last row being the current token's) and silu, q and k become unit vectors per head, q times `q_mul`.
+    Per head S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q with g = exp(neg_exp_a softplus(a + dt_bias)) and
+    beta = sigmoid(b); a and b of head h: columns a_col + h and b_col + h of `ab` (float32).  `state` float32 [slots, heads,
+    vdim, dim] and `ring` float32 [slots, taps, channels] (the convolutions' last inputs, position p in row p mod taps) are
+    read and written.  Returns float32 [tokens, heads * vdim]."""
+    _dev(x, ab, taps_w, neg_exp_a, dt_bias, state, ring)
+    c, taps = _delta_check("delta_rule", x, taps_w, ring, groups, dim, heads, vdim, ab)
+    _delta_state_check("delta_rule", state, heads, dim, vdim, neg_exp_a, dt_bias)
+    tokens, dev = x.shape[0], x.device
+    y = torch.empty((tokens, c), dtype=torch.float32, device=dev)
+    dots = torch.empty((tokens, groups, _DELTA_DOTS), dtype=torch.float32, device=dev)
+    out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=dev)
+    _check(library().vx_delta_conv(_ptr(x), x.stride(0), _ptr(taps_w), _ptr(ring), _ptr(ctx.seq_of_token), _ptr(ctx.cu_seqlens),
+                                   _ptr(ctx.state_slots), _ptr(ctx.positions), _ptr(y), _ptr(dots), tokens, groups, dim, heads,
+                                   vdim, taps, float(q_mul), dtype_code(x.dtype), _stream()), "delta_conv")
+    _check(library().vx_delta_walk(_ptr(y), _ptr(dots), _ptr(ab), ab.stride(0), int(a_col), int(b_col), _ptr(neg_exp_a),
+                                   _ptr(dt_bias), _ptr(state), _ptr(ring), _ptr(x), x.stride(0), _ptr(ctx.cu_seqlens),
+                                   _ptr(ctx.state_slots), _ptr(ctx.positions), _ptr(out), ctx.n_seqs, groups, dim, heads, vdim,
+                                   taps, dtype_code(x.dtype), _stream()), "delta_walk")
+    return out
+
+
+def delta_decode(x: torch.Tensor, g_col: int, ab: torch.Tensor, a_col: int, b_col: int, taps_w: torch.Tensor,
+                 neg_exp_a: torch.Tensor, dt_bias: torch.Tensor, norm_weight: torch.Tensor, state: torch.Tensor, ring: torch.Tensor,
+                 ctx, groups: int, dim: int, heads: int, vdim: int, q_mul: float, eps: float, out_dtype: torch.dtype) -> torch.Tensor:
+    """`delta_rule` for a step of single tokens (row t is request t's), and what follows it: every head's output divided by
+    its root mean square, times `norm_weight` [vdim], times silu of the gates [heads, vdim] at column `g_col` of x.  In
+    `out_dtype`.  `state` and `ring` must be older than x: not what the kernel launched just before this one writes (they are
+    read before that one has finished)."""
+    _dev(x, ab, taps_w, neg_exp_a, dt_bias, norm_weight, state, ring)
+    _, taps = _delta_check("delta_decode", x, taps_w, ring, groups, dim, heads, vdim, ab)
+    _delta_state_check("delta_decode", state, heads, dim, vdim, neg_exp_a, dt_bias)
+    _need(norm_weight.dtype == torch.float32 and norm_weight.numel() == vdim and x.shape[0] == ctx.n_seqs, "delta_decode: float32 norm weight [vdim], a row per request")
+    out = torch.empty((x.shape[0], heads * vdim), dtype=out_dtype, device=x.device)
+    _check(library().vx_delta_decode(_ptr(x), x.stride(0), int(g_col), _ptr(ab), ab.stride(0), int(a_col), int(b_col), _ptr(taps_w),
+                                     _ptr(neg_exp_a), _ptr(dt_bias), _ptr(norm_weight), _ptr(state), _ptr(ring), _ptr(ctx.state_slots),
+                                     _ptr(ctx.positions), _ptr(out), x.shape[0], groups, dim, heads, vdim, taps, float(q_mul), float(eps),
+                                     dtype_code(x.dtype), dtype_code(out_dtype), _stream()), "delta_decode")
     return out
 
 

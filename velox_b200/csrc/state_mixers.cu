@@ -602,9 +602,7 @@ __global__ void capped_gated_act_kernel(const float* __restrict__ sums, const fl
         const int c = (int)(i - r * inner);
         float g = sums[r * 2 * inner + c], u = sums[r * 2 * inner + inner + c];
         if (bias) { g += bias[c]; u += bias[inner + c]; }
-        g = fminf(g, limit);
-        u = fminf(fmaxf(u, -limit), limit);
-        out[i] = from_f32<T>(g / (1.f + expf(-slope * g)) * (u + 1.f));
+        out[i] = from_f32<T>(capped_gate(g, u, limit, slope));
     }
 }
 

@@ -3,6 +3,7 @@ from .base import (Block, BorrowedCache, CacheParts, Embedding, FeedForward, Fix
                    TensorSpec)
 from .block import (HyperConnectionBlock, ParallelSublayersBlock, PendingStreams, PendingSum, PostNormBlock, PreNormBlock,
                     SandwichNormBlock, TokenShiftBlock)
+from .delta_rule import GatedDeltaRule
 from .differential_attention import DifferentialAttention
 from .embedding import OutputHead, PairHashEmbedding, TokenEmbedding
 from .linear import Linear, matmul
@@ -24,6 +25,7 @@ register_part("mixer", "gated_linear_attention", GatedLinearAttention)
 register_part("mixer", "latent_attention", LatentAttention)
 register_part("mixer", "parallel", ParallelMixer)
 register_part("mixer", "wkv", WkvMixer)
+register_part("mixer", "gated_delta_rule", GatedDeltaRule)
 register_part("mixer", "differential_attention", DifferentialAttention)
 register_part("feed_forward", "gated_mlp", GatedMLP)
 register_part("feed_forward", "dense_mlp", DenseMLP)

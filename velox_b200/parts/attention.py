@@ -42,6 +42,9 @@ floor(i / C) = floor(j / C)); `sink_value` (a sink whose score is this number fo
 the denominator); `own_kv=False` (the layer has no keys and values of its own: its queries read the cache of the layer that
 its plan names with `cache_of`).  `reader_chunks` lists the chunks of the layers that read this one's cache, which keeps
 what the longest of them still sees.
+
+`bias_suffix` names the projections' biases (a matrix's name plus the suffix) and `out_bias=False` leaves the output
+projection without one; `qk_norm_weight=False` norms q and k without a weight (each head divided by its root mean square).
 """
 from __future__ import annotations
 
@@ -82,8 +85,10 @@ class PagedAttention(Mixer):
                  norm_names: Sequence[str] = ("q_norm.weight", "k_norm.weight"), sink: bool = False,
                  output_gate: bool = False, sink_name: str = "sink", gate_name: str = "g", score_softcap: float = 0.0,
                  weights_32bit: bool = False, chunk: int = 0, sink_value: Optional[float] = None, own_kv: bool = True,
-                 reader_chunks: Sequence[int] = ()):
+                 reader_chunks: Sequence[int] = (),
+                 bias_suffix: Optional[str] = None, out_bias: bool = True, qk_norm_weight: bool = True):
         super().__init__(prefix)
+        self.bias_suffix, self.out_bias, self.qk_norm_weight = bias_suffix, bool(bias and out_bias), bool(qk_norm_weight)
         self.chunk, self.own_kv, self.reader_chunks = int(chunk), bool(own_kv), tuple(int(c) for c in reader_chunks)
         self.sink_value = None if sink_value is None else float(sink_value)
         if self.chunk < 0 or (self.chunk and keep_first):
@@ -133,6 +138,9 @@ class PagedAttention(Mixer):
     def _w(self, name: str) -> str:
         return self.prefix + self.names[name]
 
+    def _b(self, name: str) -> str:
+        return self.prefix + name + ".bias" if self.bias_suffix is None else self._w(name) + self.bias_suffix
+
     @property
     def extended(self) -> bool:
         """True if the layer uses what only the kernels for biased, unequal or kept-first attention know."""
@@ -148,15 +156,15 @@ class PagedAttention(Mixer):
         return sum(self._proj_rows().values())
 
     def tensor_specs(self) -> List[TensorSpec]:
-        p, specs = self.prefix, []
+        specs = []
         for name, rows in self._proj_rows().items():
             specs.append(TensorSpec(self._w(name), (rows, self.hidden_size), "matrix"))
             if self.bias:
-                specs.append(TensorSpec(p + name + ".bias", (rows,), "bias"))
+                specs.append(TensorSpec(self._b(name), (rows,), "bias"))
         specs.append(TensorSpec(self._w("o_proj"), (self.hidden_size, self.num_heads * self.v_head_dim), "matrix"))
-        if self.bias:
-            specs.append(TensorSpec(p + "o_proj.bias", (self.hidden_size,), "bias"))
-        if self.qk_norm:
+        if self.out_bias:
+            specs.append(TensorSpec(self._b("o_proj"), (self.hidden_size,), "bias"))
+        if self.qk_norm and self.qk_norm_weight:
             specs.append(TensorSpec(self.norm_names[0], (self.head_dim,), "norm"))
             if self.own_kv:
                 specs.append(TensorSpec(self.norm_names[1], (self.head_dim,), "norm"))
@@ -173,9 +181,8 @@ class PagedAttention(Mixer):
 
     def bind(self, tensors: Dict[str, torch.Tensor], runtime: Runtime) -> None:
         super().bind(tensors, runtime)
-        p = self.prefix
         mats = [tensors[self._w(n)] for n in self._proj_rows()]
-        biases = [tensors[p + n + ".bias"] for n in self._proj_rows()] if self.bias else None
+        biases = [tensors[self._b(n)] for n in self._proj_rows()] if self.bias else None
         if self.output_gate:
             # the gates' rows, then zero rows up to a multiple of 8 (rows of the projection stay 16-byte aligned)
             g = tensors[self.gate_name]
@@ -191,8 +198,11 @@ class PagedAttention(Mixer):
             self.sinks = tensors[self.sink_name].to(torch.float32).contiguous()
         elif self.sink_value is not None:
             self.sinks = torch.full((self.num_heads,), self.sink_value, dtype=torch.float32, device=runtime.device)
-        self.out = Linear(tensors[self._w("o_proj")], tensors[p + "o_proj.bias"] if self.bias else None)
-        if self.qk_norm:
+        self.out = Linear(tensors[self._w("o_proj")], tensors[self._b("o_proj")] if self.out_bias else None)
+        if self.qk_norm and not self.qk_norm_weight:   # (the kernels read a multiplier per channel)
+            self.q_norm_weight = torch.ones(self.head_dim, dtype=torch.float32, device=runtime.device)
+            self.k_norm_weight = self.q_norm_weight if self.own_kv else None
+        elif self.qk_norm:
             self.q_norm_weight = tensors[self.norm_names[0]]
             self.k_norm_weight = tensors[self.norm_names[1]] if self.own_kv else None
         if self.position is not None:

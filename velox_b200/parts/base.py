@@ -40,6 +40,7 @@ class TensorSpec:
       bias:          N(0, 0.02); held in float32
       matrix_f32:    N(0, 0.02); held in float32 whatever the engine's element type (a router)
       share:         uniform in [0, 1); held in float32 (how far a channel is moved towards the token before it)
+      taps:          N(0, 0.5); held in float32 (a short convolution over time, [channels, taps])
       mixing:        identity + N(0, 0.05), square; held in float32 (how the copies of a stream are mixed)
       int_table:     integers; held as int32
     A dimension of -1 is left open: the file's tensor decides it, and the part reads it off when it binds."""

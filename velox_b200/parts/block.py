@@ -2,6 +2,7 @@
 
 `PreNormBlock`, the reference's decoder layer (src/paged/qwen3.rs:932-939):
     h = norm1(x); x = x + mixer(h); h = norm2(x); x = x + feed_forward(h)
+(the last two fall away in a layer without a feed-forward).
 
 The residual stream x is float32.  A sublayer's output is not added at once:
 it travels as `delta` to the next norm, whose kernel forms x + delta in float32,
@@ -76,11 +77,17 @@ class PendingSum:
 
 
 class PreNormBlock(Block):
-    norm_names = ("mixer", "feed_forward")
+    needs_feed_forward = False
+
+    def __init__(self, mixer, feed_forward, norms):
+        self.norm_names = ("mixer",) + (("feed_forward",) if feed_forward is not None else ())
+        super().__init__(mixer, feed_forward, norms)
 
     def forward(self, residual, delta, ctx, cache):
         h = self.norms["mixer"].add_norm(residual, delta)
         a = self.mixer.forward(h, ctx, cache)
+        if self.feed_forward is None:
+            return residual, a
         h = self.norms["feed_forward"].add_norm(residual, a)
         f = self.feed_forward.forward(h, ctx)
         return residual, f

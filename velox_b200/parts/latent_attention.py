@@ -24,7 +24,7 @@ layer's eps); W_dq rides in the fused projection and W_uq is a second product;
 raised way gathers and raises only the rows from the window of the step's first query on (`cache_window`, at least
 `window`, is how long the cache keeps a row: the longest window of this layer and of the layers that borrow its rows);
 `output_gate`: the joined heads are multiplied element by element by sigmoid(W_g h) before the output projection; W_g rides
-in the fused projection;
+in the fused projection; with `head_gate` W_g has one row per head and a head's whole output is multiplied by sigmoid(W_g h)_head;
 `own_rows=False`: the layer has no W_dkv and no norm weight of its own and reads the rows that another layer wrote (the
 plan's `cache_of`), with its own W_uk, W_uv, queries and window.
 """
@@ -53,10 +53,13 @@ class LatentAttention(Mixer):
     def __init__(self, prefix: str, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, v_head_dim: int,
                  kv_rank: int, scale: float, position: PartSpec, eps: float = 1e-6,
                  names: Sequence[str] = ("q", "dkv", "dkv.norm", "uk", "uv", "o"), q_rank: int = 0, window: int = 0,
-                 cache_window: Optional[int] = None, output_gate: bool = False, own_rows: bool = True,
+                 cache_window: Optional[int] = None, output_gate: bool = False, own_rows: bool = True, head_gate: bool = False,
                  query_names: Sequence[str] = ("dq", "dq.norm", "uq"), gate_name: str = "g"):
         super().__init__(prefix)
         self.q_rank, self.window, self.output_gate, self.own_rows = int(q_rank), int(window), bool(output_gate), bool(own_rows)
+        self.head_gate = bool(head_gate)
+        if self.output_gate and self.head_gate:
+            raise ValueError("%sa gate element by element or one per head, not both" % prefix)
         self.cache_window = self.window if cache_window is None else int(cache_window)
         if self.q_rank < 0 or self.window < 0 or (self.cache_window and self.cache_window < self.window) \
                 or (self.window == 0 and self.cache_window):
@@ -102,6 +105,8 @@ class LatentAttention(Mixer):
             specs += [TensorSpec(n["dkv"], (self.row, e), "matrix"), TensorSpec(n["norm"], (self.kv_rank,), "norm")]
         if self.output_gate:
             specs.append(TensorSpec(self.gate_name, (H * self.v_head_dim, e), "matrix"))
+        if self.head_gate:
+            specs.append(TensorSpec(self.gate_name, (H, e), "matrix"))
         return specs + [TensorSpec(n["uk"], (H * self.head_dim, self.kv_rank), "matrix"),
                         TensorSpec(n["uv"], (H * self.v_head_dim, self.kv_rank), "matrix"),
                         TensorSpec(n["o"], (e, H * self.v_head_dim), "matrix")] + self.position.tensor_specs()
@@ -114,7 +119,7 @@ class LatentAttention(Mixer):
         mats, self.cols, at = [], {}, 0
         first = tensors[self.query_names[0]] if self.q_rank else tensors[n["q"]]
         for key, w in (("q", first), ("dkv", tensors[n["dkv"]] if self.own_rows else None),
-                       ("g", tensors[self.gate_name] if self.output_gate else None)):
+                       ("g", tensors[self.gate_name] if self.output_gate or self.head_gate else None)):
             if w is None:
                 continue
             self.cols[key] = at
@@ -148,9 +153,11 @@ class LatentAttention(Mixer):
         return PagedLatent(self.row, self.cache_window)
 
     def _gated(self, o: torch.Tensor, x: torch.Tensor) -> torch.Tensor:
-        if not self.output_gate:
+        if not (self.output_gate or self.head_gate):
             return o
         g = self.cols["g"]
+        if self.head_gate:
+            return ops.head_gate(o, x[:, g:g + self.num_heads])
         return ops.sigmoid_gate(o, x[:, g:g + o.shape[1]])
 
     def forward(self, h: torch.Tensor, ctx, cache) -> torch.Tensor:

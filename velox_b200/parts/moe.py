@@ -7,14 +7,16 @@ A second way of routing, `scores="softmax_all"`: s = softmax(z) over ALL the rou
 s + correction (a stored vector that moves the choice and not the weights), restricted to the outputs of the
 `keep_groups` best of `groups` equal groups of neighbouring outputs (a group's score is its largest choice score);
 the weights are the chosen s times `route_scale`, not renormalised.  A third, `scores="sigmoid"`, is the second with
-s = sigmoid(z), output by output.  The router's last `identity` outputs are
+s = sigmoid(z), output by output.  With `group_pair` a group is judged by the sum of its two largest choice scores; with
+`renormalise` the chosen scores are divided by their sum (+ 1e-20).  The router's last `identity` outputs are
 identity experts: they have no matrices and return the token itself (times the weight).  With `shared_gate_name`
 the shared feed-forward's output is multiplied by sigmoid(w . h), one number per token; w is a stored [1, hidden]
 matrix that rides as one more row of the router's matrix.
 
 With `gated=False` an expert is down(act(up(h))): two matrices, `names` = (up, down).  With `weight_input` an
 assignment's weight multiplies what its expert reads instead of what it returns, sum_e expert_e(w_e h): the first product
-is linear, so the kernels multiply its float32 sums before the activation.
+is linear, so the kernels multiply its float32 sums before the activation.  With `capped` = (limit, slope) an expert's
+activation is the bounded gate min(g, limit) sigmoid(slope min(g, limit)) (clamp(u, -limit, limit) + 1).
 
 Nothing of a step comes back to the host: the router kernel leaves the assignments on the device, a plan
 kernel orders them by expert, and two grouped matrix products (gate and up with the activation on their
@@ -46,9 +48,14 @@ class RoutedExperts(FeedForward):
                  router_names: Sequence[str] = ("router", "router.b"), expert_prefix: str = "e%d.",
                  names: Sequence[str] = ("gate", "up", "down"), scores: str = "softmax_chosen",
                  correction_name: Optional[str] = None, groups: int = 1, keep_groups: int = 1, route_scale: float = 1.0,
-                 identity: int = 0, shared_gate_name: Optional[str] = None, gated: bool = True, weight_input: bool = False):
+                 identity: int = 0, shared_gate_name: Optional[str] = None, gated: bool = True, weight_input: bool = False,
+                 group_pair: bool = False, renormalise: bool = False, capped: Optional[Sequence[float]] = None):
         super().__init__(prefix)
         self.gated, self.weight_input = bool(gated), bool(weight_input)
+        self.group_pair, self.renormalise = bool(group_pair), bool(renormalise)
+        self.capped = None if capped is None else (float(capped[0]), float(capped[1]))
+        if self.capped is not None and (not self.gated or not self.capped[0] > 0):
+            raise ValueError("%sa bounded gate has a gate's matrix and a positive limit; got %r" % (prefix, capped))
         if len(names) != (3 if self.gated else 2):
             raise ValueError("%san expert %s a gate has %d matrices, got the names %s"
                              % (prefix, "with" if self.gated else "without", 3 if self.gated else 2, list(names)))
@@ -61,8 +68,8 @@ class RoutedExperts(FeedForward):
         self.scores, self.route_scale = scores, float(route_scale)
         if scores not in ops.MOE_SCORES:
             raise ValueError("%sscores %r is not one of %s" % (prefix, scores, ", ".join(ops.MOE_SCORES)))
-        if scores == "softmax_chosen" and (correction_name or self.groups != 1 or self.route_scale != 1.0):
-            raise ValueError("%sa correction, groups and a multiplier of the weights go with scores over all outputs" % prefix)
+        if scores == "softmax_chosen" and (correction_name or self.groups != 1 or self.route_scale != 1.0 or self.group_pair or self.renormalise):
+            raise ValueError("%sa correction, groups, renormalised weights and a multiplier of the weights go with scores over all outputs" % prefix)
         if self.experts <= 0 or self.identity < 0 or not 0 < self.top <= self.outputs:
             raise ValueError("%stop %d of %d experts and %d identity experts" % (prefix, self.top, self.experts, self.identity))
         if self.groups < 1 or self.outputs % self.groups or not 1 <= self.keep_groups <= self.groups \
@@ -127,12 +134,15 @@ class RoutedExperts(FeedForward):
         return ops.moe_route(h, self.router, self.bias, self.outputs, self.top, tile_rows, scores=self.scores,
                              correction=self.correction, groups=self.groups, keep_groups=self.keep_groups,
                              route_scale=self.route_scale, identity=self.identity,
-                             shared_gate=self.shared_gate_name is not None)
+                             shared_gate=self.shared_gate_name is not None, group_pair=self.group_pair,
+                             renormalise=self.renormalise)
 
     def forward(self, h: torch.Tensor, ctx=None) -> torch.Tensor:
         i, e = self.intermediate_size, self.hidden_size
         n = self.gate_up.shape[1]
         fused = dict(gated_activation=self.activation) if self.gated else dict(activation=self.activation)
+        if self.capped is not None:
+            fused = dict(capped=self.capped)
         if (self.tile or (not self.gated and self.activation in ops.TCGEN05_ACTIVATIONS)) and ops.moe_tcgen05_supported(h, h.shape[0] * self.top, n, e) and i % 8 == 0 and e % 16 == 0:
             # a prompt portion: the tokens' rows are copied into expert order once, and both grouped products run on
             # the tcgen05 tensor cores over row tiles of 128 (operands by TMA, the activation on the accumulators)
@@ -148,7 +158,11 @@ class RoutedExperts(FeedForward):
             a = ops.moe_gemm(h, self.gate_up, plan, True, h.dtype, row_scale=self._scale(plan), **fused)
         else:
             # an inner size that is no multiple of 8: all gates, then all ups; the activation by a kernel of its own
-            a = ops.gated_act(ops.moe_gemm(h, self.gate_up, plan, True, torch.float32, row_scale=self._scale(plan)), self.activation, 0, out_dtype=h.dtype)
+            sums = ops.moe_gemm(h, self.gate_up, plan, True, torch.float32, row_scale=self._scale(plan))
+            if self.capped is not None:
+                a = ops.capped_gated_act(sums, None, *self.capped, h.dtype)
+            else:
+                a = ops.gated_act(sums, self.activation, 0, out_dtype=h.dtype)
         y = ops.moe_gemm(a, self.down, plan, False, torch.float32)
         shared = self.shared.forward(h, ctx) if self.shared is not None else None
         return ops.moe_combine(y, plan, shared, h.dtype, h=h, weighted=not self.weight_input)

@@ -50,7 +50,7 @@ _INTS = (torch.int32, torch.int64, torch.int16, torch.int8, torch.uint8)
 def held_dtype(role: str, stored: torch.dtype, runtime: Runtime) -> torch.dtype:
     if role == "int_table":
         return torch.int32
-    if role in ("norm", "bias", "matrix_f32", "mixing", "share"):
+    if role in ("norm", "bias", "matrix_f32", "mixing", "share", "taps"):
         return torch.float32
     return runtime.dtype
 
