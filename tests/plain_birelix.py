@@ -182,7 +182,7 @@ def route(h, W, router):
 def router_margins(h, W, router):
     """How clearly each token's experts are chosen: the least change of one logit, about, that changes the choice.  The gap
     between the last expert chosen and the best one left out of the kept groups (in logits), and the gap between the last
-    group kept and the best one left out (in scores; a score moves by at most a quarter of what a logit does)."""
+    group kept and the best one left out (in scores, doubled: four logits move it, a score by at most a quarter of its logit)."""
     z = h @ W.T
     s = sigmoid(z)
     groups = router.get("groups") or {}
@@ -193,7 +193,7 @@ def router_margins(h, W, router):
         score = np.array([np.sort(x)[::-1][:2].sum() for x in s[t].reshape(n, -1)])
         order = np.argsort(-score, kind="stable")
         if keep < n:
-            out[t] = min(out[t], score[order[keep - 1]] - score[order[keep]])
+            out[t] = min(out[t], 2.0 * (score[order[keep - 1]] - score[order[keep]]))
         cand = np.sort(zt[order[:keep]].ravel())[::-1]
         if top < len(cand):
             out[t] = min(out[t], cand[top - 1] - cand[top])
