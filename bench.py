@@ -1079,6 +1079,173 @@ def negilorn_kernels(pk, sz):
     return rows
 
 
+# ---- Birelix beside Kapuvik at equal size (`--workload birelix`) ----------------------------------------
+# The same widths and head counts as above, four layers: latent attention (heads of 128 + 64 rotated channels, values of 128, a
+# latent row of 512 + 64, queries through a latent of 768, a gate per head) with a dense feed-forward of the size that a
+# Dobepel token runs through, two layers of the gated delta rule (128 x 128 state a head, two heads a q/k head, four taps) and
+# an attention layer (heads of 128, grouped key/value heads, biases, unit queries and keys, a window of 1,024, one added to the
+# denominator), these three with 8 experts in 4 groups, 2 of them chosen from 2 groups.  Kapuvik is the closest existing model:
+# latent attention through the same kernels, softmax attention, and linear attention with a float32 recurrence.  The experts'
+# like kernels are Dobepel's and Buvuzen's.
+BIRELIX_QRANK, BIRELIX_WINDOW, BIRELIX_TAPS, BIRELIX_GROUPS, BIRELIX_KEEP, BIRELIX_LIMIT = 768, 1024, 4, 4, 2, 7.0
+
+
+def birelix_raw(sz):
+    ff = {"kind": "dense", "ff": DOBEPEL_TOP * sz["expert_ff"] + sz["shared_ff"]}
+    moe = {"kind": "moe", "expert": {"ff": sz["expert_ff"], "limit": BIRELIX_LIMIT}, "router": {
+        "experts": DOBEPEL_EXPERTS, "top": DOBEPEL_TOP, "groups": {"count": BIRELIX_GROUPS, "keep": BIRELIX_KEEP}}}
+    lat = {"heads": sz["heads"], "dim": 128, "rot_dim": KAPUVIK_ROT, "vdim": 128, "kv_rank": KAPUVIK_RANK, "q_rank": BIRELIX_QRANK,
+           "scale": 192 ** -0.5, "rot": {"base": 10000.0, "dims": KAPUVIK_ROT}}
+    att = {"heads": sz["heads"], "kv_heads": sz["kv_heads"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": BIRELIX_WINDOW}}
+    rule = {"heads": sz["lin_heads"], "kv_heads": sz["lin_heads"] // 2, "dim": 128, "vdim": 128, "conv": BIRELIX_TAPS}
+    layers = [{"type": "latent_attention", "mixer": lat, "mlp": ff}, {"type": "delta", "mixer": rule, "mlp": moe},
+              {"type": "delta", "mixer": rule, "mlp": moe}, {"type": "attention", "mixer": att, "mlp": moe}]
+    return {"architecture": "Birelix", "vocab": DOBEPEL_VOCAB, "width": sz["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0},
+            "layers": json.loads(json.dumps(layers))}
+
+
+def birelix_workload(args, pk):
+    """Prefill (one prompt of 2,048 tokens in one step) and decode (batch 8 at 2,048 cached tokens) of Birelix and of
+    Kapuvik at equal width and depth, through the step function, timed with CUDA events; then the design's own kernels
+    beside the like kernels of Kapuvik, Dobepel and Buvuzen at the 2k size, each as a fraction of its roofline."""
+    import torch
+    from velox_b200.config import BirelixConfig, KapuvikConfig
+
+    T, B, CTX = 2048, 8, 2048
+    K, W = max(1, min(args.steps, 32)), max(3, args.warmup)
+    gen = torch.Generator().manual_seed(SEED)
+    sizes = {}
+    four = lambda sz: dict(sz, layers=4)
+    model_points(BirelixConfig.from_dict(birelix_raw(four(DOBEPEL_SIZES["1k"]))), DOBEPEL_VOCAB, T, B, CTX, K, W, gen)  # thrown away
+    for name, sz in DOBEPEL_SIZES.items():
+        sz = four(sz)
+        sizes[name] = {"birelix": model_points(BirelixConfig.from_dict(birelix_raw(sz)), DOBEPEL_VOCAB, T, B, CTX, K, W, gen),
+                       "kapuvik": model_points(KapuvikConfig.from_dict(kapuvik_raw(sz)), DOBEPEL_VOCAB, T, B, CTX, K, W, gen),
+                       "shape": sz}
+    return {"metric": "Birelix beside Kapuvik at equal size: prefill of %d tokens, decode at batch %d with %d cached tokens, bf16"
+                      % (T, B, CTX), "unit": "tokens/s", "n_gpus": 1, "steps": K, "warmup": W, "sizes": sizes,
+            "value": sizes["2k"]["birelix"]["decode_tok_s"], "higher_is_better": True,
+            "kernels": birelix_kernels(pk, four(DOBEPEL_SIZES["2k"])), "peaks": pk,
+            "data": "synthetic: random weights N(0,0.02) seed 2, uniform random token ids"}
+
+
+def birelix_kernels(pk, sz):
+    """Microseconds and fractions of the roofline of Birelix's kernels beside the like kernels of Kapuvik, Dobepel and Buvuzen."""
+    import torch
+    from types import SimpleNamespace
+    from velox_b200.csrc import ops
+    dev, bf, f32 = "cuda:0", torch.bfloat16, torch.float32
+    E, H, G, D = sz["width"], sz["heads"], sz["kv_heads"], 128
+    HL, GL, Dv, WIN, TAPS = sz["lin_heads"], sz["lin_heads"] // 2, 128, BIRELIX_WINDOW, BIRELIX_TAPS
+    C, R, QR = KAPUVIK_RANK, KAPUVIK_ROT, BIRELIX_QRANK
+    T, B, CTX, S = 2048, 8, 2048, PAGE
+    rows, row, us = kernel_rows(pk)
+    ints = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    rnd = lambda *shape: torch.randn(shape, device=dev)
+    pages = B * (CTX // S)
+    bt = torch.arange(pages, dtype=torch.int32, device=dev).view(B, CTX // S)
+    cu, off, pos_t, seq_t = ints([0, T]), ints([0]), ints(list(range(T))), ints([0] * T)
+    seqs, pos = ints(list(range(B))), ints([CTX - 1] * B)
+    # -- windowed attention --
+    kp, vp = rnd(pages, G, S, D).to(bf), rnd(pages, G, S, D).to(bf)
+    width = (H + 2 * G) * D
+    q, qd, zeros, one = rnd(T, width).to(bf), rnd(B, width).to(bf), torch.zeros(H, device=dev), torch.ones(D, device=dev)
+    pairs, full = sum(min(i + 1, WIN) for i in range(T)), T * (T + 1) // 2
+    row("prompt attention, window %d, one added to the denominator (tcgen05, P in two halves)" % WIN, us(lambda: ops.paged_prefill_attention_tc(
+        q, width, kp, vp, bt, cu, off, D ** -0.5, WIN, H, G, D, 1, T, T, halves=True, sinks=zeros)), 4.0 * pairs * D * H)
+    row("Buvuzen: the same kernel, all keys", us(lambda: ops.paged_prefill_attention_tc(
+        q, width, kp, vp, bt, cu, off, D ** -0.5, 0, H, G, D, 1, T, T, halves=True, sinks=zeros)), 4.0 * full * D * H)
+    row("Kapuvik: prompt attention, bounded scores, all keys (mma.sync)", us(lambda: ops.biased_prefill_attention(
+        q, width, kp, vp, bt, cu, off, D ** -0.5, 0, 0, 0.0, H, G, D, D, 1, T, T, softcap=KAPUVIK_CAP)), 4.0 * full * D * H)
+    row("decode attention, window %d, one added to the denominator" % WIN, us(lambda: ops.biased_decode_attention(
+        qd, width, kp, vp, bt, seqs, pos, D ** -0.5, WIN, 0, 0.0, H, G, D, D, B, max_kv=CTX, sinks=zeros), 50), 0.0, B * G * WIN * 2 * D * 2.0)
+    pos_w = ints([WIN - 1] * B)
+    row("Kapuvik: decode attention, bounded scores, %d keys (the same kernel)" % WIN, us(lambda: ops.biased_decode_attention(
+        qd, width, kp, vp, bt, seqs, pos_w, D ** -0.5, 0, 0, 0.0, H, G, D, D, B, max_kv=WIN, softcap=KAPUVIK_CAP), 50), 0.0, B * G * WIN * 2 * D * 2.0)
+    slots = torch.randperm(pages * S, device=dev)[:T].to(torch.int32)
+    inv = (1e4 ** (-torch.arange(0, D, 2, device=dev, dtype=f32) / D)).contiguous()
+    row("unit queries and keys + cache write, %d tokens" % T, us(lambda: ops.qk_norm_rope_kv(
+        q, one, one, 1e-6, None, 0, pos_t, slots, kp, vp, H, G, D, D)), 0.0, T * width * 2 * 2.0)
+    row("Kapuvik: q/k rotation + cache write, %d tokens (the same kernel)" % T, us(lambda: ops.qk_norm_rope_kv(
+        q, None, None, 1e-6, inv, D, pos_t, slots, kp, vp, H, G, D, D)), 0.0, T * width * 2 * 2.0)
+    # -- latent attention: its kernels are Kapuvik's; the query latent's norm and the gate per head beside them --
+    RW = C + R
+    pool = rnd(pages, 1, S, RW).to(bf)
+    qa = rnd(B, H, RW).to(bf)
+    row("decode latent attention, folded, %d tokens x %d heads over %d rows (Kapuvik's kernel)" % (B, H, CTX), us(lambda: ops.latent_attention(
+        qa, pool, bt, seqs, pos, RW ** -0.5, H, C, R, max_kv=CTX), 20), 0.0, B * CTX * RW * 2.0)
+    big = 16384
+    ob, gb, gw = rnd(big, H * Dv).to(bf), rnd(big, H).to(bf), rnd(big, H * Dv).to(bf)
+    row("gate per head, %d rows" % big, us(lambda: ops.head_gate(ob, gb), 10), 0.0, big * H * Dv * 4.0)
+    row("Fovenex: gate element by element, %d rows" % big, us(lambda: ops.sigmoid_gate(ob, gw), 10), 0.0, big * H * Dv * 6.0)
+    # -- the delta rule --
+    ch = 2 * GL * D + HL * Dv
+    x, xd = (rnd(T, ch + HL * Dv) * 0.5).to(bf), rnd(B, ch + HL * Dv) * 0.5
+    ab, abd = rnd(T, 2 * HL), rnd(B, 2 * HL)
+    taps, nea, dtb, nw = rnd(TAPS, ch) * 0.5, -torch.rand(HL, device=dev), torch.zeros(HL, device=dev), torch.ones(Dv, device=dev)
+    state, ring = [torch.zeros((B, HL, Dv, D), device=dev) for _ in range(4)], [torch.zeros((B, TAPS, ch), device=dev) for _ in range(4)]
+    cu_b, slots_b, slot0 = ints(list(range(B + 1))), ints(list(range(B))), ints([0])
+    ctx = SimpleNamespace(n_seqs=1, max_new=T, cu_seqlens=cu, seq_of_token=seq_t, state_slots=slot0, positions=pos_t)
+    ctxd = SimpleNamespace(n_seqs=B, max_new=1, cu_seqlens=cu_b, seq_of_token=seqs, state_slots=slots_b, positions=pos)
+    turn = [0]
+
+    def nxt(ws):
+        turn[0] += 1
+        return ws[turn[0] % len(ws)]
+    y, coef, o = rnd(T, ch), torch.empty((T, HL, 20), device=dev), torch.empty((T, HL * Dv), device=dev)
+    lib, p = ops.library(), ops._ptr
+    row("short convolutions, silu, unit vectors, %d tokens" % T, us(lambda: ops._check(lib.vx_delta_conv(
+        p(x), x.stride(0), p(taps), p(ring[0]), p(seq_t), p(cu), p(slot0), p(pos_t), p(y), T, GL, D, HL, Dv, TAPS, D ** -0.5,
+        ops.VX_BF16, ops._stream()), "delta_conv")), 0.0, T * ch * 6.0)
+    low, w2t = rnd(T, 64), rnd(64, ch) * 0.1
+    row("Negilorn: decays in float32 (tanh, product, exponential), %d tokens" % T, us(lambda: ops.low_rank_decay(low, w2t, taps[0].contiguous())), 0.0, T * (ch + 64) * 4.0)
+    fl = T * HL * 2.0 * (32 * 2 * D + 2 * D * Dv)
+    simt = T * HL * 2.0 * 3 * D * Dv
+    cores = 148 * 128 * 2 * 1.965e9
+    coefs = lambda: ops._check(lib.vx_delta_coef(p(y), p(ab), ab.stride(0), HL, 0, p(nea), p(dtb), p(seq_t), p(cu), p(coef), T, GL, D, HL, Dv,
+                                                 ops._stream()), "delta_coef")
+    row("decays, step sizes, products within eight tokens and their inverse, %d tokens" % T, us(coefs), 0.0, T * (2 * GL * D + 22 * HL) * 4.0)
+    ops.delta_rule(x, ab, HL, 0, taps, nea, dtb, state[0], ring[0], ctx, GL, D, HL, Dv, D ** -0.5)
+    t_walk = us(lambda: ops._check(lib.vx_delta_walk(
+        p(y), p(coef), p(state[0]), p(ring[0]), p(x), x.stride(0), p(cu), p(slot0), p(pos_t),
+        p(o), 1, GL, D, HL, Dv, TAPS, 0, ops.VX_BF16, ops._stream()), "delta_walk"), 5)
+    row("prompt delta rule: the walk, %d heads (%.2f of the float32 multiply-add rate)" % (HL, simt / (t_walk * 1e-6) / cores), t_walk, fl)
+    xk = (rnd(T, 4 * HL * D) * 0.5).to(bf)
+    z, st = rnd(T, HL * D) + 2.0, torch.zeros((B, HL, D, Dv), device=dev)
+    plan = ops.StretchPlan([T], dev)
+    t_k = us(lambda: ops.linear_attention_walk(xk, 0, HL * D, 2 * HL * D, st, cu, slot0, 1, HL, D, Dv, gate=z, gate_mul=1 / 16.0, q_mul=D ** -0.5,
+                                               stretches=plan), 5)
+    row("Kapuvik: prompt linear attention, decay per channel, %d heads (stretches; %.2f of the float32 multiply-add rate)"
+        % (HL, 2 * simt / (t_k * 1e-6) / cores), t_k, fl)
+    sb = B * HL * D * Dv * 4 * 2.0
+    row("decode delta rule: convolutions, rule, norm, gate in one kernel", us(lambda: ops.delta_decode(
+        xd, ch, abd, HL, 0, taps, nea, dtb, nw, nxt(state), ring[turn[0] % 4], ctxd, GL, D, HL, Dv, D ** -0.5, 1e-6, bf), 48), 0.0,
+        sb + B * ch * (TAPS + 2) * 4.0)
+    xkd, zd = (rnd(B, 4 * HL * D) * 0.5).to(bf), rnd(B, HL * D)
+    sts = [torch.zeros((B, HL, D, Dv), device=dev) for _ in range(4)]
+    row("Kapuvik: decode linear attention, decay per channel", us(lambda: ops.linear_attention_walk(
+        xkd, 0, HL * D, 2 * HL * D, nxt(sts), cu_b, slots_b, B, HL, D, Dv, gate=zd, gate_mul=1 / 16.0), 48), 0.0, sb)
+    # -- experts --
+    NE, TOP, I = DOBEPEL_EXPERTS, DOBEPEL_TOP, sz["expert_ff"]
+    h, hd = rnd(T, E).to(bf), rnd(B, E).to(bf)
+    wr = (rnd(NE, E) * 0.02).float().contiguous()
+    gu, down = (rnd(NE, 2 * I, E) * 0.02).to(bf), (rnd(NE, E, I) * 0.02).to(bf)
+    mine = dict(scores="sigmoid", groups=BIRELIX_GROUPS, keep_groups=BIRELIX_KEEP, group_pair=True, renormalise=True)
+    capped = (BIRELIX_LIMIT, 1.702)
+    pl = ops.moe_route(h, wr, None, NE, TOP, ops.MOE_TCGEN05_TILE_ROWS, **mine)
+    rows_h = ops.moe_gather_rows(h, pl)
+    row("router (sigmoid, pairs in groups, renormalised) + plan, %d tokens" % T, us(lambda: ops.moe_route(h, wr, None, NE, TOP, ops.MOE_TCGEN05_TILE_ROWS, **mine)), 0.0, T * E * 2.0)
+    row("Dobepel: router (softmax of the chosen) + plan, %d tokens" % T, us(lambda: ops.moe_route(h, wr, None, NE, TOP, ops.MOE_TCGEN05_TILE_ROWS)), 0.0, T * E * 2.0)
+    row("experts gate and up, bounded gate, %d rows (tcgen05 grouped)" % (T * TOP), us(lambda: ops.moe_gemm_tcgen05(rows_h, gu, pl, capped=capped)), 2.0 * T * TOP * 2 * I * E)
+    row("Dobepel: experts gate and up, silu, %d rows (tcgen05 grouped)" % (T * TOP), us(lambda: ops.moe_gemm_tcgen05(rows_h, gu, pl, gated_activation="silu")), 2.0 * T * TOP * 2 * I * E)
+    gus = [(rnd(NE, 2 * I, E) * 0.02).to(bf) for _ in range(3)]
+    pd = ops.moe_route(hd, wr, None, NE, TOP, ops.moe_tile_rows(hd, B * TOP), **mine)
+    live = len(set(pd.chosen.tolist()))
+    row("experts gate and up, bounded gate, %d tokens (grouped mma.sync)" % B, us(lambda: ops.moe_gemm(hd, nxt(gus), pd, True, bf, capped=capped), 48), 0.0, live * 2 * I * E * 2.0)
+    row("Dobepel: experts gate and up, silu, %d tokens" % B, us(lambda: ops.moe_gemm(hd, nxt(gus), pd, True, bf, gated_activation="silu"), 48), 0.0, live * 2 * I * E * 2.0)
+    return rows
+
+
 def main() -> int:
     global CONTEXT, PROMPT
     ap = argparse.ArgumentParser()
@@ -1088,14 +1255,15 @@ def main() -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the model has (recorded in config)")
     ap.add_argument("--batch", type=int, default=BATCH)
-    ap.add_argument("--workload", default="decode", choices=["decode", "stream", "dobepel", "buvuzen", "kapuvik", "fovenex", "negilorn"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "stream", "dobepel", "buvuzen", "kapuvik", "fovenex", "negilorn", "birelix"],
                     help="decode: the benchmark (steady decoding at a fixed batch). stream: continuous batching "
                          "under arrivals (64 requests, prompts of 128-4,096 tokens, 256 new tokens each, Poisson "
                          "arrivals); prints its own JSON line. dobepel: the Dobepel design beside Qwen3 at equal size "
                          "(prefill, decode, and the design's kernels against their rooflines); its own JSON line. buvuzen: the same for "
                          "the Buvuzen design beside Dobepel and Qwen3. kapuvik: the same for the Kapuvik design beside Dobepel. "
                          "fovenex: the same for the Fovenex design beside Kapuvik; "
-                         "negilorn: the same for the Negilorn design beside Kapuvik")
+                         "negilorn: the same for the Negilorn design beside Kapuvik; "
+                         "birelix: the same for the Birelix design beside Kapuvik")
     ap.add_argument("--arrival-rate", type=float, default=16.0, help="stream: mean arrivals a second")
     ap.add_argument("--lazy-graphs", action="store_true",
                     help="stream: capture each decode graph when a step first needs it, inside the run")
@@ -1126,10 +1294,10 @@ def main() -> int:
     from velox_b200.csrc import ops
     from velox_b200.engine import StepEntry
 
-    if args.workload in ("dobepel", "buvuzen", "kapuvik", "fovenex", "negilorn"):
+    if args.workload in ("dobepel", "buvuzen", "kapuvik", "fovenex", "negilorn", "birelix"):
         with ClockSampler() as clocks:
             res = {"dobepel": dobepel_workload, "buvuzen": buvuzen_workload, "kapuvik": kapuvik_workload, "fovenex": fovenex_workload,
-                   "negilorn": negilorn_workload}[args.workload](args, peaks())
+                   "negilorn": negilorn_workload, "birelix": birelix_workload}[args.workload](args, peaks())
         res["clocks"] = clocks.summary()
         print(json.dumps(res))
         return 0

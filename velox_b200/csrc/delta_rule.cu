@@ -4,8 +4,9 @@
 // g = exp(-exp(A_log) softplus(a + dt_bias)) and a step size beta = sigmoid(b) per head and token.  Several heads may share
 // one q/k head.
 //
-//   delta_conv      convolution, silu and unit vectors of a step's tokens (float32 out), and every key's products with the
-//                   keys and queries near it
+//   delta_conv      convolution, silu and unit vectors of a step's tokens (float32 out)
+//   delta_coef      decays, step sizes, and what follows from them and from the products among keys and queries within
+//                   eight tokens
 //   delta_walk      the recurrence over a step's tokens; afterwards the last inputs of the convolutions go into their slots
 //   delta_decode    a step of single tokens: both of these, the norm of every head's output and its gate in one kernel
 //
@@ -16,8 +17,8 @@
 #include "mma_helpers.cuh"
 
 #define DR_EPS_UNIT 1e-6f
-#define DR_DOTS 8      // per token and q/k head: k.k of the tokens 1, 2, 3 back (0 .. 2), q.k of itself and 1, 2, 3 back (3 .. 6)
-#define DR_MINI 4      // tokens of a mini-chunk
+#define DR_MINI 8      // tokens of a mini-chunk
+#define DR_COEF 20     // numbers per token and head that the walk reads
 #define DR_MAX_TAPS 64
 
 __device__ __forceinline__ float dr_silu(float z) { return z / (1.f + expf(-z)); }
@@ -67,28 +68,32 @@ __device__ __forceinline__ DrPlace dr_place(int t, const int* seq_of_token, cons
 }
 
 // ---- convolution, silu, unit vectors ----
-// y float32 [tokens, C] with C = 2 G D + H Dv: q as a unit vector times q_mul, k as a unit vector, v.  dots float32
-// [tokens, G, DR_DOTS], where the tokens it reaches back to lie among the rows that the request brings (else whatever).
-// A warp takes one unit (the q and k of one head, or a run of v's channels) of one token.  Any sizes (D up to 256).
-template <typename T>
-__device__ __forceinline__ float dr_conv_at(const T* __restrict__ x, int ldx, const float* __restrict__ w, int C, int taps, int t,
-                                            const DrPlace& at, int c) {
-    float s = 0.f;
-    for (int j = taps - 1; j >= 0; --j) {
-        float v = 0.f;
-        if (at.local >= j) v = to_f32(x[(size_t)(t - j) * ldx + c]);
-        else if (at.pos >= j) v = at.ring[(size_t)((at.pos - j) % taps) * C + c];
-        s = fmaf(w[(size_t)(taps - 1 - j) * C + c], v, s);
+// y float32 [tokens, C] with C = 2 G D + H Dv: q as a unit vector times q_mul, k as a unit vector, v.
+// The convolution of VEC channels from c on of token t, each tap's row from the step or from the ring.
+template <typename T, int VEC>
+__device__ __forceinline__ void dr_conv_at(const T* __restrict__ x, int ldx, const float* __restrict__ w, int C, int taps, int t,
+                                           const DrPlace& at, int c, float (&out)[VEC]) {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) out[e] = 0.f;
+    for (int j = min(taps - 1, at.pos); j >= 0; --j) {
+        float v[VEC], wv[VEC];
+        if (at.local >= j) dr_load<VEC>(x + (size_t)(t - j) * ldx + c, v);
+        else dr_load<VEC>(at.ring + (size_t)((at.pos - j) % taps) * C + c, v);
+        dr_load<VEC>(w + (size_t)(taps - 1 - j) * C + c, wv);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) out[e] = fmaf(wv[e], v[e], out[e]);
     }
-    return dr_silu(s);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) out[e] = dr_silu(out[e]);
 }
 
+// Any sizes (D up to 256): a warp takes one unit (a q or k head, or a run of v's channels) of one token.
 template <typename T>
 __global__ void __launch_bounds__(128)
 delta_conv_any_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ w, const float* __restrict__ ring,
                       const int* __restrict__ seq_of_token, const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots,
-                      const int* __restrict__ positions, float* __restrict__ y, float* __restrict__ dots, int tokens, int G, int D,
-                      int HDv, int taps, float q_mul, int units) {
+                      const int* __restrict__ positions, float* __restrict__ y, int tokens, int G, int D, int HDv, int taps, float q_mul,
+                      int units) {
     pdl_wait();
     pdl_trigger();
     const long long id = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
@@ -98,79 +103,40 @@ delta_conv_any_kernel(const T* __restrict__ x, int ldx, const float* __restrict_
     const int C = 2 * G * D + HDv;
     const DrPlace at = dr_place(t, seq_of_token, cu_seqlens, state_slots, positions, ring, (size_t)taps * C);
     float* yr = y + (size_t)t * C;
-    if (unit >= G) {   // 256 channels of v
-        const int c0 = 2 * G * D + (unit - G) * 256;
-        for (int i = lane; i < 256 && c0 + i < C; i += 32) yr[c0 + i] = dr_conv_at(x, ldx, w, C, taps, t, at, c0 + i);
-        return;
-    }
-    const int qc = unit * D, kc = G * D + unit * D;
-    float q[8], k[DR_MINI][8], kn[DR_MINI], qn = 0.f;
+    const bool is_v = unit >= 2 * G;
+    const int c0 = is_v ? 2 * G * D + (unit - 2 * G) * 256 : unit * D, n = is_v ? min(256, C - c0) : D;
+    float v[8], ss = 0.f;
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
-        const int d = lane + 32 * i;
-        q[i] = d < D ? dr_conv_at(x, ldx, w, C, taps, t, at, qc + d) : 0.f;
-        qn = fmaf(q[i], q[i], qn);
+        float one[1] = {0.f};
+        if (lane + 32 * i < n) dr_conv_at<T, 1>(x, ldx, w, C, taps, t, at, c0 + lane + 32 * i, one);
+        v[i] = one[0];
+        ss = fmaf(v[i], v[i], ss);
     }
-    qn = rsqrtf(warp_sum(qn) + DR_EPS_UNIT) * q_mul;
+    const float mul = is_v ? 1.f : rsqrtf(warp_sum(ss) + DR_EPS_UNIT) * (unit < G ? q_mul : 1.f);
 #pragma unroll
-    for (int b = 0; b < DR_MINI; ++b) {   // the token's key and those of the three before it
-        float ss = 0.f;
-        const bool there = at.local >= b;
-        const DrPlace ab{at.local - b, at.pos - b, at.ring};
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const int d = lane + 32 * i;
-            k[b][i] = d < D && there ? dr_conv_at(x, ldx, w, C, taps, t - b, ab, kc + d) : 0.f;
-            ss = fmaf(k[b][i], k[b][i], ss);
-        }
-        kn[b] = rsqrtf(warp_sum(ss) + DR_EPS_UNIT);
-    }
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-        const int d = lane + 32 * i;
-        if (d < D) {
-            yr[qc + d] = q[i] * qn;
-            yr[kc + d] = k[0][i] * kn[0];
-        }
-    }
-    float* dr = dots + ((size_t)t * G + unit) * DR_DOTS;
-#pragma unroll
-    for (int b = 0; b < DR_MINI; ++b) {
-        float kk = 0.f, qk = 0.f;
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            kk = fmaf(k[0][i], k[b][i], kk);
-            qk = fmaf(q[i], k[b][i], qk);
-        }
-        kk = warp_sum(kk) * kn[0] * kn[b];
-        qk = warp_sum(qk) * qn * kn[b];
-        if (lane == 0) {
-            if (b) dr[b - 1] = kk;
-            dr[3 + b] = qk;
-        }
-    }
+    for (int i = 0; i < 8; ++i)
+        if (lane + 32 * i < n) yr[c0 + lane + 32 * i] = v[i] * mul;
 }
 
-// The same for four taps and heads of 32 VEC channels, a warp taking RUN consecutive tokens of a unit: every row it needs
-// is asked for before the first is used and read once, not once a tap.
+// The same for four taps and heads of 32 VEC channels, a warp taking DR_RUN consecutive tokens of a unit.  Where all of them
+// and the three before the first belong to one request and to this step, every row is asked for before the first is used and
+// read once, not once a tap; else token by token.
 #define DR_RUN 8
 template <typename T, int VEC>
 __global__ void __launch_bounds__(128)
 delta_conv_run_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ w, const float* __restrict__ ring,
                       const int* __restrict__ seq_of_token, const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots,
-                      const int* __restrict__ positions, float* __restrict__ y, float* __restrict__ dots, int tokens, int G, int HDv,
-                      float q_mul, int units) {
-    constexpr int TAPS = 4, D = 32 * VEC, BACK = DR_MINI - 1;
+                      const int* __restrict__ positions, float* __restrict__ y, int tokens, int G, int HDv, float q_mul, int units) {
+    constexpr int TAPS = 4, D = 32 * VEC;
     const int C = 2 * G * D + HDv;
     const int lane = threadIdx.x & 31;
     const long long id = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
     const int unit = (int)(id % units), t0 = (int)(id / units) * DR_RUN;
-    if (t0 >= tokens) {   // (a warp past the end; the block's first warp never is)
-        return;
-    }
-    const bool is_v = unit >= G;
-    const int c = is_v ? 2 * G * D + (unit - G) * D + lane * VEC : unit * D + lane * VEC;   // v's or q's channel
-    const bool live = c < C;
+    if (t0 >= tokens) return;   // (a warp past the end; a block's first warp never is)
+    const int c = unit * D + lane * VEC;   // (v's channels follow those of the 2 G heads of q and k)
+    const bool live = c < C, is_v = unit >= 2 * G;
+    const float unit_mul = unit < G ? q_mul : 1.f;
     float wt[TAPS][VEC];
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) {
@@ -180,450 +146,546 @@ delta_conv_run_kernel(const T* __restrict__ x, int ldx, const float* __restrict_
     }
     pdl_wait();
     pdl_trigger();
-    // the convolution of token t from those of the rows win[first + TAPS - 1 - j] = x[t - j] that its request brings
-    auto conv = [&](const auto& win, int first, const float (&wk)[TAPS][VEC], int t, int ch, float (&out)[VEC]) {
-        const DrPlace at = dr_place(t, seq_of_token, cu_seqlens, state_slots, positions, ring, (size_t)TAPS * C);
+    const int seq = seq_of_token[t0], first = cu_seqlens[seq], last = cu_seqlens[seq + 1];
+    auto finish = [&](int t, float (&o)[VEC]) {
+        if (!is_v) {   // (a warp holds one unit)
+            float ss = 0.f;
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) out[e] = 0.f;
+            for (int e = 0; e < VEC; ++e) ss = fmaf(o[e], o[e], ss);
+            const float mul = rsqrtf(warp_sum(ss) + DR_EPS_UNIT) * unit_mul;
 #pragma unroll
-        for (int j = TAPS - 1; j >= 0; --j) {
-            float v[VEC];
-            if (at.local >= j) {
-#pragma unroll
-                for (int e = 0; e < VEC; ++e) v[e] = win[first + TAPS - 1 - j][e];
-            } else if (at.pos >= j && ch < C) {
-                dr_load<VEC>(at.ring + (size_t)((at.pos - j) % TAPS) * C + ch, v);
-            } else {
-#pragma unroll
-                for (int e = 0; e < VEC; ++e) v[e] = 0.f;
-            }
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) out[e] = fmaf(wk[TAPS - 1 - j][e], v[e], out[e]);
+            for (int e = 0; e < VEC; ++e) o[e] *= mul;
         }
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) out[e] = dr_silu(out[e]);
+        if (live) dr_store<VEC>(y + (size_t)t * C + c, o);
     };
-    auto row = [&](int r, int ch, float (&v)[VEC]) {
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) v[e] = 0.f;
-        if (r >= 0 && r < tokens && ch < C) dr_load<VEC>(x + (size_t)r * ldx + ch, v);
-    };
-    if (is_v) {
+    if (t0 - first >= TAPS - 1 && t0 + DR_RUN <= last) {
         float win[DR_RUN + TAPS - 1][VEC];
 #pragma unroll
-        for (int i = 0; i < DR_RUN + TAPS - 1; ++i) row(t0 - (TAPS - 1) + i, c, win[i]);
+        for (int i = 0; i < DR_RUN + TAPS - 1; ++i) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) win[i][e] = 0.f;
+            if (live) dr_load<VEC>(x + (size_t)(t0 - (TAPS - 1) + i) * ldx + c, win[i]);
+        }
 #pragma unroll
         for (int u = 0; u < DR_RUN; ++u) {
-            const int t = t0 + u;
-            if (t >= tokens) break;
             float o[VEC];
-            conv(win, u, wt, t, c, o);
-            if (live) dr_store<VEC>(y + (size_t)t * C + c, o);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                float s = wt[0][e] * win[u][e];
+#pragma unroll
+                for (int j = 1; j < TAPS; ++j) s = fmaf(wt[j][e], win[u + j][e], s);
+                o[e] = dr_silu(s);
+            }
+            finish(t0 + u, o);
         }
         return;
     }
-    const int ck = G * D + c;
-    float wk[TAPS][VEC];
+    for (int t = t0; t < min(t0 + DR_RUN, tokens); ++t) {
+        const DrPlace at = dr_place(t, seq_of_token, cu_seqlens, state_slots, positions, ring, (size_t)TAPS * C);
+        float o[VEC];
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j) dr_load<VEC>(w + (size_t)j * C + ck, wk[j]);
-    float qw[DR_RUN + TAPS - 1][VEC], kw[DR_RUN + BACK + TAPS - 1][VEC];
-#pragma unroll
-    for (int i = 0; i < DR_RUN + BACK + TAPS - 1; ++i) row(t0 - BACK - (TAPS - 1) + i, ck, kw[i]);
-#pragma unroll
-    for (int i = 0; i < DR_RUN + TAPS - 1; ++i) row(t0 - (TAPS - 1) + i, c, qw[i]);
-    float kh[DR_MINI][VEC];   // unit keys: [b] of the token b back
-#pragma unroll
-    for (int b = 0; b < DR_MINI; ++b)
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) kh[b][e] = 0.f;
-#pragma unroll
-    for (int u = -BACK; u < DR_RUN; ++u) {
-        const int t = t0 + u;
-        if (t >= tokens) break;
-#pragma unroll
-        for (int b = DR_MINI - 1; b > 0; --b)
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) kh[b][e] = kh[b - 1][e];
-        if (t < 0) continue;
-        conv(kw, u + BACK, wk, t, ck, kh[0]);
-        float ss = 0.f;
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) ss = fmaf(kh[0][e], kh[0][e], ss);
-        const float kn = rsqrtf(warp_sum(ss) + DR_EPS_UNIT);
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) kh[0][e] *= kn;
-        if (u < 0) continue;
-        float q[VEC];
-        conv(qw, u, wt, t, c, q);
-        ss = 0.f;
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) ss = fmaf(q[e], q[e], ss);
-        const float qn = rsqrtf(warp_sum(ss) + DR_EPS_UNIT) * q_mul;
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) q[e] *= qn;
-        dr_store<VEC>(y + (size_t)t * C + c, q);
-        dr_store<VEC>(y + (size_t)t * C + ck, kh[0]);
-        float p[DR_DOTS];
-#pragma unroll
-        for (int b = 0; b < DR_DOTS; ++b) p[b] = 0.f;
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-#pragma unroll
-            for (int b = 1; b < DR_MINI; ++b) p[b - 1] = fmaf(kh[0][e], kh[b][e], p[b - 1]);
-#pragma unroll
-            for (int b = 0; b < DR_MINI; ++b) p[3 + b] = fmaf(q[e], kh[b][e], p[3 + b]);
-        }
-        // eight sums over 32 lanes: halves of the values change sides, so lane l ends with the sum number (l >> 2)
-        float a4[4], a2[2], a1;
-        const bool h16 = lane & 16, h8 = lane & 8, h4 = lane & 4;
-#pragma unroll
-        for (int i = 0; i < 4; ++i) a4[i] = (h16 ? p[4 + i] : p[i]) + __shfl_xor_sync(0xffffffffu, h16 ? p[i] : p[4 + i], 16);
-#pragma unroll
-        for (int i = 0; i < 2; ++i) a2[i] = (h8 ? a4[2 + i] : a4[i]) + __shfl_xor_sync(0xffffffffu, h8 ? a4[i] : a4[2 + i], 8);
-        a1 = (h4 ? a2[1] : a2[0]) + __shfl_xor_sync(0xffffffffu, h4 ? a2[0] : a2[1], 4);
-        a1 += __shfl_xor_sync(0xffffffffu, a1, 2);
-        a1 += __shfl_xor_sync(0xffffffffu, a1, 1);
-        if ((lane & 3) == 0) dots[((size_t)t * G + unit) * DR_DOTS + (lane >> 2)] = a1;
+        for (int e = 0; e < VEC; ++e) o[e] = 0.f;
+        if (live) dr_conv_at<T, VEC>(x, ldx, w, C, TAPS, t, at, c, o);
+        finish(t, o);
     }
 }
 
 template <typename T>
 static int launch_delta_conv(const T* x, int ldx, const float* w, const float* ring, const int* seq_of_token, const int* cu_seqlens,
-                             const int* state_slots, const int* positions, float* y, float* dots, int tokens, int G, int D, int H,
-                             int Dv, int taps, float q_mul, cudaStream_t stream) {
+                             const int* state_slots, const int* positions, float* y, int tokens, int G, int D, int H, int Dv, int taps,
+                             float q_mul, cudaStream_t stream) {
     const int HDv = H * Dv, vec = D / 32, C = 2 * G * D + HDv;
     const bool run = taps == 4 && (D == 32 || D == 64 || D == 128) && tokens > 1 && HDv % vec == 0 && ldx % vec == 0 &&
                      !(((uintptr_t)x | (uintptr_t)w | (uintptr_t)ring | (uintptr_t)y) & 15) && C % vec == 0;
-    const int units = G + (run ? (HDv + D - 1) / D : (HDv + 255) / 256);
+    const int units = 2 * G + (run ? (HDv + D - 1) / D : (HDv + 255) / 256);
     const long long warps = (long long)units * (run ? (tokens + DR_RUN - 1) / DR_RUN : tokens);
     if ((warps + 3) / 4 > 0x7fffffffLL) return VX_ERR_LIMIT;
     const unsigned blocks = (unsigned)((warps + 3) / 4);
 #define DR_GO(V_) VX_LAUNCH_K(VX_K_ELEMENTWISE, (delta_conv_run_kernel<T, V_>), blocks, 128, 0, stream, x, ldx, w, ring, seq_of_token, \
-                              cu_seqlens, state_slots, positions, y, dots, tokens, G, HDv, q_mul, units)
+                              cu_seqlens, state_slots, positions, y, tokens, G, HDv, q_mul, units)
     if (run && vec == 1) DR_GO(1);
     else if (run && vec == 2) DR_GO(2);
     else if (run) DR_GO(4);
     else
         VX_LAUNCH_K(VX_K_ELEMENTWISE, (delta_conv_any_kernel<T>), blocks, 128, 0, stream, x, ldx, w, ring, seq_of_token, cu_seqlens,
-                    state_slots, positions, y, dots, tokens, G, D, HDv, taps, q_mul, units);
+                    state_slots, positions, y, tokens, G, D, HDv, taps, q_mul, units);
 #undef DR_GO
     VX_LAUNCH_CHECK();
     return VX_OK;
 }
 
 // x [tokens, ldx]: the projections q [G, D], k [G, D], v [H, Dv] from column 0 on.  w float32 [taps, C] (the last row is the
-// current token's), ring float32 [slots, taps, C] (read only).  y, dots: see `delta_conv_any_kernel`.
+// current token's), ring float32 [slots, taps, C] (read only).
 extern "C" int vx_delta_conv(const void* x, int ldx, const float* w, const float* ring, const int* seq_of_token,
-                             const int* cu_seqlens, const int* state_slots, const int* positions, float* y, float* dots, int tokens,
+                             const int* cu_seqlens, const int* state_slots, const int* positions, float* y, int tokens,
                              int G, int D, int H, int Dv, int taps, float q_mul, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return VX_OK;
     if (G <= 0 || D <= 0 || H <= 0 || Dv <= 0 || H % G || taps <= 0 || ldx < 2 * G * D + H * Dv) return VX_ERR_SHAPE;
     if (D > 256 || taps > DR_MAX_TAPS) return VX_ERR_LIMIT;
     if (dtype == VX_F32)
-        return launch_delta_conv<float>((const float*)x, ldx, w, ring, seq_of_token, cu_seqlens, state_slots, positions, y, dots, tokens,
-                                        G, D, H, Dv, taps, q_mul, stream);
+        return launch_delta_conv<float>((const float*)x, ldx, w, ring, seq_of_token, cu_seqlens, state_slots, positions, y, tokens, G, D,
+                                        H, Dv, taps, q_mul, stream);
     if (dtype == VX_BF16)
-        return launch_delta_conv<bf16>((const bf16*)x, ldx, w, ring, seq_of_token, cu_seqlens, state_slots, positions, y, dots, tokens,
-                                       G, D, H, Dv, taps, q_mul, stream);
+        return launch_delta_conv<bf16>((const bf16*)x, ldx, w, ring, seq_of_token, cu_seqlens, state_slots, positions, y, tokens, G, D, H,
+                                       Dv, taps, q_mul, stream);
     return VX_ERR_DTYPE;
 }
 
-// ---- the recurrence ----
-// A block owns DR_COLS columns of one head's state of one request, a warp four of them, eight lanes a column: lane i of the
-// eight holds the rows 4 i + 32 j .. + 3 (R of them) in registers.  Tokens are taken DR_MINI at a time.  With gamma_i the
-// product of the decays up to token i of the mini-chunk and rho_ij that of the decays after j up to i, the rule unrolls to
-//   u_i = beta_i (v_i - gamma_i (k_i . S) - sum_(j < i) rho_ij (k_i . k_j) u_j)
+// ---- the coefficients of a mini-chunk ----
+// A request's rows of this step are taken DR_MINI at a time.  With gamma_i the product of the decays g up to token i of the
+// mini-chunk, rho_ij that of the decays after j up to i, A_ij = beta_i rho_ij (k_i . k_j) for j < i and S the state before the
+// mini-chunk, the rule unrolls to
+//   (I + A) u = r,  r_i = beta_i v_i - beta_i gamma_i (k_i . S)
 //   o_i = gamma_i (q_i . S) + sum_(j <= i) rho_ij (q_i . k_j) u_j
-//   S  <- gamma_3 S + sum_j rho_3j k_j u_j^T
-// with S the state before the mini-chunk: the eight products with S of a mini-chunk do not wait for one another, and are
-// summed over the eight lanes together.  The products among keys and queries come from `delta_conv`.  Tokens are staged
-// DR_CHUNK at a time by asynchronous copies, a chunk ahead; their coefficients (three float4 a token) likewise, by a warp in
-// turn.  Tokens past a request's last count as k = q = v = 0, beta = 0, g = 1, which changes nothing.
-#define DR_WARPS 4
-#define DR_COLS (DR_WARPS * 4)
+//   S  <- gamma_last S + sum_j rho_(last,j) k_j u_j^T
+// Per token i and head: beta_i, beta_i gamma_i, gamma_i, rho_(last,i), then row i of (I + A)^-1, then the rho_ij (q_i . k_j).
+// A warp per eight token rows and q/k head; the products are summed over the lanes all 64 together (two rounds of 32).
+// Tokens past a request's last count as k = q = 0, beta = 0, g = 1.
+
+// 8 CC sums over 32 lanes (CC 1, 2 or 4): in the first rounds half of the values change sides, then what lanes are left is added;
+// lane l ends with the sum number l mod 8 CC.  The order of a sum's additions does not depend on CC.  With PERMUTED lane l
+// brings the value 8 c + (s xor (l mod 8)) in p[8 c + s]: then what changes sides in the first three rounds is in the same
+// place for every lane, and nothing has to be selected.
+template <int CC, bool PERMUTED>
+__device__ __forceinline__ float dr_sums(float (&p)[8 * CC], int lane) {
+#pragma unroll
+    for (int n = 4; n > 0; n >>= 1) {
+        const bool hi = lane & n;
+#pragma unroll
+        for (int c = 0; c < CC; ++c)
+#pragma unroll
+            for (int i = 0; i < n; ++i) {
+                const float keep = !PERMUTED && hi ? p[8 * c + n + i] : p[8 * c + i], give = !PERMUTED && hi ? p[8 * c + i] : p[8 * c + n + i];
+                p[8 * c + i] = keep + __shfl_xor_sync(0xffffffffu, give, n);
+            }
+    }
+#pragma unroll
+    for (int n = 1; n < 4; n <<= 1) {   // lanes 8 n apart, columns n apart
+        const bool hi = lane & (8 * n);
+        if (n < CC) {
+#pragma unroll
+            for (int c = 0; c < CC; c += 2 * n) {
+                const float keep = hi ? p[8 * (c + (n < CC ? n : 0))] : p[8 * c], give = hi ? p[8 * c] : p[8 * (c + (n < CC ? n : 0))];
+                p[8 * c] = keep + __shfl_xor_sync(0xffffffffu, give, 8 * n);
+            }
+        } else {
+            p[0] += __shfl_xor_sync(0xffffffffu, p[0], 8 * n);
+        }
+    }
+    return p[0];
+}
+
+#define DR_CW 4   // warps of a block
+__global__ void __launch_bounds__(DR_CW * 32)
+delta_coef_kernel(const float* __restrict__ y, const float* __restrict__ ab, int ldab, int a_col, int b_col,
+                  const float* __restrict__ neg_exp_a, const float* __restrict__ dt_bias, const int* __restrict__ seq_of_token,
+                  const int* __restrict__ cu_seqlens, float* __restrict__ coef, int tokens, int G, int D, int H, int C) {
+    __shared__ float kk_s[DR_CW][64], qk_s[DR_CW][64], a_s[DR_CW][4][64];
+    pdl_wait();
+    pdl_trigger();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, i = lane & 7;
+    const long long id = (long long)blockIdx.x * DR_CW + warp;
+    const int kvh = (int)(id % G);
+    const long long row0 = id / G * DR_MINI;
+    float *kk = kk_s[warp], *qk = qk_s[warp];
+    // (among eight rows of the step a mini-chunk starts once, or more often where requests end)
+    for (int u = 0; u < DR_MINI; ++u) {
+        if (row0 + u >= tokens) break;
+        const int t = (int)row0 + u, seq = seq_of_token[t];
+        if ((t - cu_seqlens[seq]) % DR_MINI != 0) continue;
+        const int n = min(DR_MINI, cu_seqlens[seq + 1] - t);
+        // products: 28 of keys (j < i) in one round of 32, 36 of queries and keys (j <= i) in the rest
+        float pk[32], pq[32], px[4];
+#pragma unroll
+        for (int v = 0; v < 32; ++v) { pk[v] = 0.f; pq[v] = 0.f; }
+#pragma unroll
+        for (int v = 0; v < 4; ++v) px[v] = 0.f;
+        for (int d = lane; d < D; d += 32) {
+            float kr[DR_MINI], qr[DR_MINI];
+#pragma unroll
+            for (int r = 0; r < DR_MINI; ++r) {
+                const float* src = y + (size_t)(t + r) * C + kvh * D + d;
+                qr[r] = r < n ? src[0] : 0.f;
+                kr[r] = r < n ? src[G * D] : 0.f;
+            }
+#pragma unroll
+            for (int a = 0; a < DR_MINI; ++a)
+#pragma unroll
+                for (int b = 0; b <= a; ++b) {
+                    // (row a starts at a (a - 1) / 2 among the keys' products and at a (a + 1) / 2 among the others)
+                    const int vk = a * (a - 1) / 2 + b, vq = a * (a + 1) / 2 + b;
+                    if (b < a) pk[vk < 0 ? 0 : vk] = fmaf(kr[a], kr[b], pk[vk < 0 ? 0 : vk]);
+                    if (vq < 32) pq[vq & 31] = fmaf(qr[a], kr[b], pq[vq & 31]);
+                    else px[(vq - 32) & 3] = fmaf(qr[a], kr[b], px[(vq - 32) & 3]);
+                }
+        }
+#pragma unroll
+        for (int v = 0; v < 4; ++v) pk[28 + v] = px[v];   // (the last four of the second kind fill up the first round)
+        const float sk = dr_sums<4, false>(pk, lane), sq = dr_sums<4, false>(pq, lane);
+        __syncwarp();
+        if (lane < 28) kk[lane] = sk; else qk[32 + lane - 28] = sk;
+        qk[lane] = sq;
+        __syncwarp();
+        for (int h0 = kvh * (H / G); h0 < (kvh + 1) * (H / G); h0 += 4) {   // four heads at a time, eight lanes each
+            const int hs = lane >> 3, h = h0 + hs;
+            const bool mine = h < (kvh + 1) * (H / G), there = mine && i < n;
+            float g = 1.f, beta = 0.f;
+            if (there) {
+                g = expf(neg_exp_a[h] * dr_softplus(ab[(size_t)(t + i) * ldab + a_col + h] + dt_bias[h]));
+                beta = 1.f / (1.f + expf(-ab[(size_t)(t + i) * ldab + b_col + h]));
+            }
+            float gs[DR_MINI], rho[DR_MINI], gamma = 1.f, after = 1.f;
+#pragma unroll
+            for (int j = 0; j < DR_MINI; ++j) gs[j] = __shfl_sync(0xffffffffu, g, j, 8);
+#pragma unroll
+            for (int j = DR_MINI - 1; j >= 0; --j) {   // rho[j]: the decays after j up to this token
+                rho[j] = j >= i ? 1.f : rho[j + 1 < DR_MINI ? j + 1 : j] * gs[j + 1 < DR_MINI ? j + 1 : j];
+                if (j > i) after *= gs[j]; else gamma *= gs[j];
+            }
+            float* A = a_s[warp][hs];
+            __syncwarp();
+#pragma unroll
+            for (int j = 0; j < DR_MINI; ++j) A[i * 8 + j] = j < i ? beta * rho[j] * kk[i * (i - 1) / 2 + j] : 0.f;
+            __syncwarp();
+            float T[DR_MINI];   // column i of the inverse
+#pragma unroll
+            for (int a = 0; a < DR_MINI; ++a) {
+                float s = a == i ? 1.f : 0.f;
+#pragma unroll
+                for (int l = 0; l < a; ++l) s = fmaf(-A[a * 8 + l], T[l], s);
+                T[a] = a < i ? 0.f : s;
+            }
+            if (mine) {
+                if (i < n) {
+                    float* dst = coef + ((size_t)(t + i) * H + h) * DR_COEF;
+                    *reinterpret_cast<float4*>(dst) = make_float4(beta, beta * gamma, gamma, after);
+#pragma unroll
+                    for (int j = 0; j < DR_MINI; ++j) dst[12 + j] = j <= i ? rho[j] * qk[i * (i + 1) / 2 + j] : 0.f;
+                }
+#pragma unroll
+                for (int a = 0; a < DR_MINI; ++a)
+                    if (a < n) coef[((size_t)(t + a) * H + h) * DR_COEF + 4 + i] = T[a];
+            }
+        }
+        __syncwarp();
+    }
+}
+
+// ---- the recurrence ----
+// A block owns COLS columns of one head's state of one request, a warp CC of them (four, or two where there are few heads: then
+// more warps share the SMs); lane l of the warp holds the rows RL l .. RL l + RL - 1 of its columns in registers, in pairs
+// of rows (`fma.rn.f32x2`).  Per mini-chunk a lane forms its part of the products of eight keys and eight queries with the
+// columns (in an order of the tokens of its own), the 8 CC of either kind are summed over the lanes together, and lane 8 c + i ends
+// with those of token i and column c.
+// u = (I + A)^-1 r is then eight products of numbers that the column's eight lanes exchange, and its multiples go through shared
+// memory to all lanes for the update.  Tokens are staged DR_CHUNK at a time by asynchronous copies, a chunk ahead.  Rows past D
+// are zeros, tokens past a request's last have zero coefficients: they change nothing.
+#define DR_VROW(COLS) ((COLS) + 4)   // (a staged token's values lie 20 or 12 numbers apart: eight tokens by four columns miss each other's banks)
 #define DR_CHUNK 16
-#define DR_COEF 12
-#define DR_SMEM(DP) (sizeof(float) * 2 * DR_CHUNK * (2 * (DP) + DR_COLS + DR_COEF))
+#define DR_SMEM(DP, COLS) (sizeof(float) * (2 * DR_CHUNK * (2 * (DP) + DR_VROW(COLS) + DR_COEF) + 2 * DR_MINI * (COLS) * 2))
 
 __device__ __forceinline__ void dr_copy4(float* dst, const float* src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
-struct DrGates {   // what a token's coefficients are made from
-    float a, b, kk[3], qk[4];
-};
+typedef unsigned long long dr_pair;   // two floats in a register pair
+__device__ __forceinline__ dr_pair dr_pack(float lo, float hi) {
+    dr_pair r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ void dr_unpack(dr_pair v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ dr_pair dr_fma2(dr_pair a, dr_pair b, dr_pair c) {
+    dr_pair r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ dr_pair dr_mul2(dr_pair a, dr_pair b) {
+    dr_pair r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+// P pairs of floats from shared memory (8 P bytes, aligned to their number).
+template <int P> __device__ __forceinline__ void dr_pairs(const float* p, dr_pair (&v)[P]) {
+    if constexpr (P == 1) {
+        v[0] = *reinterpret_cast<const dr_pair*>(p);
+    } else {
+#pragma unroll
+        for (int e = 0; e < P; e += 2) {
+            const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(p + 2 * e);
+            v[e] = a.x;
+            v[e + 1] = a.y;
+        }
+    }
+}
 
-template <int R>
-__global__ void __launch_bounds__(DR_WARPS * 32)
-delta_walk_kernel(const float* __restrict__ y, const float* __restrict__ dots, const float* __restrict__ ab, int ldab, int a_col,
-                  int b_col, const float* __restrict__ neg_exp_a, const float* __restrict__ dt_bias, float* __restrict__ state,
-                  float* __restrict__ ring, const void* __restrict__ x, int ldx, int x_bf16, const int* __restrict__ cu_seqlens,
-                  const int* __restrict__ state_slots, const int* __restrict__ positions, float* __restrict__ out, int G, int D,
-                  int H, int Dv, int taps) {
+template <int RL, int CC, int COLS>
+__global__ void __launch_bounds__(COLS / CC * 32, 1)
+delta_walk_kernel(const float* __restrict__ y, const float* __restrict__ coef, float* __restrict__ state, float* __restrict__ ring,
+                  const void* __restrict__ x, int ldx, int x_bf16, const int* __restrict__ cu_seqlens,
+                  const int* __restrict__ state_slots, const int* __restrict__ positions, float* __restrict__ out, int G, int D, int H,
+                  int Dv, int taps) {
     extern __shared__ __align__(16) float dr_smem[];
-    constexpr int DP = 8 * R;
+    constexpr int DP = 32 * RL, P = RL / 2, THREADS = COLS / CC * 32, NV = 8 * CC, VROW = DR_VROW(COLS);
     float* q_s = dr_smem;                              // [2][DR_CHUNK][DP]
     float* k_s = q_s + 2 * DR_CHUNK * DP;              // [2][DR_CHUNK][DP]
-    float* v_s = k_s + 2 * DR_CHUNK * DP;              // [2][DR_CHUNK][DR_COLS]
-    float* c_s = v_s + 2 * DR_CHUNK * DR_COLS;         // [2][DR_CHUNK][DR_COEF]
-    const int col0 = blockIdx.x * DR_COLS, h = blockIdx.y, seq = blockIdx.z;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, li = lane & 7;
+    float* v_s = k_s + 2 * DR_CHUNK * DP;              // [2][DR_CHUNK][VROW]
+    float* c_s = v_s + 2 * DR_CHUNK * VROW;         // [2][DR_CHUNK][DR_COEF]
+    float* u_s = c_s + 2 * DR_CHUNK * DR_COEF;         // [warps][2][DR_MINI][CC] twice each
+    const int col0 = blockIdx.x * COLS, h = blockIdx.y, seq = blockIdx.z;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, ti = lane & 7, tc = (lane >> 3) & (CC - 1);
     const int kvh = h / (H / G), C = 2 * G * D + H * Dv;
-    const int cl = warp * 4 + (lane >> 3), col = col0 + cl;
-    const float neg_a = neg_exp_a[h], bias = dt_bias[h];
-    for (int i = threadIdx.x; i < 2 * DR_CHUNK * (2 * DP + DR_COLS); i += DR_WARPS * 32) dr_smem[i] = 0.f;
+    for (int i = threadIdx.x; i < 2 * DR_CHUNK * (2 * DP + VROW + DR_COEF); i += THREADS) dr_smem[i] = 0.f;
     pdl_wait();
     pdl_trigger();
     const int t0 = cu_seqlens[seq], t1 = cu_seqlens[seq + 1], slot = state_slots[seq];
     const bool wide = ((D | C | Dv) & 3) == 0 && !(((uintptr_t)y) & 15);
-    float* st = state + (((size_t)slot * H + h) * Dv + (col < Dv ? col : 0)) * D;
-    float S[R];
+    float* st = state + ((size_t)slot * H + h) * (size_t)Dv * D;
+    dr_pair S[CC][P];
 #pragma unroll
-    for (int r = 0; r < R; ++r) S[r] = 0.f;
-    if (col < Dv) {
+    for (int c = 0; c < CC; ++c) {
+        const int col = col0 + warp * CC + c;
+        float s[RL];
 #pragma unroll
-        for (int j = 0; j < R / 4; ++j) {
-            const int d = 4 * li + 32 * j;
-            if ((D & 3) == 0) {
-                if (d < D) {
-                    const float4 s4 = *reinterpret_cast<const float4*>(st + d);
-                    S[4 * j] = s4.x; S[4 * j + 1] = s4.y; S[4 * j + 2] = s4.z; S[4 * j + 3] = s4.w;
-                }
-            } else {
+        for (int r = 0; r < RL; ++r) s[r] = col < Dv && RL * lane + r < D ? st[(size_t)col * D + RL * lane + r] : 0.f;
 #pragma unroll
-                for (int e = 0; e < 4; ++e)
-                    if (d + e < D) S[4 * j + e] = st[d + e];
-            }
-        }
+        for (int p = 0; p < P; ++p) S[c][p] = dr_pack(s[2 * p], s[2 * p + 1]);
     }
     __syncthreads();   // (the zeros are there before the first copies)
 
     auto stage = [&](int buf, int tb) {
         const int n = min(DR_CHUNK, t1 - tb);
-        float *qd = q_s + buf * DR_CHUNK * DP, *kd = k_s + buf * DR_CHUNK * DP, *vd = v_s + buf * DR_CHUNK * DR_COLS;
-        const int vn = min(DR_COLS, Dv - col0);
+        float *qd = q_s + buf * DR_CHUNK * DP, *kd = k_s + buf * DR_CHUNK * DP, *vd = v_s + buf * DR_CHUNK * VROW;
+        float* cd = c_s + buf * DR_CHUNK * DR_COEF;
+        const int vn = min(COLS, Dv - col0);
+        if (wide && D == DP && n == DR_CHUNK && vn == COLS) {   // (sizes that are known: no divisions)
+            const float* src0 = y + (size_t)tb * C + kvh * D;
+#pragma unroll
+            for (int it = 0; it < (DR_CHUNK * DP / 4 + THREADS - 1) / THREADS; ++it) {
+                const int i = threadIdx.x + it * THREADS, tt = i / (DP / 4), d = (i % (DP / 4)) * 4;
+                if (DR_CHUNK * DP / 4 % THREADS == 0 || i < DR_CHUNK * DP / 4) {
+                    cp_async16(qd + tt * DP + d, src0 + (size_t)tt * C + d);
+                    cp_async16(kd + tt * DP + d, src0 + (size_t)tt * C + G * D + d);
+                }
+            }
+            if (threadIdx.x < DR_CHUNK * COLS / 4) {
+                const int tt = threadIdx.x / (COLS / 4), c = (threadIdx.x % (COLS / 4)) * 4;
+                cp_async16(vd + tt * VROW + c, y + (size_t)(tb + tt) * C + 2 * G * D + h * Dv + col0 + c);
+            }
+            static_assert(THREADS >= DR_CHUNK * (DR_COEF / 4) && THREADS >= DR_CHUNK * COLS / 4, "a thread copies one piece of the coefficients and values");
+            if (threadIdx.x < DR_CHUNK * (DR_COEF / 4)) {
+                const int tt = threadIdx.x / (DR_COEF / 4), c = (threadIdx.x % (DR_COEF / 4)) * 4;
+                cp_async16(cd + tt * DR_COEF + c, coef + ((size_t)(tb + tt) * H + h) * DR_COEF + c);
+            }
+            cp_async_commit();
+            return;
+        }
         if (wide) {
             const int d4 = D >> 2, v4 = vn >> 2;
-            for (int i = threadIdx.x; i < n * d4; i += DR_WARPS * 32) {
+            for (int i = threadIdx.x; i < n * d4; i += THREADS) {
                 const int tt = i / d4, d = (i - tt * d4) * 4;
                 const float* src = y + (size_t)(tb + tt) * C + kvh * D + d;
                 cp_async16(qd + tt * DP + d, src);
                 cp_async16(kd + tt * DP + d, src + G * D);
             }
-            for (int i = threadIdx.x; i < n * v4; i += DR_WARPS * 32) {
+            for (int i = threadIdx.x; i < n * v4; i += THREADS) {
                 const int tt = i / v4, c = (i - tt * v4) * 4;
-                cp_async16(vd + tt * DR_COLS + c, y + (size_t)(tb + tt) * C + 2 * G * D + h * Dv + col0 + c);
+                cp_async16(vd + tt * VROW + c, y + (size_t)(tb + tt) * C + 2 * G * D + h * Dv + col0 + c);
             }
         } else {
-            for (int i = threadIdx.x; i < n * D; i += DR_WARPS * 32) {
+            for (int i = threadIdx.x; i < n * D; i += THREADS) {
                 const int tt = i / D, d = i - tt * D;
                 const float* src = y + (size_t)(tb + tt) * C + kvh * D + d;
                 dr_copy4(qd + tt * DP + d, src);
                 dr_copy4(kd + tt * DP + d, src + G * D);
             }
-            for (int i = threadIdx.x; i < n * vn; i += DR_WARPS * 32) {
+            for (int i = threadIdx.x; i < n * vn; i += THREADS) {
                 const int tt = i / vn, c = i - tt * vn;
-                dr_copy4(vd + tt * DR_COLS + c, y + (size_t)(tb + tt) * C + 2 * G * D + h * Dv + col0 + c);
+                dr_copy4(vd + tt * VROW + c, y + (size_t)(tb + tt) * C + 2 * G * D + h * Dv + col0 + c);
             }
         }
-        for (int i = threadIdx.x; i < (DR_CHUNK - n) * DP; i += DR_WARPS * 32) {
+        for (int i = threadIdx.x; i < n * (DR_COEF / 4); i += THREADS) {
+            const int tt = i / (DR_COEF / 4), c = (i - tt * (DR_COEF / 4)) * 4;
+            cp_async16(cd + tt * DR_COEF + c, coef + ((size_t)(tb + tt) * H + h) * DR_COEF + c);
+        }
+        for (int i = threadIdx.x; i < (DR_CHUNK - n) * DP; i += THREADS) {
             qd[n * DP + i] = 0.f;
             kd[n * DP + i] = 0.f;
         }
-        for (int i = threadIdx.x; i < (DR_CHUNK - n) * DR_COLS; i += DR_WARPS * 32) vd[n * DR_COLS + i] = 0.f;
+        for (int i = threadIdx.x; i < (DR_CHUNK - n) * VROW; i += THREADS) vd[n * VROW + i] = 0.f;
+        for (int i = threadIdx.x; i < (DR_CHUNK - n) * DR_COEF; i += THREADS) cd[n * DR_COEF + i] = 0.f;
         cp_async_commit();
     };
-    auto ask = [&](DrGates& g, int tb) {   // lane tt: token tb + tt
-        const int t = tb + lane;
-        if (lane < DR_CHUNK && t < t1) {
-            g.a = ab[(size_t)t * ldab + a_col + h];
-            g.b = ab[(size_t)t * ldab + b_col + h];
-            const float* d = dots + ((size_t)t * G + kvh) * DR_DOTS;
-#pragma unroll
-            for (int i = 0; i < 3; ++i) g.kk[i] = d[i];
-#pragma unroll
-            for (int i = 0; i < 4; ++i) g.qk[i] = d[3 + i];
-        }
-    };
-    auto coefficients = [&](const DrGates& g, int buf, int tb) {
-        const bool there = lane < DR_CHUNK && tb + lane < t1;
-        const float gt = there ? expf(neg_a * dr_softplus(g.a + bias)) : 1.f;
-        const float beta = there ? 1.f / (1.f + expf(-g.b)) : 0.f;
-        const int i = lane & 3;
-        float gs[4];
-#pragma unroll
-        for (int j = 0; j < 4; ++j) gs[j] = __shfl_sync(0xffffffffu, gt, (lane & ~3) + j);
-        float gamma = 1.f, after = 1.f, rho[4] = {1.f, 1.f, 1.f, 1.f};   // rho[j]: decays after j up to i
-#pragma unroll
-        for (int l = 0; l < 4; ++l) {
-            if (l <= i) gamma *= gs[l]; else after *= gs[l];
-#pragma unroll
-            for (int j = 0; j < 4; ++j)
-                if (l > j && l <= i) rho[j] *= gs[l];
-        }
-        float bk[3], qk[4];
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            // the product with token j of the mini-chunk, i - j tokens back
-            float kd = 0.f, qd = 0.f;
-#pragma unroll
-            for (int b = 0; b < 4; ++b)
-                if (i - j == b) { qd = g.qk[b]; if (b) kd = g.kk[b > 0 ? b - 1 : 0]; }
-            if (j < 3) bk[j] = there && j < i ? beta * rho[j] * kd : 0.f;
-            qk[j] = there && j <= i ? rho[j] * qd : 0.f;
-        }
-        if (lane < DR_CHUNK) {
-            float4* dst = reinterpret_cast<float4*>(c_s + (buf * DR_CHUNK + lane) * DR_COEF);
-            dst[0] = make_float4(beta * gamma, beta, after, gamma);
-            dst[1] = make_float4(bk[0], bk[1], bk[2], 0.f);
-            dst[2] = make_float4(qk[0], qk[1], qk[2], qk[3]);
-        }
-    };
 
-    if (t1 > t0) {
-        stage(0, t0);
-        if (warp == 0) {
-            DrGates g = {};
-            ask(g, t0);
-            coefficients(g, 0, t0);
-        }
-    }
-    int buf = 0, turn = 1;
-    for (int tb = t0; tb < t1; tb += DR_CHUNK, buf ^= 1, turn = (turn + 1) & (DR_WARPS - 1)) {
+    int off[DR_MINI];   // where a lane's slot s finds its rows: token s xor (lane mod 8) of the mini-chunk
+#pragma unroll
+    for (int i = 0; i < DR_MINI; ++i) off[i] = (i ^ ti) * DP + RL * lane;
+    if (t1 > t0) stage(0, t0);
+    int buf = 0;
+    for (int tb = t0; tb < t1; tb += DR_CHUNK, buf ^= 1) {
         const int n = min(DR_CHUNK, t1 - tb);
-        const bool more = tb + DR_CHUNK < t1;
         cp_async_wait<0>();
         __syncthreads();
-        DrGates g = {};
-        if (more) {
-            stage(buf ^ 1, tb + DR_CHUNK);
-            if (warp == turn) ask(g, tb + DR_CHUNK);
-        }
-        const float *qb = q_s + buf * DR_CHUNK * DP + 4 * li, *kb = k_s + buf * DR_CHUNK * DP + 4 * li;
-        const float *vb = v_s + buf * DR_CHUNK * DR_COLS + cl, *cb = c_s + buf * DR_CHUNK * DR_COEF;
+        if (tb + DR_CHUNK < t1) stage(buf ^ 1, tb + DR_CHUNK);
         for (int m = 0; m < n; m += DR_MINI) {
-            constexpr bool KEEP = R <= 16;   // the keys stay in registers from the products to the update
-            float kreg[KEEP ? DR_MINI : 1][KEEP ? R : 1];
-            float p[8];
-#pragma unroll
-            for (int i = 0; i < 8; ++i) p[i] = 0.f;
-#pragma unroll
-            for (int j = 0; j < R / 4; ++j) {
-#pragma unroll
-                for (int i = 0; i < DR_MINI; ++i) {
-                    const float4 k4 = *reinterpret_cast<const float4*>(kb + (m + i) * DP + 32 * j);
-                    const float4 q4 = *reinterpret_cast<const float4*>(qb + (m + i) * DP + 32 * j);
-                    if (KEEP) {
-                        kreg[KEEP ? i : 0][KEEP ? 4 * j : 0] = k4.x;
-                        kreg[KEEP ? i : 0][KEEP ? 4 * j + 1 : 0] = k4.y;
-                        kreg[KEEP ? i : 0][KEEP ? 4 * j + 2 : 0] = k4.z;
-                        kreg[KEEP ? i : 0][KEEP ? 4 * j + 3 : 0] = k4.w;
-                    }
-                    p[i] = fmaf(S[4 * j], k4.x, p[i]); p[i] = fmaf(S[4 * j + 1], k4.y, p[i]);
-                    p[i] = fmaf(S[4 * j + 2], k4.z, p[i]); p[i] = fmaf(S[4 * j + 3], k4.w, p[i]);
-                    p[4 + i] = fmaf(S[4 * j], q4.x, p[4 + i]); p[4 + i] = fmaf(S[4 * j + 1], q4.y, p[4 + i]);
-                    p[4 + i] = fmaf(S[4 * j + 2], q4.z, p[4 + i]); p[4 + i] = fmaf(S[4 * j + 3], q4.w, p[4 + i]);
-                }
-            }
-            // the eight sums over the column's eight lanes: lane i ends with the sum number i
-            float a4[4], a2[2], mine;
-            const bool h4 = lane & 4, h2 = lane & 2, h1 = lane & 1;
-#pragma unroll
-            for (int i = 0; i < 4; ++i) a4[i] = (h4 ? p[4 + i] : p[i]) + __shfl_xor_sync(0xffffffffu, h4 ? p[i] : p[4 + i], 4);
-#pragma unroll
-            for (int i = 0; i < 2; ++i) a2[i] = (h2 ? a4[2 + i] : a4[i]) + __shfl_xor_sync(0xffffffffu, h2 ? a4[i] : a4[2 + i], 2);
-            mine = (h1 ? a2[1] : a2[0]) + __shfl_xor_sync(0xffffffffu, h1 ? a2[0] : a2[1], 1);
-            float u[4], wu[4], gamma_all = 1.f;
+            const float *qb = q_s + (buf * DR_CHUNK + m) * DP, *kb = k_s + (buf * DR_CHUNK + m) * DP;
+            const float* cb = c_s + (buf * DR_CHUNK + m + ti) * DR_COEF;
+            constexpr bool KEEP = RL <= 4;   // the keys stay in registers from the products to the update
+            dr_pair kreg[KEEP ? DR_MINI : 1][P];
+            float pk[NV], pq[NV];
 #pragma unroll
             for (int i = 0; i < DR_MINI; ++i) {
-                const float4 c0 = *reinterpret_cast<const float4*>(cb + (m + i) * DR_COEF);
-                const float kS = __shfl_sync(0xffffffffu, mine, i, 8);
-                float v = fmaf(-c0.x, kS, c0.y * vb[(m + i) * DR_COLS]);
-                if (i > 0) {
-                    const float4 c1 = *reinterpret_cast<const float4*>(cb + (m + i) * DR_COEF + 4);
-                    v = fmaf(-c1.x, u[0], v);
-                    if (i > 1) v = fmaf(-c1.y, u[1], v);
-                    if (i > 2) v = fmaf(-c1.z, u[2], v);
-                }
-                u[i] = v;
-                wu[i] = c0.z * v;
-                if (i == DR_MINI - 1) gamma_all = c0.w;
-            }
-            if (li >= 4) {
-                const int tt = m + li - 4;
-                const float gamma = cb[tt * DR_COEF + 3];
-                const float4 c2 = *reinterpret_cast<const float4*>(cb + tt * DR_COEF + 8);
-                float o = gamma * mine;
-                o = fmaf(c2.x, u[0], o); o = fmaf(c2.y, u[1], o); o = fmaf(c2.z, u[2], o); o = fmaf(c2.w, u[3], o);
-                if (tt < n && col < Dv) out[((size_t)(tb + tt) * H + h) * Dv + col] = o;
-            }
+                dr_pair k2[P];
+                dr_pairs<P>(kb + off[i], k2);
 #pragma unroll
-            for (int j = 0; j < R / 4; ++j) {
+                for (int e = 0; e < P; ++e)
+                    if (KEEP) kreg[KEEP ? i : 0][e] = k2[e];
 #pragma unroll
-                for (int e = 0; e < 4; ++e) S[4 * j + e] *= gamma_all;
+                for (int c = 0; c < CC; ++c) {
+                    dr_pair a = dr_mul2(S[c][0], k2[0]);
 #pragma unroll
-                for (int i = 0; i < DR_MINI; ++i) {
-                    float kk[4];
-                    if (KEEP) {
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) kk[e] = kreg[KEEP ? i : 0][KEEP ? 4 * j + e : 0];
-                    } else {
-                        const float4 k4 = *reinterpret_cast<const float4*>(kb + (m + i) * DP + 32 * j);
-                        kk[0] = k4.x; kk[1] = k4.y; kk[2] = k4.z; kk[3] = k4.w;
-                    }
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) S[4 * j + e] = fmaf(kk[e], wu[i], S[4 * j + e]);
+                    for (int e = 1; e < P; ++e) a = dr_fma2(S[c][e], k2[e], a);
+                    float lo, hi;
+                    dr_unpack(a, lo, hi);
+                    pk[c * 8 + i] = lo + hi;
                 }
             }
+            const float kS = dr_sums<CC, true>(pk, lane);
+#pragma unroll
+            for (int i = 0; i < DR_MINI; ++i) {
+                dr_pair q2[P];
+                dr_pairs<P>(qb + off[i], q2);
+#pragma unroll
+                for (int c = 0; c < CC; ++c) {
+                    dr_pair a = dr_mul2(S[c][0], q2[0]);
+#pragma unroll
+                    for (int e = 1; e < P; ++e) a = dr_fma2(S[c][e], q2[e], a);
+                    float lo, hi;
+                    dr_unpack(a, lo, hi);
+                    pq[c * 8 + i] = lo + hi;
+                }
+            }
+            // lane 8 c + i: token m + i, column c of the warp
+            const float4 c0 = *reinterpret_cast<const float4*>(cb);
+            const float4 ta = *reinterpret_cast<const float4*>(cb + 4), tb4 = *reinterpret_cast<const float4*>(cb + 8);
+            const float4 pa = *reinterpret_cast<const float4*>(cb + 12), pb4 = *reinterpret_cast<const float4*>(cb + 16);
+            const float trow[8] = {ta.x, ta.y, ta.z, ta.w, tb4.x, tb4.y, tb4.z, tb4.w};
+            const float prow[8] = {pa.x, pa.y, pa.z, pa.w, pb4.x, pb4.y, pb4.z, pb4.w};
+            const float v = v_s[(buf * DR_CHUNK + m + ti) * VROW + warp * CC + tc];
+            const float r = fmaf(c0.x, v, -c0.y * kS);
+            float u0 = 0.f, u1 = 0.f;
+#pragma unroll
+            for (int j = 0; j < 8; j += 2) {
+                u0 = fmaf(trow[j], __shfl_sync(0xffffffffu, r, j, 8), u0);
+                u1 = fmaf(trow[j + 1], __shfl_sync(0xffffffffu, r, j + 1, 8), u1);
+            }
+            const float u = u0 + u1, wu = c0.w * u;
+            float* us = u_s + (warp * 2 + ((m / DR_MINI) & 1)) * DR_MINI * 2 * CC;
+            if (lane < NV) *reinterpret_cast<float2*>(us + (ti * CC + tc) * 2) = make_float2(wu, wu);
+            // (token 0 of the mini-chunk is always there: its decay times those after it is the decay over the mini-chunk)
+            const float gamma = __shfl_sync(0xffffffffu, c0.z * c0.w, 0, 8);
+            const dr_pair gamma2 = dr_pack(gamma, gamma);
+            __syncwarp();
+#pragma unroll
+            for (int c = 0; c < CC; ++c)
+#pragma unroll
+                for (int e = 0; e < P; ++e) S[c][e] = dr_mul2(S[c][e], gamma2);
+#pragma unroll
+            for (int i = 0; i < DR_MINI; ++i) {
+                dr_pair w2[CC], k2[P];
+                dr_pairs<CC>(us + (i ^ ti) * 2 * CC, w2);
+                if (KEEP) {
+#pragma unroll
+                    for (int e = 0; e < P; ++e) k2[e] = kreg[KEEP ? i : 0][e];
+                } else {
+                    dr_pairs<P>(kb + off[i], k2);
+                }
+#pragma unroll
+                for (int c = 0; c < CC; ++c)
+#pragma unroll
+                    for (int e = 0; e < P; ++e) S[c][e] = dr_fma2(k2[e], w2[c], S[c][e]);
+            }
+            const float qS = dr_sums<CC, true>(pq, lane);
+            float o0 = c0.z * qS, o1 = 0.f;
+#pragma unroll
+            for (int j = 0; j < 8; j += 2) {
+                o0 = fmaf(prow[j], __shfl_sync(0xffffffffu, u, j, 8), o0);
+                o1 = fmaf(prow[j + 1], __shfl_sync(0xffffffffu, u, j + 1, 8), o1);
+            }
+            const int col = col0 + warp * CC + tc;
+            if (lane < NV && m + ti < n && col < Dv) out[((size_t)(tb + m + ti) * H + h) * Dv + col] = o0 + o1;
         }
-        if (more && warp == turn) coefficients(g, buf ^ 1, tb + DR_CHUNK);
     }
-    if (col < Dv) {
 #pragma unroll
-        for (int j = 0; j < R / 4; ++j) {
-            const int d = 4 * li + 32 * j;
-            if ((D & 3) == 0) {
-                if (d < D) *reinterpret_cast<float4*>(st + d) = make_float4(S[4 * j], S[4 * j + 1], S[4 * j + 2], S[4 * j + 3]);
-            } else {
+    for (int c = 0; c < CC; ++c) {
+        const int col = col0 + warp * CC + c;
 #pragma unroll
-                for (int e = 0; e < 4; ++e)
-                    if (d + e < D) st[d + e] = S[4 * j + e];
-            }
+        for (int p = 0; p < P; ++p) {
+            float lo, hi;
+            dr_unpack(S[c][p], lo, hi);
+            const int d = RL * lane + 2 * p;
+            if (col < Dv && d < D) st[(size_t)col * D + d] = lo;
+            if (col < Dv && d + 1 < D) st[(size_t)col * D + d + 1] = hi;
         }
     }
     // the request's last inputs of the convolutions, its blocks sharing the channels
     const int part = blockIdx.y * gridDim.x + blockIdx.x, parts = gridDim.x * gridDim.y;
-    for (int c = part * DR_WARPS * 32 + threadIdx.x; c < C; c += parts * DR_WARPS * 32)
+    for (int c = part * THREADS + threadIdx.x; c < C; c += parts * THREADS)
         for (int t = max(t0, t1 - (taps - 1)); t < t1; ++t)
             ring[((size_t)slot * taps + positions[t] % taps) * C + c] =
                 x_bf16 ? to_f32(((const bf16*)x)[(size_t)t * ldx + c]) : ((const float*)x)[(size_t)t * ldx + c];
 }
 
 // neg_exp_a, dt_bias float32 [H]: -exp(A_log) and the decay's offset.  ab float32 [tokens, ldab]: a and b of head h in columns
-// a_col + h, b_col + h.  y, dots: from `vx_delta_conv` of the same step; x, ldx: what that read.  state float32
-// [slots, H, Dv, D], ring float32 [slots, taps, C]: read and written.  out float32 [tokens, H * Dv].
-extern "C" int vx_delta_walk(const float* y, const float* dots, const float* ab, int ldab, int a_col, int b_col,
-                             const float* neg_exp_a, const float* dt_bias, float* state, float* ring, const void* x, int ldx,
+// a_col + h, b_col + h.  y: from `vx_delta_conv` of the same step.  coef float32 [tokens, H, 20], 16-byte aligned.
+extern "C" int vx_delta_coef(const float* y, const float* ab, int ldab, int a_col, int b_col, const float* neg_exp_a,
+                             const float* dt_bias, const int* seq_of_token, const int* cu_seqlens, float* coef, int tokens, int G, int D,
+                             int H, int Dv, cudaStream_t stream) {
+    if (tokens <= 0) return VX_OK;
+    if (G <= 0 || D <= 0 || H <= 0 || Dv <= 0 || H % G || ldab < a_col + H || ldab < b_col + H || a_col < 0 || b_col < 0) return VX_ERR_SHAPE;
+    if (((uintptr_t)coef) & 15) return VX_ERR_ALIGN;
+    const long long warps = (long long)((tokens + DR_MINI - 1) / DR_MINI) * G;
+    if (warps / DR_CW > 0x7ffffff0LL) return VX_ERR_LIMIT;
+    VX_LAUNCH_K(VX_K_ELEMENTWISE, delta_coef_kernel, (unsigned)((warps + DR_CW - 1) / DR_CW), DR_CW * 32, 0, stream, y, ab, ldab, a_col,
+                b_col, neg_exp_a, dt_bias, seq_of_token, cu_seqlens, coef, tokens, G, D, H, 2 * G * D + H * Dv);
+    VX_LAUNCH_CHECK();
+    return VX_OK;
+}
+
+// y, coef: from the two entries above; x, ldx: what `vx_delta_conv` read.  state float32 [slots, H, Dv, D], ring float32
+// [slots, taps, C]: read and written.  out float32 [tokens, H * Dv].  layout: warps of two columns in blocks of 8 (1)
+// or 16 (2), warps of four in blocks of 16 (3), or 0 for the kernel's choice.
+extern "C" int vx_delta_walk(const float* y, const float* coef, float* state, float* ring, const void* x, int ldx,
                              const int* cu_seqlens, const int* state_slots, const int* positions, float* out, int seqs, int G, int D,
-                             int H, int Dv, int taps, int dtype, cudaStream_t stream) {
+                             int H, int Dv, int taps, int layout, int dtype, cudaStream_t stream) {
     if (seqs <= 0) return VX_OK;
-    if (G <= 0 || D <= 0 || H <= 0 || Dv <= 0 || H % G || taps <= 0) return VX_ERR_SHAPE;
-    if (ldab < a_col + H || ldab < b_col + H || a_col < 0 || b_col < 0 || ldx < 2 * G * D + H * Dv) return VX_ERR_SHAPE;
+    if (G <= 0 || D <= 0 || H <= 0 || Dv <= 0 || H % G || taps <= 0 || ldx < 2 * G * D + H * Dv) return VX_ERR_SHAPE;
     if (D > 256 || taps > DR_MAX_TAPS || seqs > 65535 || H > 65535) return VX_ERR_LIMIT;
     if (dtype != VX_F32 && dtype != VX_BF16) return VX_ERR_DTYPE;
-    static bool configured[4][VX_MAX_DEVICES];
-    dim3 grid((Dv + DR_COLS - 1) / DR_COLS, H, seqs);
-#define DR_GO(R_, SLOT)                                                                                                       \
-    do {                                                                                                                      \
-        if (int rc = vx_configure_smem(delta_walk_kernel<R_>, DR_SMEM(8 * R_), configured[SLOT])) return rc;                  \
-        VX_LAUNCH_K(VX_K_ATTENTION, (delta_walk_kernel<R_>), grid, DR_WARPS * 32, DR_SMEM(8 * R_), stream, y, dots, ab, ldab, \
-                    a_col, b_col, neg_exp_a, dt_bias, state, ring, x, ldx, dtype == VX_BF16 ? 1 : 0, cu_seqlens, state_slots, \
-                    positions, out, G, D, H, Dv, taps);                                                                       \
+    if (((uintptr_t)coef) & 15) return VX_ERR_ALIGN;
+    static bool configured[9][VX_MAX_DEVICES];
+    static int sms[VX_MAX_DEVICES];
+    // few heads: warps of two columns, in blocks of 8 or 16; many: warps of four (what a column's sums are does not depend on it)
+    const long long units = (long long)H * seqs * ((Dv + 7) / 8);
+    if (!layout) layout = units <= vx_sm_count(sms) ? 1 : (units <= 2LL * vx_sm_count(sms) ? 2 : 3);
+    if (layout < 0 || layout > 3) return VX_ERR_SHAPE;
+    const int cols = layout == 1 ? 8 : 16;
+    dim3 grid((Dv + cols - 1) / cols, H, seqs);
+#define DR_GO(RL_, CC_, COLS_, SLOT)                                                                                            \
+    do {                                                                                                                        \
+        if (int rc = vx_configure_smem(delta_walk_kernel<RL_, CC_, COLS_>, DR_SMEM(32 * RL_, COLS_), configured[SLOT])) return rc; \
+        VX_LAUNCH_K(VX_K_ATTENTION, (delta_walk_kernel<RL_, CC_, COLS_>), grid, COLS_ / CC_ * 32, DR_SMEM(32 * RL_, COLS_), stream, \
+                    y, coef, state, ring, x, ldx, dtype == VX_BF16 ? 1 : 0, cu_seqlens, state_slots, positions, out, G, D, H, Dv,  \
+                    taps);                                                                                                      \
     } while (0)
-    if (D <= 32) DR_GO(4, 3);
-    else if (D <= 64) DR_GO(8, 0);
-    else if (D <= 128) DR_GO(16, 1);
-    else DR_GO(32, 2);
+#define DR_GO_CC(RL_, SLOT)                                                                                                    \
+    do {                                                                                                                       \
+        if (layout == 1) DR_GO(RL_, 2, 8, SLOT); else if (layout == 2) DR_GO(RL_, 2, 16, SLOT + 1); else DR_GO(RL_, 4, 16, SLOT + 2); \
+    } while (0)
+    if (D <= 64) DR_GO_CC(2, 0);
+    else if (D <= 128) DR_GO_CC(4, 3);
+    else DR_GO_CC(8, 6);
+#undef DR_GO_CC
 #undef DR_GO
     VX_LAUNCH_CHECK();
     return VX_OK;

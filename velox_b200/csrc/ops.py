@@ -136,8 +136,9 @@ def _declare(lib) -> None:
         "vx_gemm_skinny_inputs": [P, P, P, I, I, I, I, I, I, I, c_longlong, I, I, P],
         "vx_moe_gemm_scaled": [P, I, P, I, P, P, P, I, P, I, I, I, I, I, I, I, I, I, P, P],
         "vx_moe_gemm_tcgen05_scaled": [P, P, P, I, I, I, I, I, I, I, I, P, P, I, P, P, P, I, P],
-        "vx_delta_conv": [P, I, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, P],
-        "vx_delta_walk": [P, P, P, I, I, I, P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, P],
+        "vx_delta_conv": [P, I, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, P],
+        "vx_delta_coef": [P, P, I, I, I, P, P, P, P, P, I, I, I, I, I, P],
+        "vx_delta_walk": [P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, P],
         "vx_delta_decode": [P, I, I, P, I, I, I, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, I, I, P],
         "vx_head_gate": [P, I, P, I, P, I, I, I, I, I, P],
         "vx_moe_route_groups": [P, I, P, P, I, I, I, I, I, P, P, P, P, P, P, P, P, P, I, I, P, I, I, F, I, P, I, I, P],
@@ -1436,7 +1437,7 @@ def low_rank_decay(x: torch.Tensor, weight_t: torch.Tensor, bias: torch.Tensor) 
 DELTA_MAX_DIM = 256      # key channels of a head that the delta rule's kernels take
 DELTA_MAX_VDIM = 4096
 DELTA_MAX_TAPS = 64
-_DELTA_DOTS = 8
+_DELTA_COEF = 20   # numbers per token and head between two of the kernels
 
 
 def _delta_check(what, x, taps_w, ring, groups, dim, heads, vdim, ab):
@@ -1458,7 +1459,7 @@ def _delta_state_check(what, state, heads, dim, vdim, *per_head):
 
 def delta_rule(x: torch.Tensor, ab: torch.Tensor, a_col: int, b_col: int, taps_w: torch.Tensor, neg_exp_a: torch.Tensor,
                dt_bias: torch.Tensor, state: torch.Tensor, ring: torch.Tensor, ctx, groups: int, dim: int, heads: int, vdim: int,
-               q_mul: float) -> torch.Tensor:
+               q_mul: float, layout: int = 0) -> torch.Tensor:
     """The gated delta rule over every request's tokens in order.  x [tokens, ..]: the projections q [groups, dim], k [groups,
     dim], v [heads, vdim] from column 0 on; each goes through a causal convolution over time (`taps_w` float32 [taps,
     channels], the last row being the current token's) and silu, q and k become unit vectors per head, q times `q_mul`.
@@ -1471,15 +1472,17 @@ def delta_rule(x: torch.Tensor, ab: torch.Tensor, a_col: int, b_col: int, taps_w
     _delta_state_check("delta_rule", state, heads, dim, vdim, neg_exp_a, dt_bias)
     tokens, dev = x.shape[0], x.device
     y = torch.empty((tokens, c), dtype=torch.float32, device=dev)
-    dots = torch.empty((tokens, groups, _DELTA_DOTS), dtype=torch.float32, device=dev)
+    coef = torch.empty((tokens, heads, _DELTA_COEF), dtype=torch.float32, device=dev)
     out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=dev)
     _check(library().vx_delta_conv(_ptr(x), x.stride(0), _ptr(taps_w), _ptr(ring), _ptr(ctx.seq_of_token), _ptr(ctx.cu_seqlens),
-                                   _ptr(ctx.state_slots), _ptr(ctx.positions), _ptr(y), _ptr(dots), tokens, groups, dim, heads,
-                                   vdim, taps, float(q_mul), dtype_code(x.dtype), _stream()), "delta_conv")
-    _check(library().vx_delta_walk(_ptr(y), _ptr(dots), _ptr(ab), ab.stride(0), int(a_col), int(b_col), _ptr(neg_exp_a),
-                                   _ptr(dt_bias), _ptr(state), _ptr(ring), _ptr(x), x.stride(0), _ptr(ctx.cu_seqlens),
+                                   _ptr(ctx.state_slots), _ptr(ctx.positions), _ptr(y), tokens, groups, dim, heads, vdim, taps,
+                                   float(q_mul), dtype_code(x.dtype), _stream()), "delta_conv")
+    _check(library().vx_delta_coef(_ptr(y), _ptr(ab), ab.stride(0), int(a_col), int(b_col), _ptr(neg_exp_a), _ptr(dt_bias),
+                                   _ptr(ctx.seq_of_token), _ptr(ctx.cu_seqlens), _ptr(coef), tokens, groups, dim, heads, vdim,
+                                   _stream()), "delta_coef")
+    _check(library().vx_delta_walk(_ptr(y), _ptr(coef), _ptr(state), _ptr(ring), _ptr(x), x.stride(0), _ptr(ctx.cu_seqlens),
                                    _ptr(ctx.state_slots), _ptr(ctx.positions), _ptr(out), ctx.n_seqs, groups, dim, heads, vdim,
-                                   taps, dtype_code(x.dtype), _stream()), "delta_walk")
+                                   taps, int(layout), dtype_code(x.dtype), _stream()), "delta_walk")
     return out
 
 
