@@ -1192,23 +1192,24 @@ def birelix_kernels(pk, sz):
     def nxt(ws):
         turn[0] += 1
         return ws[turn[0] % len(ws)]
-    y, coef, o = rnd(T, ch), torch.empty((T, HL, 20), device=dev), torch.empty((T, HL * Dv), device=dev)
+    qk, vv = rnd(GL, T, 2, 128), rnd(HL, Dv // 8, T, 8)
+    coef, o, word = torch.empty((HL, T, 20), device=dev), torch.empty((T, HL * Dv), device=dev), ops._error_word(torch.device(dev))
     lib, p = ops.library(), ops._ptr
     row("short convolutions, silu, unit vectors, %d tokens" % T, us(lambda: ops._check(lib.vx_delta_conv(
-        p(x), x.stride(0), p(taps), p(ring[0]), p(seq_t), p(cu), p(slot0), p(pos_t), p(y), T, GL, D, HL, Dv, TAPS, D ** -0.5,
+        p(x), x.stride(0), p(taps), p(ring[0]), p(seq_t), p(cu), p(slot0), p(pos_t), p(qk), p(vv), T, GL, D, HL, Dv, TAPS, D ** -0.5,
         ops.VX_BF16, ops._stream()), "delta_conv")), 0.0, T * ch * 6.0)
     low, w2t = rnd(T, 64), rnd(64, ch) * 0.1
     row("Negilorn: decays in float32 (tanh, product, exponential), %d tokens" % T, us(lambda: ops.low_rank_decay(low, w2t, taps[0].contiguous())), 0.0, T * (ch + 64) * 4.0)
     fl = T * HL * 2.0 * (32 * 2 * D + 2 * D * Dv)
     simt = T * HL * 2.0 * 3 * D * Dv
     cores = 148 * 128 * 2 * 1.965e9
-    coefs = lambda: ops._check(lib.vx_delta_coef(p(y), p(ab), ab.stride(0), HL, 0, p(nea), p(dtb), p(seq_t), p(cu), p(coef), T, GL, D, HL, Dv,
+    coefs = lambda: ops._check(lib.vx_delta_coef(p(qk), p(ab), ab.stride(0), HL, 0, p(nea), p(dtb), p(seq_t), p(cu), p(coef), T, GL, D, HL, Dv,
                                                  ops._stream()), "delta_coef")
     row("decays, step sizes, products within eight tokens and their inverse, %d tokens" % T, us(coefs), 0.0, T * (2 * GL * D + 22 * HL) * 4.0)
     ops.delta_rule(x, ab, HL, 0, taps, nea, dtb, state[0], ring[0], ctx, GL, D, HL, Dv, D ** -0.5)
     t_walk = us(lambda: ops._check(lib.vx_delta_walk(
-        p(y), p(coef), p(state[0]), p(ring[0]), p(x), x.stride(0), p(cu), p(slot0), p(pos_t),
-        p(o), 1, GL, D, HL, Dv, TAPS, 0, ops.VX_BF16, ops._stream()), "delta_walk"), 5)
+        p(qk), p(vv), p(coef), p(state[0]), p(ring[0]), p(x), x.stride(0), p(cu), p(slot0), p(pos_t),
+        p(o), T, 1, GL, D, HL, Dv, TAPS, 0, p(word), ops.VX_BF16, ops._stream()), "delta_walk"), 5)
     row("prompt delta rule: the walk, %d heads (%.2f of the float32 multiply-add rate)" % (HL, simt / (t_walk * 1e-6) / cores), t_walk, fl)
     xk = (rnd(T, 4 * HL * D) * 0.5).to(bf)
     z, st = rnd(T, HL * D) + 2.0, torch.zeros((B, HL, D, Dv), device=dev)

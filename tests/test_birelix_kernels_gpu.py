@@ -86,11 +86,11 @@ class Rule:
         ring = torch.full((slots, self.taps, self.C), float("nan"), device=DEV)
         return state, ring
 
-    def run(self, ctx, rows, state, ring, dtype):
+    def run(self, ctx, rows, state, ring, dtype, layout=0):
         from velox_b200.csrc import ops
         x = dev(np.concatenate([self.x[i][a:b] for i, a, b in rows]), dtype)
         ab = dev(np.concatenate([self.ab[i][a:b] for i, a, b in rows]))
-        return ops.delta_rule(x, ab, self.H, 0, *self.args(), state, ring, ctx, self.G, self.D, self.H, self.Dv, self.D ** -0.5)
+        return ops.delta_rule(x, ab, self.H, 0, *self.args(), state, ring, ctx, self.G, self.D, self.H, self.Dv, self.D ** -0.5, layout=layout)
 
     def decode(self, ctx, rows, state, ring, x_dtype, dtype):
         from velox_b200.csrc import ops
@@ -158,6 +158,27 @@ def test_how_a_sequence_is_cut_changes_nothing_but_rounding(G, H, D, Dv, taps):
             got = r.run(step_of([n], [at], [1]), [(0, at, at + n)], state, ring, torch.float32)
             close(got, want[at:at + n], 2e-5)
             at, k = at + n, k + 1
+
+
+@pytest.mark.parametrize("G,H,D,Dv,taps", [(2, 4, 64, 64, 4), (1, 2, 128, 40, 4), (2, 2, 12, 20, 3), (1, 2, 256, 33, 4)])
+def test_columns_a_warp_holds_change_no_bit_and_many_requests_take_more(G, H, D, Dv, taps):
+    """Both layouts of the walk, and the one the kernel chooses: two requests, then forty (more blocks than the GPU has places for
+    at once), each with the bits it has alone."""
+    lens = [37, 16] + [3 + i for i in range(38)]
+    r = Rule(G, H, D, Dv, taps, lens, 6)
+    outs = []
+    for layout in (1, 2, 0):
+        state, ring = r.buffers(40)
+        state[:] = 0.0
+        outs.append(r.run(step_of(lens[:2], [0, 0], [1, 0]), [(0, 0, 37), (1, 0, 16)], state, ring, torch.float32, layout))
+    assert torch.equal(outs[0], outs[1]) and torch.equal(outs[0], outs[2])
+    close(outs[0][:37], r.plain(0)[0].reshape(37, -1), 2e-5)
+    for layout in (1, 2, 0):
+        state, ring = r.buffers(40)
+        state[:] = 0.0
+        many = r.run(step_of(lens, [0] * 40, range(40)), [(i, 0, n) for i, n in enumerate(lens)], state, ring, torch.float32, layout)
+        assert torch.equal(many[:53], outs[0])
+        close(many[-lens[-1]:], r.plain(39)[0].reshape(lens[-1], -1), 2e-5)
 
 
 @pytest.mark.parametrize("D,Dv,T", [(64, 64, 700), (128, 32, 300), (20, 12, 700)])

@@ -14,7 +14,7 @@
 // convolutions as a ring [taps, channels]: position p lies in row p mod taps.  A token at position p reads rows p - 1 ..
 // p - taps + 1 and writes row p, which is none of those, so the blocks of a decode step need no order among them.  Rows of
 // positions before 0 count as zeros and are never read.  Channels are numbered q [G, D], k [G, D], v [H, Dv].
-#include "mma_helpers.cuh"
+#include "tcgen05_gemm.cuh"
 
 #define DR_EPS_UNIT 1e-6f
 #define DR_MINI 8      // tokens of a mini-chunk
@@ -68,7 +68,19 @@ __device__ __forceinline__ DrPlace dr_place(int t, const int* seq_of_token, cons
 }
 
 // ---- convolution, silu, unit vectors ----
-// y float32 [tokens, C] with C = 2 G D + H Dv: q as a unit vector times q_mul, k as a unit vector, v.
+// What the walk reads, in runs that one bulk copy brings: qk float32 [G, tokens, 2, DP] (q as a unit vector times q_mul, k as a
+// unit vector, zeros from D up to DP: 64, 128 or 256) and v float32 [H, ceil(Dv / 8), tokens, 8] (what lies past Dv is left alone).
+__host__ __device__ constexpr int dr_padded(int D) { return D <= 64 ? 64 : (D <= 128 ? 128 : 256); }
+// Where channel c of token t goes (c counts q [G, D], k [G, D], v [H, Dv]).
+__device__ __forceinline__ float* dr_target(float* qk, float* v, int t, int c, int tokens, int G, int D, int DP, int Dv) {
+    if (c < 2 * G * D) {
+        const int is_k = c >= G * D, r = c - is_k * G * D, g = r / D;
+        return qk + (((size_t)g * tokens + t) * 2 + is_k) * DP + (r - g * D);
+    }
+    const int r = c - 2 * G * D, h = r / Dv, col = r - h * Dv;
+    return v + (((size_t)h * ((Dv + 7) >> 3) + (col >> 3)) * tokens + t) * 8 + (col & 7);
+}
+
 // The convolution of VEC channels from c on of token t, each tap's row from the step or from the ring.
 template <typename T, int VEC>
 __device__ __forceinline__ void dr_conv_at(const T* __restrict__ x, int ldx, const float* __restrict__ w, int C, int taps, int t,
@@ -92,17 +104,16 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 delta_conv_any_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ w, const float* __restrict__ ring,
                       const int* __restrict__ seq_of_token, const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots,
-                      const int* __restrict__ positions, float* __restrict__ y, int tokens, int G, int D, int HDv, int taps, float q_mul,
-                      int units) {
+                      const int* __restrict__ positions, float* __restrict__ qk, float* __restrict__ vout, int tokens, int G, int D, int H, int Dv,
+                      int taps, float q_mul, int units) {
     pdl_wait();
     pdl_trigger();
     const long long id = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
     const int t = (int)(id / units), unit = (int)(id - (long long)t * units);
     if (t >= tokens) return;
-    const int C = 2 * G * D + HDv;
+    const int C = 2 * G * D + H * Dv, DP = dr_padded(D);
     const DrPlace at = dr_place(t, seq_of_token, cu_seqlens, state_slots, positions, ring, (size_t)taps * C);
-    float* yr = y + (size_t)t * C;
     const bool is_v = unit >= 2 * G;
     const int c0 = is_v ? 2 * G * D + (unit - 2 * G) * 256 : unit * D, n = is_v ? min(256, C - c0) : D;
     float v[8], ss = 0.f;
@@ -116,7 +127,11 @@ delta_conv_any_kernel(const T* __restrict__ x, int ldx, const float* __restrict_
     const float mul = is_v ? 1.f : rsqrtf(warp_sum(ss) + DR_EPS_UNIT) * (unit < G ? q_mul : 1.f);
 #pragma unroll
     for (int i = 0; i < 8; ++i)
-        if (lane + 32 * i < n) yr[c0 + lane + 32 * i] = v[i] * mul;
+        if (lane + 32 * i < n) *dr_target(qk, vout, t, c0 + lane + 32 * i, tokens, G, D, DP, Dv) = v[i] * mul;
+    if (!is_v) {
+        float* row = dr_target(qk, vout, t, c0, tokens, G, D, DP, Dv);
+        for (int d = D + lane; d < DP; d += 32) row[d] = 0.f;
+    }
 }
 
 // The same for four taps and heads of 32 VEC channels, a warp taking DR_RUN consecutive tokens of a unit.  Where all of them
@@ -127,9 +142,10 @@ template <typename T, int VEC>
 __global__ void __launch_bounds__(128)
 delta_conv_run_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ w, const float* __restrict__ ring,
                       const int* __restrict__ seq_of_token, const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots,
-                      const int* __restrict__ positions, float* __restrict__ y, int tokens, int G, int HDv, float q_mul, int units) {
-    constexpr int TAPS = 4, D = 32 * VEC;
-    const int C = 2 * G * D + HDv;
+                      const int* __restrict__ positions, float* __restrict__ qk, float* __restrict__ vout, int tokens, int G, int H, int Dv,
+                      float q_mul, int units) {
+    constexpr int TAPS = 4, D = 32 * VEC, DP = dr_padded(D);
+    const int C = 2 * G * D + H * Dv;
     const int lane = threadIdx.x & 31;
     const long long id = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
     const int unit = (int)(id % units), t0 = (int)(id / units) * DR_RUN;
@@ -147,6 +163,7 @@ delta_conv_run_kernel(const T* __restrict__ x, int ldx, const float* __restrict_
     pdl_wait();
     pdl_trigger();
     const int seq = seq_of_token[t0], first = cu_seqlens[seq], last = cu_seqlens[seq + 1];
+    float* const target = live ? dr_target(qk, vout, t0, c, tokens, G, D, DP, Dv) - (size_t)t0 * (is_v ? 8 : 2 * DP) : nullptr;
     auto finish = [&](int t, float (&o)[VEC]) {
         if (!is_v) {   // (a warp holds one unit)
             float ss = 0.f;
@@ -156,7 +173,8 @@ delta_conv_run_kernel(const T* __restrict__ x, int ldx, const float* __restrict_
 #pragma unroll
             for (int e = 0; e < VEC; ++e) o[e] *= mul;
         }
-        if (live) dr_store<VEC>(y + (size_t)t * C + c, o);
+        if (live) dr_store<VEC>(target + (size_t)t * (is_v ? 8 : 2 * DP), o);
+        if (D < DP && !is_v) target[(size_t)t * 2 * DP + D] = 0.f;   // (heads of 32: a lane's channel, and the pad beside it)
     };
     if (t0 - first >= TAPS - 1 && t0 + DR_RUN <= last) {
         float win[DR_RUN + TAPS - 1][VEC];
@@ -192,42 +210,43 @@ delta_conv_run_kernel(const T* __restrict__ x, int ldx, const float* __restrict_
 
 template <typename T>
 static int launch_delta_conv(const T* x, int ldx, const float* w, const float* ring, const int* seq_of_token, const int* cu_seqlens,
-                             const int* state_slots, const int* positions, float* y, int tokens, int G, int D, int H, int Dv, int taps,
+                             const int* state_slots, const int* positions, float* qk, float* v, int tokens, int G, int D, int H, int Dv, int taps,
                              float q_mul, cudaStream_t stream) {
     const int HDv = H * Dv, vec = D / 32, C = 2 * G * D + HDv;
-    const bool run = taps == 4 && (D == 32 || D == 64 || D == 128) && tokens > 1 && HDv % vec == 0 && ldx % vec == 0 &&
-                     !(((uintptr_t)x | (uintptr_t)w | (uintptr_t)ring | (uintptr_t)y) & 15) && C % vec == 0;
+    const bool run = taps == 4 && (D == 32 || D == 64 || D == 128) && tokens > 1 && Dv % vec == 0 && ldx % vec == 0 &&
+                     !(((uintptr_t)x | (uintptr_t)w | (uintptr_t)ring) & 15) && C % vec == 0;
     const int units = 2 * G + (run ? (HDv + D - 1) / D : (HDv + 255) / 256);
     const long long warps = (long long)units * (run ? (tokens + DR_RUN - 1) / DR_RUN : tokens);
     if ((warps + 3) / 4 > 0x7fffffffLL) return VX_ERR_LIMIT;
     const unsigned blocks = (unsigned)((warps + 3) / 4);
 #define DR_GO(V_) VX_LAUNCH_K(VX_K_ELEMENTWISE, (delta_conv_run_kernel<T, V_>), blocks, 128, 0, stream, x, ldx, w, ring, seq_of_token, \
-                              cu_seqlens, state_slots, positions, y, tokens, G, HDv, q_mul, units)
+                              cu_seqlens, state_slots, positions, qk, v, tokens, G, H, Dv, q_mul, units)
     if (run && vec == 1) DR_GO(1);
     else if (run && vec == 2) DR_GO(2);
     else if (run) DR_GO(4);
     else
         VX_LAUNCH_K(VX_K_ELEMENTWISE, (delta_conv_any_kernel<T>), blocks, 128, 0, stream, x, ldx, w, ring, seq_of_token, cu_seqlens,
-                    state_slots, positions, y, tokens, G, D, HDv, taps, q_mul, units);
+                    state_slots, positions, qk, v, tokens, G, D, H, Dv, taps, q_mul, units);
 #undef DR_GO
     VX_LAUNCH_CHECK();
     return VX_OK;
 }
 
 // x [tokens, ldx]: the projections q [G, D], k [G, D], v [H, Dv] from column 0 on.  w float32 [taps, C] (the last row is the
-// current token's), ring float32 [slots, taps, C] (read only).
+// current token's), ring float32 [slots, taps, C] (read only).  qk, v: see above, 16-byte aligned.
 extern "C" int vx_delta_conv(const void* x, int ldx, const float* w, const float* ring, const int* seq_of_token,
-                             const int* cu_seqlens, const int* state_slots, const int* positions, float* y, int tokens,
+                             const int* cu_seqlens, const int* state_slots, const int* positions, float* qk, float* v, int tokens,
                              int G, int D, int H, int Dv, int taps, float q_mul, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return VX_OK;
     if (G <= 0 || D <= 0 || H <= 0 || Dv <= 0 || H % G || taps <= 0 || ldx < 2 * G * D + H * Dv) return VX_ERR_SHAPE;
     if (D > 256 || taps > DR_MAX_TAPS) return VX_ERR_LIMIT;
+    if (((uintptr_t)qk | (uintptr_t)v) & 15) return VX_ERR_ALIGN;
     if (dtype == VX_F32)
-        return launch_delta_conv<float>((const float*)x, ldx, w, ring, seq_of_token, cu_seqlens, state_slots, positions, y, tokens, G, D,
-                                        H, Dv, taps, q_mul, stream);
+        return launch_delta_conv<float>((const float*)x, ldx, w, ring, seq_of_token, cu_seqlens, state_slots, positions, qk, v, tokens, G,
+                                        D, H, Dv, taps, q_mul, stream);
     if (dtype == VX_BF16)
-        return launch_delta_conv<bf16>((const bf16*)x, ldx, w, ring, seq_of_token, cu_seqlens, state_slots, positions, y, tokens, G, D, H,
-                                       Dv, taps, q_mul, stream);
+        return launch_delta_conv<bf16>((const bf16*)x, ldx, w, ring, seq_of_token, cu_seqlens, state_slots, positions, qk, v, tokens, G, D,
+                                       H, Dv, taps, q_mul, stream);
     return VX_ERR_DTYPE;
 }
 
@@ -277,9 +296,9 @@ __device__ __forceinline__ float dr_sums(float (&p)[8 * CC], int lane) {
 
 #define DR_CW 4   // warps of a block
 __global__ void __launch_bounds__(DR_CW * 32)
-delta_coef_kernel(const float* __restrict__ y, const float* __restrict__ ab, int ldab, int a_col, int b_col,
+delta_coef_kernel(const float* __restrict__ qkv, const float* __restrict__ ab, int ldab, int a_col, int b_col,
                   const float* __restrict__ neg_exp_a, const float* __restrict__ dt_bias, const int* __restrict__ seq_of_token,
-                  const int* __restrict__ cu_seqlens, float* __restrict__ coef, int tokens, int G, int D, int H, int C) {
+                  const int* __restrict__ cu_seqlens, float* __restrict__ coef, int tokens, int G, int D, int H) {
     __shared__ float kk_s[DR_CW][64], qk_s[DR_CW][64], a_s[DR_CW][4][64];
     pdl_wait();
     pdl_trigger();
@@ -304,9 +323,9 @@ delta_coef_kernel(const float* __restrict__ y, const float* __restrict__ ab, int
             float kr[DR_MINI], qr[DR_MINI];
 #pragma unroll
             for (int r = 0; r < DR_MINI; ++r) {
-                const float* src = y + (size_t)(t + r) * C + kvh * D + d;
+                const float* src = qkv + ((size_t)kvh * tokens + t + r) * 2 * dr_padded(D) + d;
                 qr[r] = r < n ? src[0] : 0.f;
-                kr[r] = r < n ? src[G * D] : 0.f;
+                kr[r] = r < n ? src[dr_padded(D)] : 0.f;
             }
 #pragma unroll
             for (int a = 0; a < DR_MINI; ++a)
@@ -357,14 +376,14 @@ delta_coef_kernel(const float* __restrict__ y, const float* __restrict__ ab, int
             }
             if (mine) {
                 if (i < n) {
-                    float* dst = coef + ((size_t)(t + i) * H + h) * DR_COEF;
+                    float* dst = coef + ((size_t)h * tokens + t + i) * DR_COEF;
                     *reinterpret_cast<float4*>(dst) = make_float4(beta, beta * gamma, gamma, after);
 #pragma unroll
                     for (int j = 0; j < DR_MINI; ++j) dst[12 + j] = j <= i ? rho[j] * qk[i * (i + 1) / 2 + j] : 0.f;
                 }
 #pragma unroll
                 for (int a = 0; a < DR_MINI; ++a)
-                    if (a < n) coef[((size_t)(t + a) * H + h) * DR_COEF + 4 + i] = T[a];
+                    if (a < n) coef[((size_t)h * tokens + t + a) * DR_COEF + 4 + i] = T[a];
             }
         }
         __syncwarp();
@@ -378,14 +397,17 @@ delta_coef_kernel(const float* __restrict__ y, const float* __restrict__ ab, int
 // columns (in an order of the tokens of its own), the 8 CC of either kind are summed over the lanes together, and lane 8 c + i ends
 // with those of token i and column c.
 // u = (I + A)^-1 r is then eight products of numbers that the column's eight lanes exchange, and its multiples go through shared
-// memory to all lanes for the update.  Tokens are staged DR_CHUNK at a time by asynchronous copies, a chunk ahead.  Rows past D
-// are zeros, tokens past a request's last have zero coefficients: they change nothing.
-#define DR_VROW(COLS) ((COLS) + 4)   // (a staged token's values lie 20 or 12 numbers apart: eight tokens by four columns miss each other's banks)
+// memory to all lanes for the update.  Tokens are staged DR_CHUNK at a time by bulk copies that one thread asks for, a chunk ahead.  Rows
+// past D are zeros, tokens past a request's last have zero coefficients: they change nothing.
 #define DR_CHUNK 16
-#define DR_SMEM(DP, COLS) (sizeof(float) * (2 * DR_CHUNK * (2 * (DP) + DR_VROW(COLS) + DR_COEF) + 2 * DR_MINI * (COLS) * 2))
+#define DR_SMEM(DP, COLS) (sizeof(float) * (2 * DR_CHUNK * (2 * (DP) + (COLS) + DR_COEF) + 2 * DR_MINI * (COLS) * 2))
+#define DR_SM_SMEM ((size_t)226 * 1024)   // what an SM's blocks share (a block's own limit is 227 KB with its static part)
+#define DR_ERR_WALK 21
 
-__device__ __forceinline__ void dr_copy4(float* dst, const float* src) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+// Contiguous bytes from memory into shared memory, counted on an mbarrier (16-byte aligned, a multiple of 16 bytes).
+__device__ __forceinline__ void dr_bulk(float* dst, const float* src, unsigned bytes, unsigned bar) {
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];\n"
+                 ::"r"(tc_smem_u32(dst)), "l"(src), "r"(bytes), "r"(bar) : "memory");
 }
 
 typedef unsigned long long dr_pair;   // two floats in a register pair
@@ -421,26 +443,46 @@ template <int P> __device__ __forceinline__ void dr_pairs(const float* p, dr_pai
 
 template <int RL, int CC, int COLS>
 __global__ void __launch_bounds__(COLS / CC * 32, 1)
-delta_walk_kernel(const float* __restrict__ y, const float* __restrict__ coef, float* __restrict__ state, float* __restrict__ ring,
-                  const void* __restrict__ x, int ldx, int x_bf16, const int* __restrict__ cu_seqlens,
-                  const int* __restrict__ state_slots, const int* __restrict__ positions, float* __restrict__ out, int G, int D, int H,
-                  int Dv, int taps) {
+delta_walk_kernel(const float* __restrict__ qk, const float* __restrict__ v, const float* __restrict__ coef, float* __restrict__ state,
+                  float* __restrict__ ring, const void* __restrict__ x, int ldx, int x_bf16, const int* __restrict__ cu_seqlens,
+                  const int* __restrict__ state_slots, const int* __restrict__ positions, float* __restrict__ out, int tokens, int G,
+                  int D, int H, int Dv, int taps, int* __restrict__ error) {
     extern __shared__ __align__(16) float dr_smem[];
-    constexpr int DP = 32 * RL, P = RL / 2, THREADS = COLS / CC * 32, NV = 8 * CC, VROW = DR_VROW(COLS);
-    float* q_s = dr_smem;                              // [2][DR_CHUNK][DP]
-    float* k_s = q_s + 2 * DR_CHUNK * DP;              // [2][DR_CHUNK][DP]
-    float* v_s = k_s + 2 * DR_CHUNK * DP;              // [2][DR_CHUNK][VROW]
-    float* c_s = v_s + 2 * DR_CHUNK * VROW;         // [2][DR_CHUNK][DR_COEF]
+    __shared__ __align__(8) unsigned long long full_bar[2];
+    __shared__ int failed;
+    constexpr int DP = 32 * RL, P = RL / 2, THREADS = COLS / CC * 32, NV = 8 * CC;
+    float* qk_s = dr_smem;                             // [2][DR_CHUNK][2][DP]
+    float* v_s = qk_s + 2 * DR_CHUNK * 2 * DP;         // [2][COLS / 8][DR_CHUNK][8]
+    float* c_s = v_s + 2 * DR_CHUNK * COLS;            // [2][DR_CHUNK][DR_COEF]
     float* u_s = c_s + 2 * DR_CHUNK * DR_COEF;         // [warps][2][DR_MINI][CC] twice each
     const int col0 = blockIdx.x * COLS, h = blockIdx.y, seq = blockIdx.z;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, ti = lane & 7, tc = (lane >> 3) & (CC - 1);
-    const int kvh = h / (H / G), C = 2 * G * D + H * Dv;
-    for (int i = threadIdx.x; i < 2 * DR_CHUNK * (2 * DP + VROW + DR_COEF); i += THREADS) dr_smem[i] = 0.f;
+    const int kvh = h / (H / G), C = 2 * G * D + H * Dv, vblocks = (Dv + 7) >> 3;
+    for (int i = threadIdx.x; i < 2 * DR_CHUNK * (2 * DP + COLS + DR_COEF); i += THREADS) dr_smem[i] = 0.f;
+    if (threadIdx.x == 0) {
+        tc_mbar_init(tc_smem_u32(&full_bar[0]), 1);
+        tc_mbar_init(tc_smem_u32(&full_bar[1]), 1);
+        failed = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
+    }
+    asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");   // (the zeros before what the copies write)
+    __syncthreads();
     pdl_wait();
     pdl_trigger();
     const int t0 = cu_seqlens[seq], t1 = cu_seqlens[seq + 1], slot = state_slots[seq];
-    const bool wide = ((D | C | Dv) & 3) == 0 && !(((uintptr_t)y) & 15);
     float* st = state + ((size_t)slot * H + h) * (size_t)Dv * D;
+
+    // one thread asks for a chunk: the keys and queries, eight columns of values at a time, the coefficients
+    auto stage = [&](int buf, int tb) {
+        const int n = min(DR_CHUNK, t1 - tb), vb = min(COLS / 8, vblocks - col0 / 8);
+        const unsigned bar = tc_smem_u32(&full_bar[buf]);
+        tc_mbar_expect_tx(bar, (unsigned)(n * (2 * DP + vb * 8 + DR_COEF) * 4));
+        dr_bulk(qk_s + buf * DR_CHUNK * 2 * DP, qk + ((size_t)kvh * tokens + tb) * 2 * DP, n * 2 * DP * 4, bar);
+        for (int b = 0; b < vb; ++b)
+            dr_bulk(v_s + (buf * (COLS / 8) + b) * DR_CHUNK * 8, v + (((size_t)h * vblocks + col0 / 8 + b) * tokens + tb) * 8, n * 32, bar);
+        dr_bulk(c_s + buf * DR_CHUNK * DR_COEF, coef + ((size_t)h * tokens + tb) * DR_COEF, n * DR_COEF * 4, bar);
+    };
+    if (threadIdx.x == 0 && t1 > t0) stage(0, t0);
     dr_pair S[CC][P];
 #pragma unroll
     for (int c = 0; c < CC; ++c) {
@@ -451,84 +493,23 @@ delta_walk_kernel(const float* __restrict__ y, const float* __restrict__ coef, f
 #pragma unroll
         for (int p = 0; p < P; ++p) S[c][p] = dr_pack(s[2 * p], s[2 * p + 1]);
     }
-    __syncthreads();   // (the zeros are there before the first copies)
-
-    auto stage = [&](int buf, int tb) {
-        const int n = min(DR_CHUNK, t1 - tb);
-        float *qd = q_s + buf * DR_CHUNK * DP, *kd = k_s + buf * DR_CHUNK * DP, *vd = v_s + buf * DR_CHUNK * VROW;
-        float* cd = c_s + buf * DR_CHUNK * DR_COEF;
-        const int vn = min(COLS, Dv - col0);
-        if (wide && D == DP && n == DR_CHUNK && vn == COLS) {   // (sizes that are known: no divisions)
-            const float* src0 = y + (size_t)tb * C + kvh * D;
-#pragma unroll
-            for (int it = 0; it < (DR_CHUNK * DP / 4 + THREADS - 1) / THREADS; ++it) {
-                const int i = threadIdx.x + it * THREADS, tt = i / (DP / 4), d = (i % (DP / 4)) * 4;
-                if (DR_CHUNK * DP / 4 % THREADS == 0 || i < DR_CHUNK * DP / 4) {
-                    cp_async16(qd + tt * DP + d, src0 + (size_t)tt * C + d);
-                    cp_async16(kd + tt * DP + d, src0 + (size_t)tt * C + G * D + d);
-                }
-            }
-            if (threadIdx.x < DR_CHUNK * COLS / 4) {
-                const int tt = threadIdx.x / (COLS / 4), c = (threadIdx.x % (COLS / 4)) * 4;
-                cp_async16(vd + tt * VROW + c, y + (size_t)(tb + tt) * C + 2 * G * D + h * Dv + col0 + c);
-            }
-            static_assert(THREADS >= DR_CHUNK * (DR_COEF / 4) && THREADS >= DR_CHUNK * COLS / 4, "a thread copies one piece of the coefficients and values");
-            if (threadIdx.x < DR_CHUNK * (DR_COEF / 4)) {
-                const int tt = threadIdx.x / (DR_COEF / 4), c = (threadIdx.x % (DR_COEF / 4)) * 4;
-                cp_async16(cd + tt * DR_COEF + c, coef + ((size_t)(tb + tt) * H + h) * DR_COEF + c);
-            }
-            cp_async_commit();
-            return;
-        }
-        if (wide) {
-            const int d4 = D >> 2, v4 = vn >> 2;
-            for (int i = threadIdx.x; i < n * d4; i += THREADS) {
-                const int tt = i / d4, d = (i - tt * d4) * 4;
-                const float* src = y + (size_t)(tb + tt) * C + kvh * D + d;
-                cp_async16(qd + tt * DP + d, src);
-                cp_async16(kd + tt * DP + d, src + G * D);
-            }
-            for (int i = threadIdx.x; i < n * v4; i += THREADS) {
-                const int tt = i / v4, c = (i - tt * v4) * 4;
-                cp_async16(vd + tt * VROW + c, y + (size_t)(tb + tt) * C + 2 * G * D + h * Dv + col0 + c);
-            }
-        } else {
-            for (int i = threadIdx.x; i < n * D; i += THREADS) {
-                const int tt = i / D, d = i - tt * D;
-                const float* src = y + (size_t)(tb + tt) * C + kvh * D + d;
-                dr_copy4(qd + tt * DP + d, src);
-                dr_copy4(kd + tt * DP + d, src + G * D);
-            }
-            for (int i = threadIdx.x; i < n * vn; i += THREADS) {
-                const int tt = i / vn, c = i - tt * vn;
-                dr_copy4(vd + tt * VROW + c, y + (size_t)(tb + tt) * C + 2 * G * D + h * Dv + col0 + c);
-            }
-        }
-        for (int i = threadIdx.x; i < n * (DR_COEF / 4); i += THREADS) {
-            const int tt = i / (DR_COEF / 4), c = (i - tt * (DR_COEF / 4)) * 4;
-            cp_async16(cd + tt * DR_COEF + c, coef + ((size_t)(tb + tt) * H + h) * DR_COEF + c);
-        }
-        for (int i = threadIdx.x; i < (DR_CHUNK - n) * DP; i += THREADS) {
-            qd[n * DP + i] = 0.f;
-            kd[n * DP + i] = 0.f;
-        }
-        for (int i = threadIdx.x; i < (DR_CHUNK - n) * VROW; i += THREADS) vd[n * VROW + i] = 0.f;
-        for (int i = threadIdx.x; i < (DR_CHUNK - n) * DR_COEF; i += THREADS) cd[n * DR_COEF + i] = 0.f;
-        cp_async_commit();
-    };
-
     int off[DR_MINI];   // where a lane's slot s finds its rows: token s xor (lane mod 8) of the mini-chunk
 #pragma unroll
-    for (int i = 0; i < DR_MINI; ++i) off[i] = (i ^ ti) * DP + RL * lane;
-    if (t1 > t0) stage(0, t0);
-    int buf = 0;
-    for (int tb = t0; tb < t1; tb += DR_CHUNK, buf ^= 1) {
+    for (int i = 0; i < DR_MINI; ++i) off[i] = (i ^ ti) * 2 * DP + RL * lane;
+    int buf = 0, uses = 0;
+    for (int tb = t0; tb < t1; tb += DR_CHUNK, buf ^= 1, ++uses) {
         const int n = min(DR_CHUNK, t1 - tb);
-        cp_async_wait<0>();
-        __syncthreads();
-        if (tb + DR_CHUNK < t1) stage(buf ^ 1, tb + DR_CHUNK);
+        if (!tc_mbar_wait(tc_smem_u32(&full_bar[buf]), (unsigned)((uses >> 1) & 1))) {
+            failed = 1;
+            atomicExch(error, DR_ERR_WALK);
+        }
+        // a request's last chunk: what an earlier one left in the rows past its end has coefficients too
+        for (int i = n * DR_COEF + threadIdx.x; i < DR_CHUNK * DR_COEF; i += THREADS) c_s[buf * DR_CHUNK * DR_COEF + i] = 0.f;
+        __syncthreads();   // (and everybody is done with the other buffer)
+        if (failed) break;
+        if (threadIdx.x == 0 && tb + DR_CHUNK < t1) stage(buf ^ 1, tb + DR_CHUNK);
         for (int m = 0; m < n; m += DR_MINI) {
-            const float *qb = q_s + (buf * DR_CHUNK + m) * DP, *kb = k_s + (buf * DR_CHUNK + m) * DP;
+            const float *qb = qk_s + (buf * DR_CHUNK + m) * 2 * DP, *kb = qb + DP;
             const float* cb = c_s + (buf * DR_CHUNK + m + ti) * DR_COEF;
             constexpr bool KEEP = RL <= 4;   // the keys stay in registers from the products to the update
             dr_pair kreg[KEEP ? DR_MINI : 1][P];
@@ -571,8 +552,9 @@ delta_walk_kernel(const float* __restrict__ y, const float* __restrict__ coef, f
             const float4 pa = *reinterpret_cast<const float4*>(cb + 12), pb4 = *reinterpret_cast<const float4*>(cb + 16);
             const float trow[8] = {ta.x, ta.y, ta.z, ta.w, tb4.x, tb4.y, tb4.z, tb4.w};
             const float prow[8] = {pa.x, pa.y, pa.z, pa.w, pb4.x, pb4.y, pb4.z, pb4.w};
-            const float v = v_s[(buf * DR_CHUNK + m + ti) * VROW + warp * CC + tc];
-            const float r = fmaf(c0.x, v, -c0.y * kS);
+            const int cl = warp * CC + tc;
+            const float vt = v_s[((buf * (COLS / 8) + (cl >> 3)) * DR_CHUNK + m + ti) * 8 + (cl & 7)];
+            const float r = fmaf(c0.x, vt, -c0.y * kS);
             float u0 = 0.f, u1 = 0.f;
 #pragma unroll
             for (int j = 0; j < 8; j += 2) {
@@ -637,8 +619,8 @@ delta_walk_kernel(const float* __restrict__ y, const float* __restrict__ coef, f
 }
 
 // neg_exp_a, dt_bias float32 [H]: -exp(A_log) and the decay's offset.  ab float32 [tokens, ldab]: a and b of head h in columns
-// a_col + h, b_col + h.  y: from `vx_delta_conv` of the same step.  coef float32 [tokens, H, 20], 16-byte aligned.
-extern "C" int vx_delta_coef(const float* y, const float* ab, int ldab, int a_col, int b_col, const float* neg_exp_a,
+// a_col + h, b_col + h.  qk: from `vx_delta_conv` of the same step.  coef float32 [H, tokens, 20], 16-byte aligned.
+extern "C" int vx_delta_coef(const float* qk, const float* ab, int ldab, int a_col, int b_col, const float* neg_exp_a,
                              const float* dt_bias, const int* seq_of_token, const int* cu_seqlens, float* coef, int tokens, int G, int D,
                              int H, int Dv, cudaStream_t stream) {
     if (tokens <= 0) return VX_OK;
@@ -646,45 +628,52 @@ extern "C" int vx_delta_coef(const float* y, const float* ab, int ldab, int a_co
     if (((uintptr_t)coef) & 15) return VX_ERR_ALIGN;
     const long long warps = (long long)((tokens + DR_MINI - 1) / DR_MINI) * G;
     if (warps / DR_CW > 0x7ffffff0LL) return VX_ERR_LIMIT;
-    VX_LAUNCH_K(VX_K_ELEMENTWISE, delta_coef_kernel, (unsigned)((warps + DR_CW - 1) / DR_CW), DR_CW * 32, 0, stream, y, ab, ldab, a_col,
-                b_col, neg_exp_a, dt_bias, seq_of_token, cu_seqlens, coef, tokens, G, D, H, 2 * G * D + H * Dv);
+    VX_LAUNCH_K(VX_K_ELEMENTWISE, delta_coef_kernel, (unsigned)((warps + DR_CW - 1) / DR_CW), DR_CW * 32, 0, stream, qk, ab, ldab, a_col,
+                b_col, neg_exp_a, dt_bias, seq_of_token, cu_seqlens, coef, tokens, G, D, H);
     VX_LAUNCH_CHECK();
     return VX_OK;
 }
 
-// y, coef: from the two entries above; x, ldx: what `vx_delta_conv` read.  state float32 [slots, H, Dv, D], ring float32
-// [slots, taps, C]: read and written.  out float32 [tokens, H * Dv].  layout: warps of two columns in blocks of 8 (1)
-// or 16 (2), warps of four in blocks of 16 (3), or 0 for the kernel's choice.
-extern "C" int vx_delta_walk(const float* y, const float* coef, float* state, float* ring, const void* x, int ldx,
-                             const int* cu_seqlens, const int* state_slots, const int* positions, float* out, int seqs, int G, int D,
-                             int H, int Dv, int taps, int layout, int dtype, cudaStream_t stream) {
+// qk, v, coef: from the two entries above; x, ldx: what `vx_delta_conv` read.  state float32 [slots, H, Dv, D], ring float32
+// [slots, taps, C]: read and written.  out float32 [tokens, H * Dv].  layout: warps of two columns in blocks of 8 (1),
+// warps of four in blocks of 16 (2), or 0 for the kernel's choice.  `error`: a device int that a block sets if its wait
+// for its own copies runs out.
+extern "C" int vx_delta_walk(const float* qk, const float* v, const float* coef, float* state, float* ring, const void* x, int ldx,
+                             const int* cu_seqlens, const int* state_slots, const int* positions, float* out, int tokens, int seqs, int G,
+                             int D, int H, int Dv, int taps, int layout, int* error, int dtype, cudaStream_t stream) {
     if (seqs <= 0) return VX_OK;
     if (G <= 0 || D <= 0 || H <= 0 || Dv <= 0 || H % G || taps <= 0 || ldx < 2 * G * D + H * Dv) return VX_ERR_SHAPE;
     if (D > 256 || taps > DR_MAX_TAPS || seqs > 65535 || H > 65535) return VX_ERR_LIMIT;
     if (dtype != VX_F32 && dtype != VX_BF16) return VX_ERR_DTYPE;
-    if (((uintptr_t)coef) & 15) return VX_ERR_ALIGN;
-    static bool configured[9][VX_MAX_DEVICES];
+    if (((uintptr_t)qk | (uintptr_t)v | (uintptr_t)coef) & 15) return VX_ERR_ALIGN;
+    if (!error || tokens <= 0) return VX_ERR_SHAPE;
+    static bool configured[6][VX_MAX_DEVICES];
     static int sms[VX_MAX_DEVICES];
-    // few heads: warps of two columns, in blocks of 8 or 16; many: warps of four (what a column's sums are does not depend on it)
+    // few heads: warps of two columns, blocks of 8; many: warps of four, blocks of 16 (a column's sums do not depend on it)
     const long long units = (long long)H * seqs * ((Dv + 7) / 8);
-    if (!layout) layout = units <= vx_sm_count(sms) ? 1 : (units <= 2LL * vx_sm_count(sms) ? 2 : 3);
-    if (layout < 0 || layout > 3) return VX_ERR_SHAPE;
+    if (!layout) layout = D <= 128 && units <= 2LL * vx_sm_count(sms) ? 1 : 2;
+    if (layout < 0 || layout > 2) return VX_ERR_SHAPE;
     const int cols = layout == 1 ? 8 : 16;
     dim3 grid((Dv + cols - 1) / cols, H, seqs);
+    // as much shared memory a block as lets no SM take more blocks than its share: these blocks become resident while the kernel
+    // before them still runs, and would crowd on the SMs that are free first
+    const long long share = ((long long)grid.x * grid.y * grid.z + vx_sm_count(sms) - 1) / vx_sm_count(sms);
+    const size_t spread = share <= 4 ? DR_SM_SMEM / share - 2048 : 0;
 #define DR_GO(RL_, CC_, COLS_, SLOT)                                                                                            \
     do {                                                                                                                        \
-        if (int rc = vx_configure_smem(delta_walk_kernel<RL_, CC_, COLS_>, DR_SMEM(32 * RL_, COLS_), configured[SLOT])) return rc; \
-        VX_LAUNCH_K(VX_K_ATTENTION, (delta_walk_kernel<RL_, CC_, COLS_>), grid, COLS_ / CC_ * 32, DR_SMEM(32 * RL_, COLS_), stream, \
-                    y, coef, state, ring, x, ldx, dtype == VX_BF16 ? 1 : 0, cu_seqlens, state_slots, positions, out, G, D, H, Dv,  \
-                    taps);                                                                                                      \
+        if (int rc = vx_configure_smem(delta_walk_kernel<RL_, CC_, COLS_>, DR_SM_SMEM, configured[SLOT])) return rc;           \
+        const size_t need = DR_SMEM(32 * RL_, COLS_);                                                                           \
+        VX_LAUNCH_K(VX_K_ATTENTION, (delta_walk_kernel<RL_, CC_, COLS_>), grid, COLS_ / CC_ * 32, need > spread ? need : spread, stream, \
+                    qk, v, coef, state, ring, x, ldx, dtype == VX_BF16 ? 1 : 0, cu_seqlens, state_slots, positions, out, tokens, G, \
+                    D, H, Dv, taps, error);                                                                                    \
     } while (0)
 #define DR_GO_CC(RL_, SLOT)                                                                                                    \
     do {                                                                                                                       \
-        if (layout == 1) DR_GO(RL_, 2, 8, SLOT); else if (layout == 2) DR_GO(RL_, 2, 16, SLOT + 1); else DR_GO(RL_, 4, 16, SLOT + 2); \
+        if (layout == 1) DR_GO(RL_, 2, 8, SLOT); else DR_GO(RL_, 4, 16, SLOT + 1);                                             \
     } while (0)
     if (D <= 64) DR_GO_CC(2, 0);
-    else if (D <= 128) DR_GO_CC(4, 3);
-    else DR_GO_CC(8, 6);
+    else if (D <= 128) DR_GO_CC(4, 2);
+    else DR_GO_CC(8, 4);
 #undef DR_GO_CC
 #undef DR_GO
     VX_LAUNCH_CHECK();

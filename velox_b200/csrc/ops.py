@@ -136,9 +136,9 @@ def _declare(lib) -> None:
         "vx_gemm_skinny_inputs": [P, P, P, I, I, I, I, I, I, I, c_longlong, I, I, P],
         "vx_moe_gemm_scaled": [P, I, P, I, P, P, P, I, P, I, I, I, I, I, I, I, I, I, P, P],
         "vx_moe_gemm_tcgen05_scaled": [P, P, P, I, I, I, I, I, I, I, I, P, P, I, P, P, P, I, P],
-        "vx_delta_conv": [P, I, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, P],
+        "vx_delta_conv": [P, I, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, P],
         "vx_delta_coef": [P, P, I, I, I, P, P, P, P, P, I, I, I, I, I, P],
-        "vx_delta_walk": [P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, P],
+        "vx_delta_walk": [P, P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, P, I, P],
         "vx_delta_decode": [P, I, I, P, I, I, I, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, I, I, P],
         "vx_head_gate": [P, I, P, I, P, I, I, I, I, I, P],
         "vx_moe_route_groups": [P, I, P, P, I, I, I, I, I, P, P, P, P, P, P, P, P, P, I, I, P, I, I, F, I, P, I, I, P],
@@ -1471,18 +1471,21 @@ def delta_rule(x: torch.Tensor, ab: torch.Tensor, a_col: int, b_col: int, taps_w
     c, taps = _delta_check("delta_rule", x, taps_w, ring, groups, dim, heads, vdim, ab)
     _delta_state_check("delta_rule", state, heads, dim, vdim, neg_exp_a, dt_bias)
     tokens, dev = x.shape[0], x.device
-    y = torch.empty((tokens, c), dtype=torch.float32, device=dev)
-    coef = torch.empty((tokens, heads, _DELTA_COEF), dtype=torch.float32, device=dev)
+    padded = 64 if dim <= 64 else (128 if dim <= 128 else 256)
+    qk = torch.empty((groups, tokens, 2, padded), dtype=torch.float32, device=dev)
+    v = torch.empty((heads, -(-vdim // 8), tokens, 8), dtype=torch.float32, device=dev)
+    coef = torch.empty((heads, tokens, _DELTA_COEF), dtype=torch.float32, device=dev)
     out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=dev)
     _check(library().vx_delta_conv(_ptr(x), x.stride(0), _ptr(taps_w), _ptr(ring), _ptr(ctx.seq_of_token), _ptr(ctx.cu_seqlens),
-                                   _ptr(ctx.state_slots), _ptr(ctx.positions), _ptr(y), tokens, groups, dim, heads, vdim, taps,
-                                   float(q_mul), dtype_code(x.dtype), _stream()), "delta_conv")
-    _check(library().vx_delta_coef(_ptr(y), _ptr(ab), ab.stride(0), int(a_col), int(b_col), _ptr(neg_exp_a), _ptr(dt_bias),
+                                   _ptr(ctx.state_slots), _ptr(ctx.positions), _ptr(qk), _ptr(v), tokens, groups, dim, heads, vdim,
+                                   taps, float(q_mul), dtype_code(x.dtype), _stream()), "delta_conv")
+    _check(library().vx_delta_coef(_ptr(qk), _ptr(ab), ab.stride(0), int(a_col), int(b_col), _ptr(neg_exp_a), _ptr(dt_bias),
                                    _ptr(ctx.seq_of_token), _ptr(ctx.cu_seqlens), _ptr(coef), tokens, groups, dim, heads, vdim,
                                    _stream()), "delta_coef")
-    _check(library().vx_delta_walk(_ptr(y), _ptr(coef), _ptr(state), _ptr(ring), _ptr(x), x.stride(0), _ptr(ctx.cu_seqlens),
-                                   _ptr(ctx.state_slots), _ptr(ctx.positions), _ptr(out), ctx.n_seqs, groups, dim, heads, vdim,
-                                   taps, int(layout), dtype_code(x.dtype), _stream()), "delta_walk")
+    _check(library().vx_delta_walk(_ptr(qk), _ptr(v), _ptr(coef), _ptr(state), _ptr(ring), _ptr(x), x.stride(0), _ptr(ctx.cu_seqlens),
+                                   _ptr(ctx.state_slots), _ptr(ctx.positions), _ptr(out), tokens, ctx.n_seqs, groups, dim, heads, vdim,
+                                   taps, int(layout), _ptr(_error_word(dev)), dtype_code(x.dtype), _stream()), "delta_walk")
+    note_bounded_wait()
     return out
 
 
