@@ -108,7 +108,7 @@ def test_a_random_model_folder_can_be_written_and_read_back(tmp_path):
 
 
 def test_parts_refuse_what_they_cannot_do():
-    from velox_b200.parts import GatedDeltaRule, LatentAttention, PartSpec, RoutedExperts
+    from velox_b200.parts import GatedDeltaRule, LatentAttention, PartSpec, PreNormBlock, RoutedExperts
     sizes = dict(hidden_size=64, num_heads=4, num_kv_heads=2, head_dim=32, v_head_dim=32, conv_taps=4)
     GatedDeltaRule("x.", **sizes)
     for change in (dict(num_kv_heads=3), dict(head_dim=257), dict(v_head_dim=0), dict(conv_taps=65)):
@@ -118,6 +118,8 @@ def test_parts_refuse_what_they_cannot_do():
         LatentAttention("x.", 64, 2, 16, 8, 16, 32, 0.2, PartSpec("rotary", "", dict(head_dim=8, theta=100.0)), output_gate=True, head_gate=True)
     with pytest.raises(ValueError, match="bounded gate"):
         RoutedExperts("x.", 64, 4, 2, 32, scores="sigmoid", gated=False, names=("up", "down"), capped=(1.0, 1.7))
+    with pytest.raises(ValueError, match="needs a feed-forward"):
+        PreNormBlock(GatedDeltaRule("x.", **sizes), None, {"mixer": None, "feed_forward": None})
     with pytest.raises(ValueError, match="renormalised"):
         RoutedExperts("x.", 64, 4, 2, 32, renormalise=True)
 

@@ -81,6 +81,8 @@ class PreNormBlock(Block):
 
     def __init__(self, mixer, feed_forward, norms):
         self.norm_names = ("mixer",) + (("feed_forward",) if feed_forward is not None else ())
+        if feed_forward is None and "feed_forward" in norms:
+            raise ValueError("PreNormBlock with a norm before its feed-forward needs a feed-forward; the layer's plan gives none")
         super().__init__(mixer, feed_forward, norms)
 
     def forward(self, residual, delta, ctx, cache):
