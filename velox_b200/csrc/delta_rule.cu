@@ -8,7 +8,7 @@
 //   delta_coef      decays, step sizes, and what follows from them and from the products among keys and queries within
 //                   eight tokens
 //   delta_walk      the recurrence over a step's tokens; afterwards the last inputs of the convolutions go into their slots
-//   delta_decode    a step of single tokens: both of these, the norm of every head's output and its gate in one kernel
+//   delta_decode    a step of single tokens: all of this, the norm of every head's output and its gate in one kernel
 //
 // State per request (float32): S transposed, [H, Dv, D] (a column of S is contiguous), and the last inputs of the
 // convolutions as a ring [taps, channels]: position p lies in row p mod taps.  A token at position p reads rows p - 1 ..
